@@ -30,8 +30,9 @@ typedef struct vkl_model vkl_model;
 typedef struct vkl_gguf vkl_gguf;
 typedef struct vkl_sampler vkl_sampler;
 
-/* src/core/common.h:15-22 (enum DType), same numeric values. */
-enum vkl_dtype { VKL_FP32 = 0, VKL_FP16 = 1, VKL_UINT32 = 2, VKL_INT8 = 3, VKL_Q8_0 = 4 };
+/* src/core/common.h:15-22 (enum DType), same numeric values; BF16 is this library's own
+ * (weights and activations of the layer-list decoder designs, not an operand of the ops). */
+enum vkl_dtype { VKL_FP32 = 0, VKL_FP16 = 1, VKL_UINT32 = 2, VKL_INT8 = 3, VKL_Q8_0 = 4, VKL_BF16 = 5 };
 
 /* absl::StatusCode values used by the reference's ops. */
 enum vkl_status {
@@ -264,6 +265,31 @@ int vkl_model_synth_weights(vkl_model *m, uint64_t seed, float wstd, float nstd)
  * the reference does after clipping Q). */
 int vkl_model_forward(vkl_model *m, const uint32_t *toks, size_t n, size_t offset,
                       float *logits_out);
+/* The same pass with the logits of chosen tokens of the call: rows[i] indexes toks, logits_out is
+ * [n_rows, vocab]. n_rows may be 0 (the pass only extends the caches). A Llama-2 model leaves the
+ * last token's logits only (the reference clips the last block), other rows are UNIMPLEMENTED. */
+int vkl_model_forward_rows(vkl_model *m, const uint32_t *toks, size_t n, size_t offset,
+                           const uint32_t *rows, size_t n_rows, float *logits_out);
+/* The residual stream of a decoder design after every layer run (a looped layer counts every
+ * pass): runs the tokens like vkl_model_forward and writes fp32 [layer runs, n, width]. */
+int vkl_model_trace_layers(vkl_model *m, const uint32_t *toks, size_t n, size_t offset, float *out);
+/* vocabulary, width, layers (layer runs of a decoder design), maxlen, compute dtype, heads. */
+int vkl_model_shape(const vkl_model *m, uint32_t out6[6]);
+/* One layer's (layer run's) key cache: heads, maxlen, head width in memory, dtype. */
+int vkl_model_kv_shape(const vkl_model *m, uint32_t layer, uint32_t out4[4]);
+/* A model from a checkpoint folder: config.json names the architecture and its sizes,
+ * model.safetensors holds the weights (bfloat16, integer tables int32). The architecture is looked
+ * up in the library's registry; maxlen is the context length, compute_dtype VKL_BF16 or VKL_FP32
+ * (everything in true 32-bit). */
+int vkl_model_load_folder(vkl_device *dev, const char *path, uint32_t maxlen, int compute_dtype, vkl_model **out);
+/* The same from the text of a config.json, without weights (vkl_model_set_weight by the
+ * checkpoint's tensor names, BF16 or UINT32, or vkl_model_synth_weights). */
+int vkl_model_create_config(vkl_device *dev, const char *config_json, uint32_t maxlen, int compute_dtype, vkl_model **out);
+/* Names of the registered architectures, separated by commas. */
+const char *vkl_model_architectures(void);
+/* Row of a distance-bias table with `rows` rows for a key n positions back; -1 when the table
+ * cannot reach `far`. */
+int vkl_distance_bucket(uint32_t n, uint32_t rows, uint32_t far);
 /* llama2_infer's loop (app/llama2_infer.cpp:141-210) with the greedy pick kept
  * on the device: prefill `prompt`, then n_gen - 1 one-token steps. With Q8_0 weights a
  * step is one launch of the persistent decode kernel (all ops of the token in one

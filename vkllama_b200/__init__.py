@@ -7,11 +7,11 @@ The shared library is built in-tree by `python -m vkllama_b200.build`; there is
 no fallback when it, or a CUDA device, is missing.
 """
 from .api import (  # noqa: F401
-    FP32, FP16, UINT32, INT8, Q8_0,
+    FP32, FP16, UINT32, INT8, Q8_0, BF16,
     VklError, Device, Tensor, Command,
     MatMul, FeedForward, MultiHeadAttentionV2, UpdateKVCache, RMSNorm, Rope, Softmax,
     ArgOp, ArgMax, ArgMin, Embedding, ElementWise, Transpose, Slice, Cast, Concat, Reduce, ReadKVCache,
     Model, ModelConfig, q8_0_quantize, q8_0_quantize36, q8_0_dequantize, blocks36_to_34,
     kernel_launches, library_path, load_library, matmul_run_many,
-    Gguf, Sampler, TopkSampler, TopPSampler,
+    load_model, architectures, distance_bucket, Gguf, Sampler, TopkSampler, TopPSampler,
 )

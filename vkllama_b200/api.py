@@ -1,11 +1,12 @@
 """ctypes bindings of include/vkllama_b200.h with the reference's class names."""
 import ctypes as C
+import json
 import os
 
 import numpy as np
 
-FP32, FP16, UINT32, INT8, Q8_0 = 0, 1, 2, 3, 4
-_NP = {FP32: np.float32, FP16: np.uint16, UINT32: np.uint32, INT8: np.int8, Q8_0: np.uint8}
+FP32, FP16, UINT32, INT8, Q8_0, BF16 = 0, 1, 2, 3, 4, 5
+_NP = {FP32: np.float32, FP16: np.uint16, UINT32: np.uint32, INT8: np.int8, Q8_0: np.uint8, BF16: np.uint16}
 
 _HERE = os.path.dirname(os.path.abspath(__file__))
 # the in-tree build; VKLLAMA_B200_LIB names another build of the same library (A/B comparisons)
@@ -46,6 +47,7 @@ def load_library():
     L = C.CDLL(_LIB_PATH)
     L.vkl_last_error.restype = C.c_char_p
     L.vkl_kernel_launches.restype = u64
+    L.vkl_model_architectures.restype = C.c_char_p
     sigs = {
         "vkl_device_create": [i32, pvp], "vkl_device_destroy": [vp],
         "vkl_device_info": [vp, C.c_char_p, C.POINTER(i32), C.POINTER(sz)],
@@ -86,6 +88,12 @@ def load_library():
         "vkl_model_set_weight": [vp, C.c_char_p, i32, vp, sz],
         "vkl_model_synth_weights": [vp, u64, f32, f32],
         "vkl_model_forward": [vp, vp, sz, sz, vp],
+        "vkl_model_forward_rows": [vp, vp, sz, sz, vp, sz, vp],
+        "vkl_model_trace_layers": [vp, vp, sz, sz, vp],
+        "vkl_model_shape": [vp, C.POINTER(u32)], "vkl_model_kv_shape": [vp, u32, C.POINTER(u32)],
+        "vkl_model_load_folder": [vp, C.c_char_p, u32, i32, pvp],
+        "vkl_model_create_config": [vp, C.c_char_p, u32, i32, pvp],
+        "vkl_distance_bucket": [u32, u32, u32],
         "vkl_model_generate": [vp, vp, sz, sz, vp, C.POINTER(f32), C.POINTER(f32)],
         "vkl_model_last_token": [vp, C.POINTER(u32)], "vkl_model_read_kv": [vp, u32, vp, vp], "vkl_model_write_kv": [vp, u32, vp, vp],
         "vkl_model_block_forward": [vp, u32, vp, sz, sz, vp],
@@ -116,6 +124,16 @@ def load_library():
 def _ck(status):
     if status != 0:
         raise VklError(status, load_library().vkl_last_error().decode("utf-8", "replace"))
+
+
+def architectures():
+    """Decoder designs that Model.from_folder knows, as config.json names them."""
+    return load_library().vkl_model_architectures().decode().split(",")
+
+
+def distance_bucket(n, rows, far):
+    """Row of a distance-bias table for a key n positions back."""
+    return load_library().vkl_distance_bucket(n, rows, far)
 
 
 def kernel_launches():
@@ -623,11 +641,58 @@ class Model:
                                {0: FP32, 1: FP16, 8: Q8_0}[outw["type"]], tp_rank, max(1, tp_size))
         return self
 
+    @classmethod
+    def from_folder(cls, dev, path, maxlen, compute=BF16):
+        """A registered decoder design from a folder with config.json and model.safetensors."""
+        self = cls.__new__(cls)
+        self.L, self.dev, self.h = load_library(), dev, vp()
+        _ck(self.L.vkl_model_load_folder(dev.h, os.fsencode(path), maxlen, compute, C.byref(self.h)))
+        self._take_shape()
+        return self
+
+    @classmethod
+    def from_config(cls, dev, config, maxlen, compute=BF16):
+        """The same without weights; `config` is the text of a config.json or the object it holds."""
+        self = cls.__new__(cls)
+        self.L, self.dev, self.h = load_library(), dev, vp()
+        text = config if isinstance(config, str) else json.dumps(config)
+        _ck(self.L.vkl_model_create_config(dev.h, text.encode(), maxlen, compute, C.byref(self.h)))
+        self._take_shape()
+        return self
+
+    def _take_shape(self):
+        o = (u32 * 6)()
+        _ck(self.L.vkl_model_shape(self.h, o))
+        self.cfg = ModelConfig(o[1], o[5], 0, o[0], o[2], o[3], 0.0, 0.0, BF16, 0, 1)
+        self.compute = o[4]
+
+    def forward_rows(self, toks, offset, rows):
+        """fp32 logits [len(rows), vocab] of chosen tokens of the call (none: the caches are extended, nothing returned)."""
+        t, r = np.ascontiguousarray(toks, np.uint32), np.ascontiguousarray(rows, np.uint32)
+        out = np.empty((r.size, self.cfg.vocab), np.float32)
+        _ck(self.L.vkl_model_forward_rows(self.h, _ptr(t), t.size, offset, _ptr(r), r.size, _ptr(out)))
+        return out
+
+    def trace_layers(self, toks, offset=0):
+        """fp32 residual stream [layer runs, tokens, width] after every layer run (decoder designs)."""
+        t = np.ascontiguousarray(toks, np.uint32)
+        out = np.empty((self.cfg.layers, t.size, self.cfg.dim), np.float32)
+        _ck(self.L.vkl_model_trace_layers(self.h, _ptr(t), t.size, offset, _ptr(out)))
+        return out
+
     def topk(self, k):
         """The k largest logits of the last step and their ids, selected on the device."""
         vals, ids = np.empty(k, np.float32), np.empty(k, np.uint32)
         _ck(self.L.vkl_model_topk(self.h, k, _ptr(vals), _ptr(ids)))
         return vals, ids
+
+    def cache_bytes(self):
+        """Device bytes of all key (and value) caches."""
+        n = 0
+        for layer in range(self.cfg.layers):
+            a, b, c = self.kv_shape(layer)
+            n += a * b * c * (4 if self._kv_dtype == FP32 else 2) * (1 if self.cfg.weight_dtype == BF16 else 2)
+        return n
 
     def set_weight(self, name, dtype, data):
         a = np.ascontiguousarray(data)
@@ -662,13 +727,17 @@ class Model:
         _ck(self.L.vkl_model_last_token(self.h, C.byref(t)))
         return t.value
 
-    def kv_shape(self):
-        c = self.cfg
-        return (c.heads // max(1, c.tp_size), c.maxlen, c.dim // c.heads)
+    def kv_shape(self, layer=0):
+        o = (u32 * 4)()
+        _ck(self.L.vkl_model_kv_shape(self.h, layer, o))
+        self._kv_dtype = o[3]
+        return (o[0], o[1], o[2])
 
     def read_kv(self, layer):
-        k = np.empty(self.kv_shape(), np.uint16)
-        v = np.empty(self.kv_shape(), np.uint16)
+        """(keys, values) as raw bits. A decoder design whose keys are its values has one cache: values are zeros."""
+        shape = self.kv_shape(layer)
+        k = np.empty(shape, np.uint32 if self._kv_dtype == FP32 else np.uint16)
+        v = np.zeros_like(k)
         _ck(self.L.vkl_model_read_kv(self.h, layer, _ptr(k), _ptr(v)))
         return k, v
 
@@ -746,6 +815,19 @@ class Model:
             self.close()
         except Exception:
             pass
+
+
+def load_model(dev, path, maxlen=0, compute=BF16):
+    """A model by what `path` is: a GGUF file (Llama-2) or a checkpoint folder of a registered design."""
+    if os.path.isdir(path):
+        return Model.from_folder(dev, path, maxlen or 4096, compute)
+    if compute == FP32:
+        raise VklError(12, "load_model: Llama-2 models do not run in 32-bit")
+    g = Gguf(path)
+    try:
+        return Model.from_gguf(dev, g, maxlen)
+    finally:
+        g.close()
 
 
 # ---- checkpoint container and samplers ---------------------------------------------------

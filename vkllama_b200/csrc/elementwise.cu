@@ -6,6 +6,7 @@
 
 #include "common.cuh"
 #include "kernels.h"
+#include "rows.h"
 #include "runtime.h"
 
 namespace vkl {
@@ -133,6 +134,10 @@ __global__ void synth_f16_kernel(__half *dst, uint64_t key, uint64_t first, uint
   for (uint64_t i = (uint64_t)blockIdx.x * blockDim.x + threadIdx.x; i < n;
        i += (uint64_t)gridDim.x * blockDim.x)
     dst[i] = __float2half_rn(__fmaf_rn(synth_z(key, first + i), stdv, mean));
+}
+__global__ void synth_bf16_kernel(bf16 *dst, uint64_t key, uint64_t n, float mean, float stdv) {
+  for (uint64_t i = (uint64_t)blockIdx.x * blockDim.x + threadIdx.x; i < n; i += (uint64_t)gridDim.x * blockDim.x)
+    dst[i] = __float2bfloat16_rn(__fmaf_rn(synth_z(key, i), stdv, mean));
 }
 __global__ void synth_q8_kernel(uint8_t *dst, uint64_t key, uint32_t N, uint32_t K, float mean,
                                 float stdv, uint32_t row0, uint32_t col0, uint32_t ld_full) {
@@ -275,10 +280,13 @@ __device__ __forceinline__ bool better(float v, uint32_t i, float bv, uint32_t b
   if (op == 0) return v > bv || (v == bv && i < bi);
   return v < bv || (v == bv && i < bi);
 }
-__global__ void __launch_bounds__(256) argop0_kernel(const __half *__restrict__ x, Pair *part,
+__device__ __forceinline__ float arg_value(__half v) { return __half2float(v); }
+__device__ __forceinline__ float arg_value(float v) { return v; }
+template <class E>
+__global__ void __launch_bounds__(256) argop0_kernel(const E *__restrict__ x, Pair *part,
                                                      uint32_t W, uint32_t chunks, int op) {
   const uint32_t row = blockIdx.y, chunk = blockIdx.x;
-  const __half *xr = x + (size_t)row * W;
+  const E *xr = x + (size_t)row * W;
   const uint32_t base = chunk * 1024;
   float bv = op == 0 ? -INFINITY : INFINITY;
   uint32_t bi = 0xffffffffu;
@@ -286,7 +294,7 @@ __global__ void __launch_bounds__(256) argop0_kernel(const __half *__restrict__ 
   for (int j = 0; j < 4; ++j) {
     const uint32_t i = base + j * 256 + threadIdx.x;
     if (i < W) {
-      const float v = __half2float(xr[i]);
+      const float v = arg_value(xr[i]);
       if (bi == 0xffffffffu || better(v, i, bv, bi, op)) {
         bv = v;
         bi = i;
@@ -478,6 +486,11 @@ cudaError_t launch_synth_f16(__half *dst, uint64_t seed, uint64_t tensor, uint64
   synth_f16_kernel<<<std::min(nblk(n, 256), 148u * 32), 256, 0, s>>>(dst, synth_key(seed, tensor), first, n, mean, stdv);
   return cudaGetLastError();
 }
+cudaError_t launch_synth_bf16(bf16 *dst, uint64_t seed, uint64_t tensor, uint64_t n, float mean, float stdv, cudaStream_t s) {
+  if (!n) return cudaSuccess;
+  synth_bf16_kernel<<<std::min(nblk(n, 256), 148u * 32), 256, 0, s>>>(dst, synth_key(seed, tensor), n, mean, stdv);
+  return cudaGetLastError();
+}
 cudaError_t launch_synth_q8(uint8_t *dst, uint64_t seed, uint64_t tensor, uint32_t N, uint32_t K,
                             float mean, float stdv, uint32_t row0, uint32_t col0, uint32_t ld_full,
                             cudaStream_t s) {
@@ -530,13 +543,20 @@ cudaError_t launch_embedding(const uint8_t *vocab, int is_q8, const uint32_t *id
   return cudaGetLastError();
 }
 size_t argop_partials_bytes(uint32_t rows, uint32_t W) { return (size_t)rows * ((W + 1023) / 1024) * sizeof(Pair); }
-cudaError_t launch_argop(const __half *x, uint32_t *out, void *partials, uint32_t rows,
-                         uint32_t W, int op, cudaStream_t s) {
+template <class E>
+static cudaError_t launch_argop_t(const E *x, uint32_t *out, void *partials, uint32_t rows, uint32_t W, int op, cudaStream_t s) {
   if (!rows || !W) return cudaSuccess;
   const uint32_t chunks = (W + 1023) / 1024;
   argop0_kernel<<<dim3(chunks, rows), 256, 0, s>>>(x, (Pair *)partials, W, chunks, op);
   argop1_kernel<<<nblk(rows, 128), 128, 0, s>>>((const Pair *)partials, out, rows, chunks, op);
   return cudaGetLastError();
+}
+cudaError_t launch_argop(const __half *x, uint32_t *out, void *partials, uint32_t rows,
+                         uint32_t W, int op, cudaStream_t s) {
+  return launch_argop_t(x, out, partials, rows, W, op, s);
+}
+cudaError_t launch_argmax_f32(const float *x, uint32_t *out, void *partials, uint32_t rows, uint32_t W, cudaStream_t s) {
+  return launch_argop_t(x, out, partials, rows, W, 0, s);
 }
 cudaError_t launch_softmax(const __half *in, __half *out, uint32_t C, uint32_t H, uint32_t W,
                            int seq_mask, uint32_t offset, cudaStream_t s) {

@@ -1,5 +1,6 @@
 // Dense GEMM for multi-token (prefill) passes on the 5th-generation tensor cores:
-// C[M,N] = A[M,K] . W[N,K]^T with fp32 accumulation in tensor memory (TMEM), W in FP16 or Q8_0.
+// C[M,N] = A[M,K] . W[N,K]^T with fp32 accumulation in tensor memory (TMEM), A and W in FP16, W in Q8_0, or
+// both in bfloat16 with the epilogues of the layer-list decoders (rows.cuh) and tiles grouped by expert.
 //
 // Replaces, for many rows, the reference's matmul_b0_tb_fp16_v2.comp and matmul_b0_fp16_x_q8_0.comp
 // (src/ops/mat_mul.cpp:71-103), which re-read the whole weight matrix for every input row.
@@ -29,6 +30,7 @@
 
 #include "common.cuh"
 #include "kernels.h"
+#include "rows.cuh"
 
 #ifndef VKL_GEMM_TRACE
 #define VKL_GEMM_TRACE 0  // diagnostic build: CTA (0,0) stamps the global timer at fixed points of every K step
@@ -149,9 +151,9 @@ __device__ __forceinline__ uint64_t smem_desc(uint32_t addr) {
   return d;
 }
 
-// kind::f16 instruction descriptor: fp16 x fp16 -> fp32, both operands K-major, M x N tile.
-__host__ __device__ constexpr uint32_t instr_desc(uint32_t m, uint32_t n) {
-  return (1u << 4) | ((n >> 3) << 17) | ((m >> 4) << 24);
+// kind::f16 instruction descriptor: fp16 x fp16 or bf16 x bf16 -> fp32, both operands K-major, M x N tile.
+__host__ __device__ constexpr uint32_t instr_desc(uint32_t m, uint32_t n, bool bf) {
+  return (1u << 4) | (bf ? (1u << 7) | (1u << 10) : 0u) | ((n >> 3) << 17) | ((m >> 4) << 24);
 }
 
 __device__ __forceinline__ void tma_load_2d(uint32_t dst, const CUtensorMap *map, uint32_t x, uint32_t y, uint32_t bar) {
@@ -197,9 +199,15 @@ __device__ __forceinline__ void dequant_unit_at(unsigned char *wtile, uint32_t o
   *reinterpret_cast<uint4 *>(wtile + off_b) = make_uint4(b[0], b[1], b[2], b[3]);
 }
 
-template <int BN, bool Q8>
-__global__ void __launch_bounds__(Q8 ? GEMM_THREADS_Q8 : GEMM_THREADS, 1)
-    gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant__ CUtensorMap map_w, const GemmParams p) {
+// The kernel's operands: FP16 weights, Q8_0 weights, or bfloat16 with GemmRows' epilogues.
+enum GemmKind { GK_F16, GK_Q8, GK_ROWS };
+template <int KIND> struct GemmArgs { using Type = GemmParams; };
+template <> struct GemmArgs<GK_ROWS> { using Type = GemmRows; };
+
+template <int BN, int KIND>
+__global__ void __launch_bounds__(KIND == GK_Q8 ? GEMM_THREADS_Q8 : GEMM_THREADS, 1)
+    gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant__ CUtensorMap map_w, const typename GemmArgs<KIND>::Type p) {
+  constexpr bool Q8 = KIND == GK_Q8;
   using C = Cfg<BN, Q8>;
   extern __shared__ unsigned char smem_raw[];
   // swizzle atoms are 1024 bytes: align the stage ring
@@ -216,6 +224,14 @@ __global__ void __launch_bounds__(Q8 ? GEMM_THREADS_Q8 : GEMM_THREADS, 1)
   const uint32_t warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const uint32_t m0 = blockIdx.x * BM, n0 = blockIdx.y * BN;
   const uint32_t nkb = p.K / BK;
+  uint32_t w_row = n0;  // first weight row of the tile
+  if constexpr (KIND == GK_ROWS) {
+    if (p.tile_expert) {
+      const int32_t e = p.tile_expert[blockIdx.x];
+      if (e < 0) return;  // uniform over the CTA
+      w_row += (uint32_t)e * p.N;
+    }
+  }
   if (threadIdx.x == 0) {
     for (int s = 0; s < C::STAGES; ++s) {
       asm volatile("mbarrier.init.shared::cta.b64 [%0], %1;" ::"r"(sa(&full[s])), "r"(Q8 ? 1u + NDWG : 1u) : "memory");  // the TMA lane (+ one lane per dequantising warp)
@@ -258,10 +274,11 @@ __global__ void __launch_bounds__(Q8 ? GEMM_THREADS_Q8 : GEMM_THREADS, 1)
         asm volatile("mbarrier.arrive.expect_tx.shared::cta.b64 _, [%0], %1;" ::"r"(bar), "r"(Q8 ? A_TILE_BYTES : C::STAGE_BYTES) : "memory");
         unsigned char *st = stages + (size_t)s * C::STAGE_BYTES;
         tma_load_2d(sa(st), &map_a, kb * BK, m0, bar);
-        if (!Q8) tma_load_2d(sa(st + A_TILE_BYTES), &map_w, kb * BK, n0, bar);
+        if (!Q8) tma_load_2d(sa(st + A_TILE_BYTES), &map_w, kb * BK, w_row, bar);
       }
     }
   } else if (Q8 && warp >= 6 && (warp & 3u) != 1u && !VKL_GEMM_MMAONLY) {
+    if constexpr (Q8) {
     // ------------------------------------------- W tile: Q8_0 -> fp16 in shared memory
     // BN rows x 64 columns = (BN / 16) row tiles x 2 blocks: units of 512 bytes of codes, dealt round robin to
     // the dequantising warps. The scales of a row tile and 4-block group are 8 x 16 bytes: row g's four blocks, then row g + 8's.
@@ -367,10 +384,11 @@ __global__ void __launch_bounds__(Q8 ? GEMM_THREADS_Q8 : GEMM_THREADS, 1)
       if (stop) break;
     }
     asm volatile("cp.async.wait_all;" ::: "memory");  // nothing of this warp may still be landing when the CTA exits
+    }
   } else if (warp == 1) {
     // --------------------------------------------------------------------- MMA
     if (lane == 0) {
-      constexpr uint32_t idesc = instr_desc(BM, BN);
+      constexpr uint32_t idesc = instr_desc(BM, BN, KIND == GK_ROWS);
       for (uint32_t kb = 0; kb < nkb; ++kb) {
         const uint32_t s = kb % C::STAGES, use = kb / C::STAGES;
         if (!VKL_GEMM_MMAONLY && !(VKL_GEMM_TESTWAIT ? mbar_spin_bounded(sa(&full[s]), use & 1u) : mbar_wait_bounded(sa(&full[s]), use & 1u))) {
@@ -427,7 +445,14 @@ __global__ void __launch_bounds__(Q8 ? GEMM_THREADS_Q8 : GEMM_THREADS, 1)
 #pragma unroll
           for (int j = 0; j < 32; ++j) r[j] = __float_as_uint(__uint_as_float(r[j]) + __uint_as_float(r2[j]));
         }
-        if (row < p.M) {
+        if constexpr (KIND == GK_ROWS) {
+          if (row < p.M) {
+            float v[32];
+#pragma unroll
+            for (int j = 0; j < 32; ++j) v[j] = __uint_as_float(r[j]);
+            rows_chunk<bf16>(p.out, row, n0 + cc, v);
+          }
+        } else if (row < p.M) {
           const size_t o = (size_t)row * p.N + n0 + cc;
 #pragma unroll
           for (int j = 0; j < 32; j += 8) {
@@ -493,31 +518,32 @@ EncodeTiled encode_tiled() {
   return fn;
 }
 
-// Tensor map over a row-major fp16 matrix [rows, K]: boxes of 64 columns x box_rows rows,
+// Tensor map over a row-major fp16 or bf16 matrix [rows, K]: boxes of 64 columns x box_rows rows,
 // 128-byte swizzle, rows beyond the matrix read as zero.
-bool make_map(CUtensorMap *map, const __half *base, uint32_t rows, uint32_t K, uint32_t box_rows) {
+bool make_map(CUtensorMap *map, const void *base, uint32_t rows, uint32_t K, uint32_t box_rows, bool bf = false) {
   EncodeTiled enc = encode_tiled();
   if (!enc) return false;
   const cuuint64_t dims[2] = {K, rows};
   const cuuint64_t strides[1] = {(cuuint64_t)K * 2};
   const cuuint32_t box[2] = {BK, box_rows};
   const cuuint32_t estr[2] = {1, 1};
-  return enc(map, CU_TENSOR_MAP_DATA_TYPE_FLOAT16, 2, const_cast<__half *>(base), dims, strides, box, estr, CU_TENSOR_MAP_INTERLEAVE_NONE,
+  return enc(map, bf ? CU_TENSOR_MAP_DATA_TYPE_BFLOAT16 : CU_TENSOR_MAP_DATA_TYPE_FLOAT16, 2, const_cast<void *>(base), dims, strides, box, estr, CU_TENSOR_MAP_INTERLEAVE_NONE,
              CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_256B, CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE) == CUDA_SUCCESS;
 }
 
-template <int BN, bool Q8> cudaError_t launch_bn(const GemmParams &p, cudaStream_t s) {
+template <int BN, int KIND> cudaError_t launch_bn(const typename GemmArgs<KIND>::Type &p, cudaStream_t s, uint32_t w_rows) {
+  constexpr bool Q8 = KIND == GK_Q8;
   CUtensorMap ma, mw;
-  if (!make_map(&ma, p.a, p.M, p.K, BM)) return cudaErrorInvalidValue;
-  if (Q8) {
+  if (!make_map(&ma, p.a, p.M, p.K, BM, KIND == GK_ROWS)) return cudaErrorInvalidValue;
+  if constexpr (Q8) {
     mw = ma;  // unused: the W tile is written by the dequantising warps
-  } else if (!make_map(&mw, p.w, p.N, p.K, BN)) {
+  } else if (!make_map(&mw, p.w, w_rows, p.K, BN, KIND == GK_ROWS)) {
     return cudaErrorInvalidValue;
   }
-  cudaError_t e = cudaFuncSetAttribute(gemm_tcgen05_kernel<BN, Q8>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)Cfg<BN, Q8>::SMEM);
+  cudaError_t e = cudaFuncSetAttribute(gemm_tcgen05_kernel<BN, KIND>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)Cfg<BN, Q8>::SMEM);
   if (e != cudaSuccess) return e;
   // x = row tile, so that the CTAs sharing one tile of W run together and W crosses HBM once
-  gemm_tcgen05_kernel<BN, Q8><<<dim3((p.M + BM - 1) / BM, (p.N + BN - 1) / BN), Q8 ? GEMM_THREADS_Q8 : GEMM_THREADS, Cfg<BN, Q8>::SMEM, s>>>(ma, mw, p);
+  gemm_tcgen05_kernel<BN, KIND><<<dim3((p.M + BM - 1) / BM, (p.N + BN - 1) / BN), Q8 ? GEMM_THREADS_Q8 : GEMM_THREADS, Cfg<BN, Q8>::SMEM, s>>>(ma, mw, p);
   return cudaGetLastError();
 }
 
@@ -540,14 +566,14 @@ static int forced_bn() {
   static const int forced = [] { const char *e = getenv("VKLLAMA_GEMM_BN"); return e ? atoi(e) : 0; }();  // experiments
   return forced == 256 || forced == 128 || forced == 64 || forced == 32 ? forced : 0;
 }
-static int pick_bn(const GemmParams &p, bool q8) {
+static int pick_bn(uint32_t M, uint32_t N, bool q8) {
   if (int f = forced_bn()) return (q8 || f >= 128) ? f : 128;
-  const size_t mt = (p.M + BM - 1) / BM, sms = sm_count();
+  const size_t mt = (M + BM - 1) / BM, sms = sm_count();
   int best = 0;
   double best_cost = 0.0;
   for (int bn : {256, 128, 64, 32}) {
     if (!q8 && bn < 128) break;
-    const size_t ctas = mt * ((p.N + bn - 1) / bn), waves = (ctas + sms - 1) / sms;
+    const size_t ctas = mt * ((N + bn - 1) / bn), waves = (ctas + sms - 1) / sms;
     // measured time of one wave at K = 4096, us: Q8_0 30.9 / 31.2 / 43.0 / 73.4 for 32 / 64 / 128 / 256 columns, FP16 27 + 0.022 bn
     const double wave = q8 ? (bn == 32 ? 30.9 : bn == 64 ? 31.2 : bn == 128 ? 43.0 : 73.4) : 27.0 + 0.022 * bn;
     const double cost = (double)waves * wave;
@@ -562,18 +588,26 @@ static int pick_bn(const GemmParams &p, bool q8) {
 cudaError_t launch_gemm_f16_tcgen05(const GemmParams &p, cudaStream_t s) {
   if (!gemm_tcgen05_supported(p.M, p.N, p.K)) return cudaErrorInvalidValue;
   if ((reinterpret_cast<uintptr_t>(p.a) | reinterpret_cast<uintptr_t>(p.w)) & 15) return cudaErrorMisalignedAddress;
-  return pick_bn(p, false) == 256 ? launch_bn<256, false>(p, s) : launch_bn<128, false>(p, s);
+  return pick_bn(p.M, p.N, false) == 256 ? launch_bn<256, GK_F16>(p, s, p.N) : launch_bn<128, GK_F16>(p, s, p.N);
 }
 
 cudaError_t launch_gemm_q8_tcgen05(const GemmParams &p, cudaStream_t s) {
   if (!gemm_tcgen05_supported(p.M, p.N, p.K) || !p.w_codes || !p.w_scales) return cudaErrorInvalidValue;
   if (reinterpret_cast<uintptr_t>(p.a) & 15) return cudaErrorMisalignedAddress;
-  switch (pick_bn(p, true)) {
-    case 256: return launch_bn<256, true>(p, s);
-    case 128: return launch_bn<128, true>(p, s);
-    case 64: return launch_bn<64, true>(p, s);
-    default: return launch_bn<32, true>(p, s);
+  switch (pick_bn(p.M, p.N, true)) {
+    case 256: return launch_bn<256, GK_Q8>(p, s, p.N);
+    case 128: return launch_bn<128, GK_Q8>(p, s, p.N);
+    case 64: return launch_bn<64, GK_Q8>(p, s, p.N);
+    default: return launch_bn<32, GK_Q8>(p, s, p.N);
   }
+}
+
+cudaError_t launch_gemm_rows_bf16(const GemmRows &p, cudaStream_t s) {
+  if (!gemm_tcgen05_supported(p.M, p.N, p.K) || p.N % 32 || (p.tile_expert && p.M % BM)) return cudaErrorInvalidValue;
+  if ((reinterpret_cast<uintptr_t>(p.a) | reinterpret_cast<uintptr_t>(p.w)) & 15) return cudaErrorMisalignedAddress;
+  // grouped: a tile's weight rows beyond its expert's N are read (the next expert's, or zeros) and dropped by the epilogue
+  const uint32_t w_rows = p.tile_expert ? p.w_rows : p.N;
+  return pick_bn(p.M, p.N, false) == 256 ? launch_bn<256, GK_ROWS>(p, s, w_rows) : launch_bn<128, GK_ROWS>(p, s, w_rows);
 }
 
 cudaError_t launch_swiglu_f32(const float *gate, const float *up, __half *out, size_t n, cudaStream_t s) {

@@ -88,6 +88,7 @@ cudaError_t launch_embedding(const uint8_t *vocab, int vocab_is_q8, const uint32
 // Two-stage arg-max/min over rows of width W; partials needs rows*ceil(W/1024)*8 bytes.
 cudaError_t launch_argop(const __half *x, uint32_t *out, void *partials, uint32_t rows,
                          uint32_t W, int op_type, cudaStream_t s);
+cudaError_t launch_argmax_f32(const float *x, uint32_t *out, void *partials, uint32_t rows, uint32_t W, cudaStream_t s);
 size_t argop_partials_bytes(uint32_t rows, uint32_t W);
 // The k largest of n fp32 values and their indices, descending (equal values: lowest index first).
 cudaError_t launch_topk_f32(const float *x, uint32_t n, uint32_t k, float *vals, uint32_t *ids, cudaStream_t s);

@@ -19,7 +19,8 @@
 
 #include <string>
 
-#include "runtime.h"
+#include "decoder.h"
+#include "model.h"
 
 namespace vkl {
 int rope_tables(vkl_device *dev, cudaStream_t s, int dim, int rows, vkl_tensor **fc, vkl_tensor **fs);
@@ -27,13 +28,6 @@ int rope_tables(vkl_device *dev, cudaStream_t s, int dim, int rows, vkl_tensor *
 using namespace vkl;
 
 namespace {
-struct Layer {
-  vkl_tensor *attn_norm = nullptr, *ffn_norm = nullptr;
-  vkl_tensor *wq = nullptr, *wk = nullptr, *wv = nullptr, *wo = nullptr;
-  vkl_tensor *gate = nullptr, *up = nullptr, *down = nullptr;
-  vkl_tensor *kcache = nullptr, *vcache = nullptr;
-};
-
 __global__ void set_u32(uint32_t *p, uint32_t v) { *p = v; }
 // After the arg-max: publish the picked id, feed it back, advance the position.
 __global__ void advance_kernel(const uint32_t *next, uint32_t *tok, uint32_t *pos, uint32_t *step,
@@ -46,83 +40,14 @@ __global__ void advance_kernel(const uint32_t *next, uint32_t *tok, uint32_t *po
 }
 }  // namespace
 
-struct vkl_model {
-  vkl_device *dev = nullptr;
-  vkl_model_config cfg;
-  cudaStream_t stream = nullptr;
-  uint32_t head_dim = 0, heads_l = 0, dim_l = 0, ffn_l = 0, vocab_l = 0;
-  std::vector<Layer> L;
-  vkl_tensor *tok_embd = nullptr, *output_norm = nullptr, *output = nullptr;
-  vkl_tensor *fc = nullptr, *fs = nullptr;
-  // activations, sized for `cap_T` rows
-  uint32_t cap_T = 0;
-  vkl_tensor *x = nullptr, *xn = nullptr, *q = nullptr, *k = nullptr, *v = nullptr, *ao = nullptr, *t = nullptr;
-  vkl_tensor *gu32 = nullptr;  // [2, cap_T, ffn] fp32 gate and up results of the FP16 prefill GEMMs
-  bool gemm_used = false;      // a tensor-core GEMM ran since the last check of state[6]
-  vkl_tensor *logits16 = nullptr, *logits32 = nullptr;
-  vkl_tensor *toks = nullptr;  // [cap_T] device token ids; toks[0] is the decode token
-  vkl_tensor *state = nullptr; // uint32[8]: [0] pos, [1] step, [2] next id, [3] all-reduces, [4] arg exchanges, [5] forced tokens, [6] GEMM wait error
-  vkl_tensor *forced = nullptr;  // prompt ids for token-by-token prefill
-  // tensor parallelism: this rank's exchange buffer (plain cudaMalloc so that it can be
-  // exported over CUDA IPC) and every rank's mapping of it
-  void *tp_buf = nullptr;
-  size_t tp_bytes = 0;
-  uint32_t tp_flag_off = 0;
-  void *tp_peer[8] = {};
-  bool tp_connected = false;
-  // many-token passes of a sharded model: two alternating regions of fp32 partial sums [tp_pf_rows, dim]
-  // and the ranks' flag words behind the one-token exchange area, and the count of all-reduces so far
-  size_t tp_pf_off = 0, tp_pf_flag_off = 0;
-  uint32_t tp_pf_rows = 0, tp_pf_seq = 0;
-  vkl_tensor *out_ids = nullptr;
-  vkl_tensor *argpart = nullptr, *attn_scratch = nullptr, *attn_counters = nullptr;
-  uint32_t splits = 8, out_cap = 0;
-  cudaGraphExec_t decode_graph = nullptr;
-  bool use_pdl = true;
-  // persistent single-kernel decode step (decode_mega.cu)
-  bool mega_ready = false, mega_tried = false;
-  int mega_grid = 0;
-  vkl_tensor *mega_ops = nullptr, *mega_sync = nullptr, *mega_arg = nullptr, *mega_attn = nullptr, *mega_stages = nullptr, *mega_counts = nullptr, *mega_ll = nullptr;
-  std::vector<vkl_tensor *> mega_packed;  // the ops' weight streams in the persistent kernel's layout
-  MegaParams mp;
-  uint32_t mega_launches_per_token = 1;
-  uint32_t sm_mhz = 0;  // measured SM clock, for the profiled launches' cycle counts
-  uint32_t wait_limit = 0;  // polls a wait of the decode kernel may spin (0: the default of build_mega)
-  bool tp_failed = false;   // a wait on another rank ran out: the ranks' sequence counters are out of step until they reconnect
-  unsigned char *pin = nullptr;  // pinned host staging of the one-token call: this rank's fp32 logits, then the decode kernel's error word
-  cudaEvent_t ev0 = nullptr, ev1 = nullptr, ev2 = nullptr;
-  uint32_t *pos_dev() { return (uint32_t *)state->data(); }
-  uint32_t *step_dev() { return (uint32_t *)state->data() + 1; }
-  uint32_t *next_dev() { return (uint32_t *)state->data() + 2; }
-  ~vkl_model() {
-    if (decode_graph) cudaGraphExecDestroy(decode_graph);
-    if (tp_buf) cudaFree(tp_buf);
-    if (pin) cudaFreeHost(pin);
-    for (auto &l : L)
-      for (vkl_tensor *p : {l.attn_norm, l.ffn_norm, l.wq, l.wk, l.wv, l.wo, l.gate, l.up, l.down, l.kcache, l.vcache}) vkl_tensor_release(p);
-    for (vkl_tensor *p : mega_packed) vkl_tensor_release(p);
-    for (vkl_tensor *p : {tok_embd, output_norm, output, fc, fs, x, xn, q, k, v, ao, t, gu32, logits16, logits32, toks, state, out_ids, forced, argpart, attn_scratch, attn_counters, mega_ops, mega_sync, mega_arg, mega_attn, mega_stages, mega_counts, mega_ll})
-      vkl_tensor_release(p);
-    if (ev0) cudaEventDestroy(ev0);
-    if (ev1) cudaEventDestroy(ev1);
-    if (ev2) cudaEventDestroy(ev2);
-    if (stream) {
-      dev->remove_stream(stream);
-      cudaStreamDestroy(stream);
-    }
-  }
-};
-
 namespace {
 
 bool q8(const vkl_model *m) { return m->cfg.weight_dtype == VKL_Q8_0; }
 
 int ensure_rows(vkl_model *m, uint32_t T) {
   if (T <= m->cap_T) return VKL_OK;
-  if (m->decode_graph) {  // the graph holds the old buffers
-    cudaGraphExecDestroy(m->decode_graph);
-    m->decode_graph = nullptr;
-  }
+  if (m->dec) return decoder_ensure_rows(m, T);
+  model_drop_graph(m);  // the graph holds the old buffers
   VKL_CUDA(cudaStreamSynchronize(m->stream));
   if (m->mega_tried) {  // the op table of the persistent kernel holds the old buffers too
     for (vkl_tensor **t : {&m->mega_ops, &m->mega_sync, &m->mega_arg, &m->mega_attn, &m->mega_stages, &m->mega_counts, &m->mega_ll}) {
@@ -191,21 +116,6 @@ bool use_gemm(const vkl_model *m, uint32_t rows) {
          gemm_tcgen05_supported(rows, m->cfg.dim, m->ffn_l);
 }
 
-// Optional per-kernel timing of a pass: an event after every launch, tagged with
-// the kernel's class (0 embedding, 1 norm+QKV, 2 attention, 3 o_proj, 4 gate/up,
-// 5 down, 6 lm head, 7 arg-max).
-struct Marker {
-  std::vector<cudaEvent_t> ev;
-  std::vector<int> cls;
-  cudaStream_t s;
-  void mark(int c) {
-    cudaEvent_t e;
-    cudaEventCreate(&e);
-    cudaEventRecord(e, s);
-    ev.push_back(e);
-    cls.push_back(c);
-  }
-};
 #define MARK(c) do { if (mk) mk->mark(c); } while (0)
 
 // One pass over T tokens already in m->toks, first position in state[0].
@@ -214,6 +124,7 @@ struct Marker {
 // last block's attention and clips nothing); the one form tensor-parallel models run with T > 1, their
 // K-split projections summed over the ranks by launch_tp_reduce_rows. `tok_off`: first token in m->toks.
 int run_tokens(vkl_model *m, uint32_t T, bool pdl, Marker *mk = nullptr, bool fill_only = false, uint32_t tok_off = 0) {
+  if (m->dec) return decoder_run(m, T, pdl, mk);
   cudaStream_t s = m->stream;
   MARK(-1);
   const uint32_t D = m->cfg.dim, nl = m->cfg.layers;
@@ -739,7 +650,7 @@ int decode_step(vkl_model *m) {
     return VKL_OK;
   }
   VKL_CUDA(cudaGraphLaunch(m->decode_graph, m->stream));
-  count_launches(5 * m->cfg.layers + 5);
+  count_launches(m->dec ? m->dec->launches_per_token + 1 : 5 * m->cfg.layers + 5);
   return VKL_OK;
 }
 
@@ -774,6 +685,7 @@ int build_decode_graph(vkl_model *m) {
 
 int check_ready(vkl_model *m) {
   if (!m) return fail(VKL_INVALID_ARGUMENT, "model: null handle");
+  if (m->dec) return decoder_ready(m);
   if (!m->tok_embd || !m->output || !m->output_norm) return fail(VKL_FAILED_PRECONDITION, "model: token_embd/output/output_norm weights are not set");
   for (uint32_t l = 0; l < m->cfg.layers; ++l) {
     Layer &y = m->L[l];
@@ -821,9 +733,45 @@ int find_slot(vkl_model *m, const char *name, Slot *s) {
   return fail(VKL_INVALID_ARGUMENT, "model: tensor name '%s' is not part of a Llama-2 model with %u blocks", name, c.layers);
 }
 
+// Positions a sequence may reach: the Llama-2 caches are rings and end with the RoPE table, a decoder design's
+// attention looks at every position.
+size_t max_positions(const vkl_model *m) { return m->dec ? (size_t)m->cfg.maxlen : (size_t)2 * m->cfg.maxlen; }
+
+int check_ids(const vkl_model *m, const uint32_t *toks, size_t n) {
+  if (!m->dec) return VKL_OK;  // the Llama-2 embedding maps unknown ids to its UNK row
+  for (size_t i = 0; i < n; ++i)
+    if (toks[i] >= m->cfg.vocab) return fail(VKL_OUT_OF_RANGE, "model: token id %u of a vocabulary of %u", toks[i], m->cfg.vocab);
+  return VKL_OK;
+}
+
 const char *kLayerNames[9] = {"attn_norm", "attn_q", "attn_k", "attn_v", "attn_output", "ffn_norm", "ffn_gate", "ffn_up", "ffn_down"};
 
 }  // namespace
+
+namespace vkl {
+void model_drop_graph(vkl_model *m) {
+  if (!m->decode_graph) return;
+  cudaStreamSynchronize(m->stream);
+  cudaGraphExecDestroy(m->decode_graph);
+  m->decode_graph = nullptr;
+}
+
+int model_init_common(vkl_model *m) {
+  cudaError_t e = cudaStreamCreateWithFlags(&m->stream, cudaStreamNonBlocking);
+  if (e != cudaSuccess) return fail(VKL_INTERNAL, "cudaStreamCreate: %s", cudaGetErrorString(e));
+  m->dev->add_stream(m->stream);
+  cudaEventCreate(&m->ev0);
+  cudaEventCreate(&m->ev1);
+  cudaEventCreate(&m->ev2);
+  m->out_cap = 2 * m->cfg.maxlen + 16;
+  VKL_OKAY(tensor_new(m->dev, 1, 1, (m->vocab_l + 31) / 32 * 32, VKL_FP32, &m->logits32));
+  VKL_OKAY(tensor_new(m->dev, 1, 1, 8, VKL_UINT32, &m->state));
+  VKL_OKAY(tensor_new(m->dev, 1, 1, m->out_cap, VKL_UINT32, &m->out_ids));
+  VKL_OKAY(tensor_new(m->dev, 1, 1, argop_partials_bytes(1, m->vocab_l) / 4 + 2, VKL_FP32, &m->argpart));
+  VKL_CUDA(cudaMemsetAsync(m->state->data(), 0, 32, m->stream));
+  return VKL_OK;
+}
+}  // namespace vkl
 
 extern "C" {
 
@@ -857,12 +805,8 @@ int vkl_model_create(vkl_device *dev, const vkl_model_config *cfg, vkl_model **o
     delete m;
     return st;
   };
-  cudaError_t e = cudaStreamCreateWithFlags(&m->stream, cudaStreamNonBlocking);
-  if (e != cudaSuccess) return bail(fail(VKL_INTERNAL, "cudaStreamCreate: %s", cudaGetErrorString(e)));
-  dev->add_stream(m->stream);
-  cudaEventCreate(&m->ev0);
-  cudaEventCreate(&m->ev1);
-  cudaEventCreate(&m->ev2);
+  int st = model_init_common(m);
+  if (st) return bail(st);
   for (auto &l : m->L) {
     if (int st = tensor_new(dev, m->heads_l, c.maxlen, hd, VKL_FP16, &l.kcache)) return bail(st);
     if (int st = tensor_new(dev, m->heads_l, c.maxlen, hd, VKL_FP16, &l.vcache)) return bail(st);
@@ -872,14 +816,9 @@ int vkl_model_create(vkl_device *dev, const vkl_model_config *cfg, vkl_model **o
   // Positions up to 2*maxlen are valid, the size the reference gives its tables (rope.cpp:73-76).
   if (int st = rope_tables(dev, m->stream, hd, 2 * c.maxlen, &m->fc, &m->fs)) return bail(st);
   m->splits = 8;
-  m->out_cap = 2 * c.maxlen + 16;
-  int st = VKL_OK;
-  if ((st = tensor_new(dev, 1, 1, m->vocab_l, VKL_FP16, &m->logits16)) || (st = tensor_new(dev, 1, 1, m->vocab_l, VKL_FP32, &m->logits32)) ||
-      (st = tensor_new(dev, 1, 1, 8, VKL_UINT32, &m->state)) || (st = tensor_new(dev, 1, 1, c.maxlen, VKL_UINT32, &m->forced)) || (st = tensor_new(dev, 1, 1, m->out_cap, VKL_UINT32, &m->out_ids)) ||
-      (st = tensor_new(dev, 1, 1, argop_partials_bytes(1, m->vocab_l) / 4 + 2, VKL_FP32, &m->argpart)) ||
+  if ((st = tensor_new(dev, 1, 1, m->vocab_l, VKL_FP16, &m->logits16)) || (st = tensor_new(dev, 1, 1, c.maxlen, VKL_UINT32, &m->forced)) ||
       (st = tensor_new(dev, 1, 1, m->heads_l, VKL_UINT32, &m->attn_counters)))
     return bail(st);
-  cudaMemsetAsync(m->state->data(), 0, 32, m->stream);
   if (tp > 1) {
     m->tp_flag_off = 4 * tp * c.dim;  // partial sums: [2 parities][tp][dim] words of {fp32 sum, sequence number}
     m->tp_bytes = ((size_t)m->tp_flag_off + 64) * 4;
@@ -893,7 +832,7 @@ int vkl_model_create(vkl_device *dev, const vkl_model_config *cfg, vkl_model **o
   }
   cudaMemsetAsync(m->attn_counters->data(), 0, m->attn_counters->device_bytes(), m->stream);
   if ((st = ensure_rows(m, 1))) return bail(st);
-  e = cudaStreamSynchronize(m->stream);
+  cudaError_t e = cudaStreamSynchronize(m->stream);
   if (e != cudaSuccess) return bail(fail(VKL_INTERNAL, "model_create: %s", cudaGetErrorString(e)));
   *out = m;
   return VKL_OK;
@@ -923,6 +862,7 @@ static void drop_packed(vkl_model *m) {
 int vkl_model_set_weight(vkl_model *m, const char *name, int dtype, const void *data, size_t bytes) {
   if (!m || !name || !data) return fail(VKL_INVALID_ARGUMENT, "model_set_weight: null argument");
   VKL_CUDA(cudaSetDevice(m->dev->ordinal));
+  if (m->dec) return decoder_set_weight(m, name, dtype, data, bytes);
   drop_packed(m);
   Slot s;
   VKL_OKAY(find_slot(m, name, &s));
@@ -970,6 +910,7 @@ int vkl_model_set_weight(vkl_model *m, const char *name, int dtype, const void *
 int vkl_model_synth_weights(vkl_model *m, uint64_t seed, float wstd, float nstd) {
   if (!m) return fail(VKL_INVALID_ARGUMENT, "model_synth_weights: null model");
   VKL_CUDA(cudaSetDevice(m->dev->ordinal));
+  if (m->dec) return decoder_synth(m, seed, wstd, nstd);
   drop_packed(m);
   std::vector<std::string> names = {"token_embd.weight", "output_norm.weight", "output.weight"};
   for (uint32_t l = 0; l < m->cfg.layers; ++l)
@@ -1012,7 +953,9 @@ int vkl_model_forward(vkl_model *m, const uint32_t *toks, size_t n, size_t offse
   if (!toks || !logits_out) return fail(VKL_INVALID_ARGUMENT, "model_forward: null argument");
   if (n == 0) return fail(VKL_INVALID_ARGUMENT, "model_forward: no tokens");
   if (n > m->cfg.maxlen) return fail(VKL_OUT_OF_RANGE, "model_forward: %zu tokens exceed the context length %u", n, m->cfg.maxlen);
-  if (offset + n > (size_t)2 * m->cfg.maxlen) return fail(VKL_OUT_OF_RANGE, "model_forward: position %zu is beyond the RoPE table (2*maxlen)", offset + n);
+  if (offset + n > max_positions(m))
+    return fail(VKL_OUT_OF_RANGE, "model_forward: position %zu is beyond %s", offset + n, m->dec ? "the context length" : "the RoPE table (2*maxlen)");
+  VKL_OKAY(check_ids(m, toks, n));
   VKL_CUDA(cudaSetDevice(m->dev->ordinal));
   VKL_OKAY(ensure_rows(m, (uint32_t)n));
   if (n == 1 || m->cfg.tp_size > 1) VKL_OKAY(prepare_decode(m));
@@ -1085,14 +1028,83 @@ int vkl_model_forward(vkl_model *m, const uint32_t *toks, size_t n, size_t offse
   return VKL_OK;
 }
 
+int vkl_model_forward_rows(vkl_model *m, const uint32_t *toks, size_t n, size_t offset, const uint32_t *rows, size_t n_rows, float *logits_out) {
+  if (!m || (n_rows && (!rows || !logits_out))) return fail(VKL_INVALID_ARGUMENT, "model_forward_rows: null argument");
+  for (size_t i = 0; i < n_rows; ++i)
+    if (rows[i] >= n) return fail(VKL_OUT_OF_RANGE, "model_forward_rows: row %u of %zu tokens", rows[i], n);
+  const size_t V = m->cfg.vocab;
+  if (!m->dec) {
+    // the Llama-2 pass clips the last block to the last token, as the reference does
+    if (n_rows > 1 || (n_rows == 1 && rows[0] + 1 != n)) return fail(VKL_UNIMPLEMENTED, "model_forward_rows: a Llama-2 pass leaves the last token's logits only");
+  }
+  std::vector<float> last(V);
+  if (!m->dec || n == 1 || n_rows == 0) {
+    VKL_OKAY(vkl_model_forward(m, toks, n, offset, last.data()));
+    for (size_t i = 0; i < n_rows; ++i) memcpy(logits_out + i * V, last.data(), V * 4);
+    return VKL_OK;
+  }
+  Decoder *d = m->dec.get();
+  d->want_rows.assign(rows, rows + n_rows);
+  const int st = vkl_model_forward(m, toks, n, offset, last.data());
+  d->want_rows.clear();
+  VKL_OKAY(st);
+  VKL_CUDA(cudaMemcpy2D(logits_out, V * 4, d->logits_rows->data(), (size_t)d->vocab_p * 4, V * 4, n_rows, cudaMemcpyDeviceToHost));
+  return VKL_OK;
+}
+
+int vkl_model_trace_layers(vkl_model *m, const uint32_t *toks, size_t n, size_t offset, float *out) {
+  VKL_OKAY(check_ready(m));
+  if (!toks || !out || !n) return fail(VKL_INVALID_ARGUMENT, "model_trace_layers: null or empty argument");
+  if (!m->dec) return fail(VKL_UNIMPLEMENTED, "model_trace_layers: for the layer-list decoder designs (vkl_model_block_forward runs a Llama-2 block)");
+  if (offset + n > m->cfg.maxlen) return fail(VKL_OUT_OF_RANGE, "model_trace_layers: position %zu is beyond the context length", offset + n);
+  VKL_OKAY(check_ids(m, toks, n));
+  VKL_CUDA(cudaSetDevice(m->dev->ordinal));
+  Decoder *d = m->dec.get();
+  VKL_OKAY(ensure_rows(m, (uint32_t)n));
+  const size_t R = d->runs.size();
+  VKL_OKAY(ensure_tensor(m->dev, &d->trace, R, n, d->ldw, VKL_FP32));
+  const uint32_t st[2] = {(uint32_t)offset, 0};
+  VKL_CUDA(cudaMemcpyAsync(m->state->data(), st, 8, cudaMemcpyHostToDevice, m->stream));
+  VKL_CUDA(cudaMemcpyAsync(m->toks->data(), toks, n * 4, cudaMemcpyHostToDevice, m->stream));
+  d->tracing = true;
+  const int rc = run_tokens(m, (uint32_t)n, false);
+  d->tracing = false;
+  VKL_OKAY(rc);
+  VKL_CUDA(cudaMemcpy2DAsync(out, (size_t)m->cfg.dim * 4, d->trace->data(), (size_t)d->ldw * 4, (size_t)m->cfg.dim * 4, R * n, cudaMemcpyDeviceToHost, m->stream));
+  VKL_CUDA(cudaStreamSynchronize(m->stream));
+  return check_gemm(m);
+}
+
+int vkl_model_shape(const vkl_model *m, uint32_t out6[6]) {
+  if (!m || !out6) return fail(VKL_INVALID_ARGUMENT, "model_shape: null argument");
+  out6[0] = m->cfg.vocab;
+  out6[1] = m->cfg.dim;
+  out6[2] = m->cfg.layers;
+  out6[3] = m->cfg.maxlen;
+  out6[4] = m->dec ? (m->dec->f32 ? VKL_FP32 : VKL_BF16) : VKL_FP16;
+  out6[5] = m->cfg.heads;
+  return VKL_OK;
+}
+
+int vkl_model_kv_shape(const vkl_model *m, uint32_t layer, uint32_t out4[4]) {
+  if (!m || !out4 || layer >= m->cfg.layers) return fail(VKL_INVALID_ARGUMENT, "model_kv_shape: bad model or layer");
+  const vkl_tensor *k = m->L[layer].kcache;
+  out4[0] = (uint32_t)k->c;
+  out4[1] = (uint32_t)k->h;
+  out4[2] = (uint32_t)k->w;
+  out4[3] = (uint32_t)k->dtype;
+  return VKL_OK;
+}
+
 int vkl_model_generate(vkl_model *m, const uint32_t *prompt, size_t n_prompt, size_t n_gen, uint32_t *out_ids, float *prefill_ms,
                        float *decode_ms) {
   VKL_OKAY(check_ready(m));
   if (!prompt || !out_ids) return fail(VKL_INVALID_ARGUMENT, "model_generate: null argument");
   if (n_prompt == 0 || n_gen == 0) return fail(VKL_INVALID_ARGUMENT, "model_generate: empty prompt or nothing to generate");
   if (n_prompt > m->cfg.maxlen) return fail(VKL_OUT_OF_RANGE, "model_generate: prompt of %zu tokens exceeds the context length %u", n_prompt, m->cfg.maxlen);
-  if (n_prompt + n_gen > (size_t)2 * m->cfg.maxlen || n_gen > m->out_cap)
-    return fail(VKL_OUT_OF_RANGE, "model_generate: %zu + %zu tokens run past the RoPE table (2*maxlen)", n_prompt, n_gen);
+  if (n_prompt + n_gen > max_positions(m) || n_gen > m->out_cap)
+    return fail(VKL_OUT_OF_RANGE, "model_generate: %zu + %zu tokens run past %s", n_prompt, n_gen, m->dec ? "the context length" : "the RoPE table (2*maxlen)");
+  VKL_OKAY(check_ids(m, prompt, n_prompt));
   VKL_CUDA(cudaSetDevice(m->dev->ordinal));
   VKL_OKAY(ensure_rows(m, (uint32_t)n_prompt));
   VKL_OKAY(prepare_decode(m));
@@ -1188,7 +1200,7 @@ int vkl_model_read_kv(vkl_model *m, uint32_t layer, void *kcache, void *vcache) 
   VKL_CUDA(cudaSetDevice(m->dev->ordinal));
   Layer &y = m->L[layer];
   if (kcache) VKL_CUDA(cudaMemcpyAsync(kcache, y.kcache->data(), y.kcache->device_bytes(), cudaMemcpyDeviceToHost, m->stream));
-  if (vcache) VKL_CUDA(cudaMemcpyAsync(vcache, y.vcache->data(), y.vcache->device_bytes(), cudaMemcpyDeviceToHost, m->stream));
+  if (vcache && y.vcache) VKL_CUDA(cudaMemcpyAsync(vcache, y.vcache->data(), y.vcache->device_bytes(), cudaMemcpyDeviceToHost, m->stream));
   VKL_CUDA(cudaStreamSynchronize(m->stream));
   return VKL_OK;
 }
@@ -1197,13 +1209,14 @@ int vkl_model_write_kv(vkl_model *m, uint32_t layer, const void *kcache, const v
   VKL_CUDA(cudaSetDevice(m->dev->ordinal));
   Layer &y = m->L[layer];
   if (kcache) VKL_CUDA(cudaMemcpyAsync(y.kcache->data(), kcache, y.kcache->device_bytes(), cudaMemcpyHostToDevice, m->stream));
-  if (vcache) VKL_CUDA(cudaMemcpyAsync(y.vcache->data(), vcache, y.vcache->device_bytes(), cudaMemcpyHostToDevice, m->stream));
+  if (vcache && y.vcache) VKL_CUDA(cudaMemcpyAsync(y.vcache->data(), vcache, y.vcache->device_bytes(), cudaMemcpyHostToDevice, m->stream));
   VKL_CUDA(cudaStreamSynchronize(m->stream));
   return VKL_OK;
 }
 
 int vkl_model_block_forward(vkl_model *m, uint32_t layer, const void *x_fp16, size_t T, size_t offset, void *out_fp16) {
   if (!m || layer >= m->cfg.layers || !x_fp16 || !out_fp16 || T == 0) return fail(VKL_INVALID_ARGUMENT, "model_block_forward: bad argument");
+  if (m->dec) return fail(VKL_UNIMPLEMENTED, "model_block_forward: Llama-2 blocks only (see vkl_model_trace_layers)");
   if (T > m->cfg.maxlen || offset + T > (size_t)2 * m->cfg.maxlen) return fail(VKL_OUT_OF_RANGE, "model_block_forward: rows or position out of range");
   Layer &y = m->L[layer];
   if (!y.attn_norm || !y.ffn_norm || !y.wq || !y.wk || !y.wv || !y.wo || !y.gate || !y.up || !y.down)
@@ -1266,7 +1279,7 @@ int vkl_model_block_forward(vkl_model *m, uint32_t layer, const void *x_fp16, si
 int vkl_model_decode_profile(vkl_model *m, uint32_t token, size_t offset, float out_us[20]) {
   VKL_OKAY(check_ready(m));
   if (!out_us) return fail(VKL_INVALID_ARGUMENT, "model_decode_profile: null output");
-  if (offset + 1 > (size_t)2 * m->cfg.maxlen) return fail(VKL_OUT_OF_RANGE, "model_decode_profile: position out of range");
+  if (offset + 1 > max_positions(m)) return fail(VKL_OUT_OF_RANGE, "model_decode_profile: position out of range");
   VKL_CUDA(cudaSetDevice(m->dev->ordinal));
   VKL_OKAY(prepare_decode(m));
   const uint32_t st[2] = {(uint32_t)offset, 0};

@@ -1,0 +1,154 @@
+// Parameters of the layer-list decoder kernels: "rows" of a weight matrix multiplied with one token
+// (rows_matvec.cu) or many (gemm_tcgen05.cu in bfloat16, gemm_f32.cu in 32-bit), and what becomes of the
+// results. All pointers are device pointers.
+//
+// Padding: every width is a multiple of 64 in memory (ldw), a head's a multiple of 16 (dp), and what a matrix
+// does with its rows changes on 32-row boundaries only; the weights' padding is zero, so the kernels have no
+// ragged edge and the padding of every activation stays zero.
+#pragma once
+#include <cuda_bf16.h>
+#include <cuda_runtime.h>
+#include <stdint.h>
+
+namespace vkl {
+
+using bf16 = __nv_bfloat16;
+
+// What the rows of a segment are.
+enum RowKind : uint32_t {
+  ROW_QUERY,      // + bias -> q [tokens, q_ld]
+  ROW_KEY,        // + bias -> this token's row of the key cache [kv head][position][dp]
+  ROW_HEAD_GATE,  // sigmoid -> gate [tokens, gate_ld] (fp32), one number per head
+  ROW_GLU,        // 32 rows = 16 gate rows, then the 16 up rows of the same outputs -> glu [tokens, glu_ld]
+  ROW_RESIDUAL,   // added to the residual stream, see Residual
+  ROW_STORE       // * scale -> f32 [tokens, f32_ld]
+};
+enum GluAct : uint32_t {
+  GLU_SILU,     // silu(g) * u
+  GLU_CLAMPED   // g = min(g, limit), u = clamp(u, +-limit); g * sigmoid(1.702 g) * (u + 1)
+};
+struct RowSeg {
+  uint32_t n0, n1;  // rows [n0, n1), multiples of 32
+  uint32_t kind;
+};
+
+// The residual stream's step: x += acc, then what comes between two layer runs (a loop's pass adds the token's
+// embedding and the pass's vector), then the next norm, which for this kind of norm needs no other element of
+// the row and so runs in the epilogue of whatever wrote x.
+struct Residual {
+  float *x;             // [tokens, ldw]
+  uint32_t ldw;
+  const float *bias;    // [ldw] or null
+  float *trace;         // optional [tokens, ldw]: x right after the layer run
+  const bf16 *emb;      // next run's pass adds embed[token], or null
+  const uint32_t *toks;
+  const float *step;    // next run's pass adds this vector [ldw], or null
+  void *h;              // next norm's output [tokens, ldw] in the compute type, or null: no norm here
+  const float *nw, *nb; // Dynamic Tanh: h = tanh(alpha x) * nw + nb
+  float alpha;
+};
+
+struct RowsOut {
+  RowSeg seg[4];
+  uint32_t nseg;
+  const float *bias;    // per row, or null
+  void *q;
+  uint32_t q_ld;
+  void *kcache;
+  uint32_t kv_heads, dp, maxlen;
+  const uint32_t *pos;  // position of token 0
+  float *gate;
+  uint32_t gate_ld;
+  void *glu;
+  uint32_t glu_ld, act;
+  float limit;
+  float *f32;
+  uint32_t f32_ld;
+  float scale;
+  Residual res;
+};
+
+// ---- one token: y = W x, weights bf16 [N, K], x in the compute type, fp32 accumulation (rows_matvec.cu) ----
+struct MvRows {
+  const bf16 *w;
+  uint32_t N, K;
+  const void *x;            // [K]
+  // Routed experts. In-projection form: the chosen experts' gate/up rows (ne each, GLU order) read x too and
+  // write xe [top, ke]. Out-projection form: N rows per expert over ke columns of xe, summed and weighted.
+  const bf16 *we;
+  uint32_t ne, ke, top;
+  const int32_t *table;     // [vocab, top]: a token id's experts
+  const uint32_t *tok;
+  void *xe;
+  uint32_t xe_ld, xe_act;
+  float xe_scale;
+  bool out_proj;
+  int use_pdl;
+  RowsOut out;
+};
+cudaError_t launch_rows_matvec(const MvRows &p, bool f32, int sms, cudaStream_t s);
+
+// ---- many tokens: Y[M,N] = A[M,K] . W[N,K]^T ----
+struct GemmRows {
+  const void *a;            // [M, K] compute type
+  const bf16 *w;            // [N, K]; grouped: [experts * N, K]
+  uint32_t M, N, K;
+  const int32_t *tile_expert;  // grouped: expert of every 128-row tile of A (-1: no tokens), or null
+  uint32_t w_rows;             // grouped: experts * N
+  uint32_t *error;
+  RowsOut out;
+};
+cudaError_t launch_gemm_rows_bf16(const GemmRows &p, cudaStream_t s);  // tcgen05
+cudaError_t launch_gemm_rows_f32(const GemmRows &p, cudaStream_t s);   // true 32-bit
+
+// ---- attention over a cache that holds one row per key head, which is key and value (shared_kv_attention.cu) ----
+struct KvAttn {
+  const void *q;            // [T, q_ld]
+  uint32_t q_ld;
+  const void *cache;        // [kv_heads][maxlen][dp]
+  void *out;                // [T, out_ld], head h at column h * dp
+  uint32_t out_ld;
+  const float *gate;        // [T, gate_ld] or null
+  uint32_t gate_ld;
+  const float *bias;        // [heads][bias_n]: log2(e) * bias at distance n (the last entry from bias_n - 1 on), or null
+  uint32_t bias_n;
+  const uint32_t *pos;      // position of row 0
+  float scale;
+  float temp_coef, temp_every;  // q is multiplied by 1 + coef * ln(floor((p + 1) / every) + 1); coef 0: not
+  uint32_t T, heads, kv_heads, dp, maxlen, splits;
+  float *scratch;           // kv_attn_scratch_bytes
+  uint32_t *counters;       // one per (row, head group), zero before and after
+  int use_pdl;
+};
+size_t kv_attn_scratch_bytes(uint32_t T, uint32_t heads, uint32_t dp, uint32_t splits);
+uint32_t kv_attn_counters(uint32_t T, uint32_t heads);
+cudaError_t launch_kv_attention(const KvAttn &p, bool f32, cudaStream_t s);
+
+// ---- routing by a token-id table, and rows (experts.cu) ----
+struct RouteTable {         // one routed layer
+  const int32_t *table;     // [vocab, top]
+  uint32_t top, experts;
+  int32_t *slot;            // [T * top]: row of the grouped buffers that holds (token, choice)
+  int32_t *token;           // [rows_pad]: token of a grouped row, -1: none
+  int32_t *tile_expert;     // [rows_pad / 128]
+};
+// Rows of the grouped buffers for T tokens: every expert's tokens padded to whole 128-row tiles.
+inline uint32_t route_rows(uint32_t T, uint32_t top, uint32_t experts) {
+  const uint32_t n = T * top, used = n < experts ? n : experts;
+  return (n / 128 + used) * 128;
+}
+cudaError_t launch_route(const RouteTable *layers, uint32_t n, uint32_t max_experts, const uint32_t *toks, uint32_t T, cudaStream_t s);
+cudaError_t launch_gather_rows(const void *src, const int32_t *rows, uint32_t n, uint32_t row_bytes, void *dst, cudaStream_t s);
+// x += sum over the token's choices of y[slot], then the residual step.
+cudaError_t launch_combine(const float *y, uint32_t y_ld, const int32_t *slot, uint32_t top, uint32_t T, const Residual &r, bool f32, cudaStream_t s);
+// x = embed[token], then the residual step without its acc.
+cudaError_t launch_embed_rows(const bf16 *emb, const uint32_t *toks, uint32_t T, const Residual &r, bool f32, cudaStream_t s);
+
+// Places a bf16 tensor [rows, cols] into a padded matrix: row r -> (r / ra) * rb + r % ra + r0, columns alike.
+struct PackMap {
+  uint32_t ra, rb, r0, ca, cb, c0;
+};
+cudaError_t launch_pack_rows(const bf16 *src, uint32_t rows, uint32_t cols, bf16 *dst, uint32_t ld, const PackMap &m, cudaStream_t s);
+cudaError_t launch_synth_bf16(bf16 *dst, uint64_t seed, uint64_t tensor, uint64_t n, float mean, float stdv, cudaStream_t s);
+
+}  // namespace vkl

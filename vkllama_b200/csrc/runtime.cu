@@ -32,6 +32,7 @@ size_t dtype_elem_bytes(int dtype) {
     case VKL_UINT32: return 4;
     case VKL_INT8: return 1;
     case VKL_Q8_0: return 1;
+    case VKL_BF16: return 2;
   }
   return 0;
 }
@@ -45,7 +46,7 @@ int recording(vkl_command *cmd, const char *who) {
 
 int tensor_new(vkl_device *dev, size_t c, size_t h, size_t w, int dtype, vkl_tensor **out) {
   if (!dev || !out) return fail(VKL_INVALID_ARGUMENT, "tensor: null device or output");
-  if (dtype < VKL_FP32 || dtype > VKL_Q8_0) return fail(VKL_INVALID_ARGUMENT, "tensor: dtype %d is unknown", dtype);
+  if (dtype < VKL_FP32 || dtype > VKL_BF16) return fail(VKL_INVALID_ARGUMENT, "tensor: dtype %d is unknown", dtype);
   vkl_tensor *t = new vkl_tensor();
   t->dev = dev;
   t->dtype = dtype;

@@ -1,0 +1,411 @@
+// Causal attention over a cache in which one row per key head is both key and value, grouped queries, no
+// rotation: a position enters as a temperature of its query and as a bias by distance; a gate per head scales
+// the output. Scores, softmax and accumulation are fp32 (scores in units of log2).
+//
+// row kernel   one token (decode), few tokens, and every call of the 32-bit mode. A CTA takes a query row, a
+//              key head and a range of the cache, and up to four of the head's query heads: every cache row is
+//              read once, and the registers that held it for the score are added to the outputs. Ranges are
+//              merged by the CTA that finishes last.
+// tile kernel  64 query rows of a head per CTA on mma.sync m16n8k16 (bf16, fp32 accumulate): a 64-row cache tile
+//              is copied to shared memory once (cp.async, double buffered) and serves Q.K^T directly and P.K
+//              through transposing loads. The 127 biases that a tile pair can need travel with the tile.
+#include <algorithm>
+
+#include "rows.cuh"
+
+namespace vkl {
+namespace {
+
+constexpr float kLog2e = 1.4426950408889634f;
+
+__device__ __forceinline__ float query_scale(const KvAttn &p, uint32_t pos) {
+  float s = p.scale;
+  if (p.temp_coef != 0.f) s *= 1.0f + p.temp_coef * logf(floorf((float)(pos + 1) / p.temp_every) + 1.0f);
+  return s * kLog2e;
+}
+__device__ __forceinline__ float bias_at(const KvAttn &p, uint32_t h, uint32_t n) {
+  return p.bias ? p.bias[(size_t)h * p.bias_n + min(n, p.bias_n - 1)] : 0.f;
+}
+
+constexpr int kRowThreads = 128;
+
+template <class T> struct Raw8;
+template <> struct Raw8<bf16> {
+  uint4 u = make_uint4(0, 0, 0, 0);
+  __device__ __forceinline__ void load(const bf16 *p) { u = *reinterpret_cast<const uint4 *>(p); }
+  __device__ __forceinline__ void get(float (&v)[8]) const { unpack8(u, v); }
+};
+template <> struct Raw8<float> {
+  float4 a = make_float4(0.f, 0.f, 0.f, 0.f), b = make_float4(0.f, 0.f, 0.f, 0.f);
+  __device__ __forceinline__ void load(const float *p) {
+    a = *reinterpret_cast<const float4 *>(p);
+    b = *reinterpret_cast<const float4 *>(p + 4);
+  }
+  __device__ __forceinline__ void get(float (&v)[8]) const {
+    v[0] = a.x; v[1] = a.y; v[2] = a.z; v[3] = a.w; v[4] = b.x; v[5] = b.y; v[6] = b.z; v[7] = b.w;
+  }
+};
+
+// LPR lanes hold one cache row (8 values each), NQ query heads per CTA. grid (kv heads x head groups, rows, splits)
+template <class T, int LPR, int NQ> __global__ void __launch_bounds__(kRowThreads) kv_row_kernel(const KvAttn p) {
+  constexpr uint32_t NS = kRowThreads / LPR, U = 4, DMAX = LPR * 8;
+  __shared__ float sm_o[kRowThreads / 32][NQ][DMAX], sm_m[kRowThreads / 32][NQ], sm_l[kRowThreads / 32][NQ];
+  __shared__ uint32_t last_s;
+  const uint32_t per = p.heads / p.kv_heads, groups = (per + NQ - 1) / NQ;
+  const uint32_t g = blockIdx.x / groups, hg = blockIdx.x % groups, h0 = g * per + hg * NQ, nh = min((uint32_t)NQ, per - hg * NQ);
+  const uint32_t m = blockIdx.y, split = blockIdx.z, tid = threadIdx.x, sub = tid / LPR, l = tid % LPR, e0 = l * 8, warp = tid >> 5;
+  const bool ev = e0 < p.dp;
+  if (p.use_pdl) asm volatile("griddepcontrol.wait;" ::: "memory");
+  const uint32_t pos = *p.pos + m, vis = pos + 1;
+  uint32_t chunk = (vis + p.splits - 1) / p.splits;
+  chunk = (chunk + 31) & ~31u;
+  const uint32_t c0 = min(split * chunk, vis), c1 = min(c0 + chunk, vis);
+  const float qs = query_scale(p, pos);
+
+  float q[NQ][8], acc[NQ][8], mx[NQ], sum[NQ];
+#pragma unroll
+  for (int i = 0; i < NQ; ++i) {
+    Raw8<T> r;
+    if (ev && i < nh) r.load(static_cast<const T *>(p.q) + (size_t)m * p.q_ld + (size_t)(h0 + i) * p.dp + e0);
+    r.get(q[i]);
+#pragma unroll
+    for (int e = 0; e < 8; ++e) {
+      q[i][e] *= qs;
+      acc[i][e] = 0.f;
+    }
+    mx[i] = -INFINITY;
+    sum[i] = 0.f;
+  }
+  const T *base = static_cast<const T *>(p.cache) + (size_t)g * p.maxlen * p.dp + e0;
+  for (uint32_t jb = c0; jb < c1; jb += NS * U) {  // the same trip count for every thread
+    Raw8<T> kr[U];
+    float s[U][NQ];
+#pragma unroll
+    for (int u = 0; u < U; ++u) {
+      const uint32_t j = jb + u * NS + sub;
+      if (ev && j < c1) kr[u].load(base + (size_t)j * p.dp);
+    }
+#pragma unroll
+    for (int u = 0; u < U; ++u) {
+      float k[8];
+      kr[u].get(k);
+      const uint32_t j = jb + u * NS + sub;
+#pragma unroll
+      for (int i = 0; i < NQ; ++i) {
+        float d = 0.f;
+#pragma unroll
+        for (int e = 0; e < 8; ++e) d = fmaf(q[i][e], k[e], d);
+#pragma unroll
+        for (int o = LPR / 2; o > 0; o >>= 1) d += __shfl_xor_sync(0xffffffffu, d, o);
+        s[u][i] = (j < c1 && i < nh) ? d + bias_at(p, h0 + i, pos - j) : -INFINITY;
+      }
+    }
+#pragma unroll
+    for (int i = 0; i < NQ; ++i) {
+      float mn = mx[i];
+#pragma unroll
+      for (int u = 0; u < U; ++u) mn = fmaxf(mn, s[u][i]);
+      const float ref = mn == -INFINITY ? 0.f : mn, corr = exp2f(mx[i] - ref);
+      mx[i] = mn;
+      sum[i] *= corr;
+#pragma unroll
+      for (int e = 0; e < 8; ++e) acc[i][e] *= corr;
+#pragma unroll
+      for (int u = 0; u < U; ++u) {
+        s[u][i] = exp2f(s[u][i] - ref);
+        sum[i] += s[u][i];
+      }
+    }
+#pragma unroll
+    for (int u = 0; u < U; ++u) {
+      float k[8];
+      kr[u].get(k);
+#pragma unroll
+      for (int i = 0; i < NQ; ++i)
+#pragma unroll
+        for (int e = 0; e < 8; ++e) acc[i][e] = fmaf(s[u][i], k[e], acc[i][e]);
+    }
+  }
+  // merge the warp's row streams, then the warps, in a fixed order
+#pragma unroll
+  for (int i = 0; i < NQ; ++i) {
+#pragma unroll
+    for (int o = LPR; o < 32; o <<= 1) {
+      const float om = __shfl_xor_sync(0xffffffffu, mx[i], o), os = __shfl_xor_sync(0xffffffffu, sum[i], o);
+      const float M = fmaxf(mx[i], om), ref = M == -INFINITY ? 0.f : M, ca = exp2f(mx[i] - ref), cb = exp2f(om - ref);
+      mx[i] = M;
+      sum[i] = sum[i] * ca + os * cb;
+#pragma unroll
+      for (int e = 0; e < 8; ++e) acc[i][e] = acc[i][e] * ca + __shfl_xor_sync(0xffffffffu, acc[i][e], o) * cb;
+    }
+    if ((tid & 31) < LPR) {
+#pragma unroll
+      for (int e = 0; e < 8; ++e) sm_o[warp][i][e0 + e] = acc[i][e];
+      if (l == 0) {
+        sm_m[warp][i] = mx[i];
+        sm_l[warp][i] = sum[i];
+      }
+    }
+  }
+  __syncthreads();
+  if (p.use_pdl) asm volatile("griddepcontrol.launch_dependents;");
+  const size_t unit = (size_t)m * gridDim.x + blockIdx.x;
+  const uint32_t rec = p.dp + 2;
+  float *part = p.scratch + unit * p.splits * NQ * rec;  // [split][NQ][dp + 2]
+  auto write = [&](uint32_t i, uint32_t d, float v) {
+    if (p.gate) v *= p.gate[(size_t)m * p.gate_ld + h0 + i];
+    store1(static_cast<T *>(p.out) + (size_t)m * p.out_ld + (size_t)(h0 + i) * p.dp + d, v);
+  };
+  for (uint32_t x = tid; x < nh * p.dp; x += kRowThreads) {
+    const uint32_t i = x / p.dp, d = x % p.dp;
+    float M = -INFINITY;
+#pragma unroll
+    for (int w = 0; w < kRowThreads / 32; ++w) M = fmaxf(M, sm_m[w][i]);
+    const float ref = M == -INFINITY ? 0.f : M;
+    float num = 0.f, den = 0.f;
+#pragma unroll
+    for (int w = 0; w < kRowThreads / 32; ++w) {
+      const float c = exp2f(sm_m[w][i] - ref);
+      num += c * sm_o[w][i][d];
+      den += c * sm_l[w][i];
+    }
+    if (p.splits == 1) {
+      write(i, d, num / den);
+    } else {
+      float *r = part + ((size_t)split * NQ + i) * rec;
+      r[d] = num;
+      if (d == 0) {
+        r[p.dp] = M;
+        r[p.dp + 1] = den;
+      }
+    }
+  }
+  if (p.splits == 1) return;
+  __threadfence();
+  __syncthreads();
+  if (tid == 0) last_s = atomicAdd(&p.counters[unit], 1u) == p.splits - 1;
+  __syncthreads();
+  if (!last_s) return;
+  __threadfence();
+  for (uint32_t x = tid; x < nh * p.dp; x += kRowThreads) {
+    const uint32_t i = x / p.dp, d = x % p.dp;
+    float M = -INFINITY;
+    for (uint32_t s = 0; s < p.splits; ++s) M = fmaxf(M, __ldcg(part + ((size_t)s * NQ + i) * rec + p.dp));
+    float num = 0.f, den = 0.f;  // split 0 is never empty: M is finite
+    for (uint32_t s = 0; s < p.splits; ++s) {
+      const float *r = part + ((size_t)s * NQ + i) * rec;
+      const float c = exp2f(__ldcg(r + p.dp) - M);
+      num += c * __ldcg(r + d);
+      den += c * __ldcg(r + p.dp + 1);
+    }
+    write(i, d, num / den);
+  }
+  if (tid == 0) p.counters[unit] = 0;
+}
+
+template <class T, int LPR> cudaError_t launch_row(const KvAttn &p, cudaStream_t s) {
+  const uint32_t per = p.heads / p.kv_heads;
+  auto kern = per >= 3 ? kv_row_kernel<T, LPR, 4> : per == 2 ? kv_row_kernel<T, LPR, 2> : kv_row_kernel<T, LPR, 1>;
+  const uint32_t nq = per >= 3 ? 4 : per;
+  cudaLaunchConfig_t cfg = {};
+  cfg.gridDim = dim3(p.kv_heads * ((per + nq - 1) / nq), p.T, p.splits);
+  cfg.blockDim = dim3(kRowThreads);
+  cfg.stream = s;
+  cudaLaunchAttribute attr[1];
+  attr[0].id = cudaLaunchAttributeProgrammaticStreamSerialization;
+  attr[0].val.programmaticStreamSerializationAllowed = 1;
+  cfg.attrs = attr;
+  cfg.numAttrs = p.use_pdl ? 1 : 0;
+  return cudaLaunchKernelEx(&cfg, kern, p);
+}
+template <class T> cudaError_t launch_row_d(const KvAttn &p, cudaStream_t s) {
+  if (p.dp <= 64) return launch_row<T, 8>(p, s);
+  if (p.dp <= 128) return launch_row<T, 16>(p, s);
+  return launch_row<T, 32>(p, s);
+}
+
+// ------------------------------------------------------------------------------------------ tiles
+__device__ __forceinline__ void mma_bf16(float (&c)[4], uint32_t a0, uint32_t a1, uint32_t a2, uint32_t a3, uint32_t b0, uint32_t b1) {
+  asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
+               : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3])
+               : "r"(a0), "r"(a1), "r"(a2), "r"(a3), "r"(b0), "r"(b1));
+}
+__device__ __forceinline__ void cp_async16(void *dst, const void *src, bool valid) {  // zero-fills when not valid
+  asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"((uint32_t)__cvta_generic_to_shared(dst)), "l"(src), "r"(valid ? 16u : 0u) : "memory");
+}
+__device__ __forceinline__ void cp_async4(void *dst, const void *src) {
+  asm volatile("cp.async.ca.shared.global [%0], [%1], 4;" ::"r"((uint32_t)__cvta_generic_to_shared(dst)), "l"(src) : "memory");
+}
+
+constexpr int QT = 64, KT = 64;
+template <int D> struct TileSmem {
+  static constexpr int LD = D + 8;  // padded rows: conflict-free fragment loads
+  bf16 q[QT * LD];
+  bf16 k[2][KT * LD];
+  float bias[2][128];
+};
+
+// D: head width rounded up to what is instantiated; dp the width in memory.
+template <int D> __global__ void __launch_bounds__(128) kv_tile_kernel(const KvAttn p) {
+  constexpr int LD = TileSmem<D>::LD;
+  extern __shared__ __align__(16) unsigned char raw[];
+  TileSmem<D> &sm = *reinterpret_cast<TileSmem<D> *>(raw);
+  const uint32_t h = blockIdx.x, g = h / (p.heads / p.kv_heads), tiles = gridDim.y, m0 = (tiles - 1 - blockIdx.y) * QT;  // longest rows first
+  const uint32_t tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, gq = lane >> 2, t = lane & 3;
+  const uint32_t T = p.T, pos0 = *p.pos, vecs = p.dp / 8;
+  const bf16 *cache = static_cast<const bf16 *>(p.cache) + (size_t)g * p.maxlen * p.dp;
+  const uint32_t jmax = pos0 + min(m0 + QT, T);  // cache rows that some row of the tile sees
+  auto fetch = [&](uint32_t j0, uint32_t b) {
+    for (uint32_t i = tid; i < KT * (D / 8); i += 128) {
+      const uint32_t r = i / (D / 8), c = i % (D / 8);
+      const bool ok = j0 + r < jmax && c < vecs;
+      cp_async16(&sm.k[b][r * LD + c * 8], cache + (ok ? (size_t)(j0 + r) * p.dp + c * 8 : 0), ok);
+    }
+    if (p.bias && tid < 127) {  // distance of (row r, column c): pos0 + m0 + r - j0 - c = entry r - c + 63
+      const int n = (int)(pos0 + m0) - (int)j0 + (int)tid - 63;
+      cp_async4(&sm.bias[b][tid], p.bias + (size_t)h * p.bias_n + min((uint32_t)max(n, 0), p.bias_n - 1));
+    }
+    asm volatile("cp.async.commit_group;" ::: "memory");
+  };
+  for (uint32_t i = tid; i < QT * (D / 8); i += 128) {
+    const uint32_t r = i / (D / 8), c = i % (D / 8);
+    const bool ok = m0 + r < T && c < vecs;
+    cp_async16(&sm.q[r * LD + c * 8], static_cast<const bf16 *>(p.q) + (ok ? (size_t)(m0 + r) * p.q_ld + (size_t)h * p.dp + c * 8 : 0), ok);
+  }
+  if (!p.bias)
+    for (uint32_t i = tid; i < 256; i += 128) sm.bias[i >> 7][i & 127] = 0.f;
+  fetch(0, 0);
+  const uint32_t rl = warp * 16 + gq, rh = rl + 8;                                       // rows in the tile
+  const uint32_t vis_lo = m0 + rl < T ? pos0 + m0 + rl + 1 : 0u, vis_hi = m0 + rh < T ? pos0 + m0 + rh + 1 : 0u;
+  const float qs_lo = query_scale(p, pos0 + m0 + rl), qs_hi = query_scale(p, pos0 + m0 + rh);
+  float o[D / 8][4];
+#pragma unroll
+  for (int i = 0; i < D / 8; ++i) o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.f;
+  float mx_lo = -INFINITY, mx_hi = -INFINITY, l_lo = 0.f, l_hi = 0.f;
+  const bf16 *qw = sm.q + rl * LD + 2 * t;
+  uint32_t b = 0;
+  for (uint32_t j0 = 0; j0 < jmax; j0 += KT, b ^= 1) {
+    asm volatile("cp.async.wait_group 0;" ::: "memory");
+    __syncthreads();  // tile b has landed for everyone, tile b ^ 1 is consumed
+    if (j0 + KT < jmax) fetch(j0 + KT, b ^ 1);
+    const bf16 *ks = sm.k[b];
+    const float *bs = sm.bias[b] + 63;
+    float sc[KT / 8][4];
+#pragma unroll
+    for (int nt = 0; nt < KT / 8; ++nt) sc[nt][0] = sc[nt][1] = sc[nt][2] = sc[nt][3] = 0.f;
+#pragma unroll
+    for (int kk = 0; kk < D / 16; ++kk) {
+      const uint32_t a0 = *reinterpret_cast<const uint32_t *>(qw + kk * 16), a1 = *reinterpret_cast<const uint32_t *>(qw + 8 * LD + kk * 16);
+      const uint32_t a2 = *reinterpret_cast<const uint32_t *>(qw + kk * 16 + 8), a3 = *reinterpret_cast<const uint32_t *>(qw + 8 * LD + kk * 16 + 8);
+#pragma unroll
+      for (int nt = 0; nt < KT / 8; ++nt) {
+        const bf16 *kr = ks + (nt * 8 + gq) * LD + kk * 16 + 2 * t;
+        mma_bf16(sc[nt], a0, a1, a2, a3, *reinterpret_cast<const uint32_t *>(kr), *reinterpret_cast<const uint32_t *>(kr + 8));
+      }
+    }
+    float tm_lo = -INFINITY, tm_hi = -INFINITY;
+#pragma unroll
+    for (int nt = 0; nt < KT / 8; ++nt) {
+      const int c = nt * 8 + 2 * t;
+      const uint32_t j = j0 + c;
+      sc[nt][0] = j < vis_lo ? fmaf(sc[nt][0], qs_lo, bs[(int)rl - c]) : -INFINITY;
+      sc[nt][1] = j + 1 < vis_lo ? fmaf(sc[nt][1], qs_lo, bs[(int)rl - c - 1]) : -INFINITY;
+      sc[nt][2] = j < vis_hi ? fmaf(sc[nt][2], qs_hi, bs[(int)rh - c]) : -INFINITY;
+      sc[nt][3] = j + 1 < vis_hi ? fmaf(sc[nt][3], qs_hi, bs[(int)rh - c - 1]) : -INFINITY;
+      tm_lo = fmaxf(tm_lo, fmaxf(sc[nt][0], sc[nt][1]));
+      tm_hi = fmaxf(tm_hi, fmaxf(sc[nt][2], sc[nt][3]));
+    }
+#pragma unroll
+    for (int w = 1; w < 4; w <<= 1) {
+      tm_lo = fmaxf(tm_lo, __shfl_xor_sync(0xffffffffu, tm_lo, w));
+      tm_hi = fmaxf(tm_hi, __shfl_xor_sync(0xffffffffu, tm_hi, w));
+    }
+    const float mn_lo = fmaxf(mx_lo, tm_lo), mn_hi = fmaxf(mx_hi, tm_hi);
+    const float ref_lo = mn_lo == -INFINITY ? 0.f : mn_lo, ref_hi = mn_hi == -INFINITY ? 0.f : mn_hi;
+    const float corr_lo = exp2f(mx_lo - ref_lo), corr_hi = exp2f(mx_hi - ref_hi);
+    mx_lo = mn_lo;
+    mx_hi = mn_hi;
+    float rs_lo = 0.f, rs_hi = 0.f;
+#pragma unroll
+    for (int nt = 0; nt < KT / 8; ++nt) {
+      sc[nt][0] = exp2f(sc[nt][0] - ref_lo);
+      sc[nt][1] = exp2f(sc[nt][1] - ref_lo);
+      sc[nt][2] = exp2f(sc[nt][2] - ref_hi);
+      sc[nt][3] = exp2f(sc[nt][3] - ref_hi);
+      rs_lo += sc[nt][0] + sc[nt][1];
+      rs_hi += sc[nt][2] + sc[nt][3];
+    }
+    l_lo = l_lo * corr_lo + rs_lo;  // this thread's columns; summed over the four threads of a row at the end
+    l_hi = l_hi * corr_hi + rs_hi;
+#pragma unroll
+    for (int i = 0; i < D / 8; ++i) {
+      o[i][0] *= corr_lo;
+      o[i][1] *= corr_lo;
+      o[i][2] *= corr_hi;
+      o[i][3] *= corr_hi;
+    }
+#pragma unroll
+    for (int j16 = 0; j16 < KT / 16; ++j16) {
+      const uint32_t a0 = pack_bf2(sc[2 * j16][0], sc[2 * j16][1]), a1 = pack_bf2(sc[2 * j16][2], sc[2 * j16][3]);
+      const uint32_t a2 = pack_bf2(sc[2 * j16 + 1][0], sc[2 * j16 + 1][1]), a3 = pack_bf2(sc[2 * j16 + 1][2], sc[2 * j16 + 1][3]);
+      const bf16 *vrow = ks + (j16 * 16 + (lane & 7) + ((lane >> 3) & 1) * 8) * LD + ((lane >> 4) & 1) * 8;
+#pragma unroll
+      for (int dt = 0; dt < D / 16; ++dt) {
+        uint32_t b0, b1, b2, b3;
+        const uint32_t addr = (uint32_t)__cvta_generic_to_shared(vrow + dt * 16);
+        asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0,%1,%2,%3}, [%4];" : "=r"(b0), "=r"(b1), "=r"(b2), "=r"(b3) : "r"(addr));
+        mma_bf16(o[2 * dt], a0, a1, a2, a3, b0, b1);
+        mma_bf16(o[2 * dt + 1], a0, a1, a2, a3, b2, b3);
+      }
+    }
+  }
+#pragma unroll
+  for (int w = 1; w < 4; w <<= 1) {
+    l_lo += __shfl_xor_sync(0xffffffffu, l_lo, w);
+    l_hi += __shfl_xor_sync(0xffffffffu, l_hi, w);
+  }
+  const uint32_t ml = m0 + rl, mh = m0 + rh;
+  const float f_lo = ml < T ? (p.gate ? p.gate[(size_t)ml * p.gate_ld + h] : 1.f) / l_lo : 0.f;
+  const float f_hi = mh < T ? (p.gate ? p.gate[(size_t)mh * p.gate_ld + h] : 1.f) / l_hi : 0.f;
+  bf16 *out = static_cast<bf16 *>(p.out) + (size_t)h * p.dp;
+#pragma unroll
+  for (int nt = 0; nt < D / 8; ++nt) {
+    const uint32_t d = nt * 8 + 2 * t;
+    if (d >= p.dp) continue;
+    if (ml < T) *reinterpret_cast<uint32_t *>(out + (size_t)ml * p.out_ld + d) = pack_bf2(o[nt][0] * f_lo, o[nt][1] * f_lo);
+    if (mh < T) *reinterpret_cast<uint32_t *>(out + (size_t)mh * p.out_ld + d) = pack_bf2(o[nt][2] * f_hi, o[nt][3] * f_hi);
+  }
+}
+
+template <int D> cudaError_t launch_tile(const KvAttn &p, cudaStream_t s) {
+  cudaError_t e = cudaFuncSetAttribute(kv_tile_kernel<D>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)sizeof(TileSmem<D>));
+  if (e != cudaSuccess) return e;
+  kv_tile_kernel<D><<<dim3(p.heads, (p.T + QT - 1) / QT), 128, sizeof(TileSmem<D>), s>>>(p);
+  return cudaGetLastError();
+}
+
+constexpr uint32_t kTileRows = 16;  // from this many query rows the tile kernel is used
+
+}  // namespace
+
+size_t kv_attn_scratch_bytes(uint32_t T, uint32_t heads, uint32_t dp, uint32_t splits) {
+  return splits < 2 ? 0 : (size_t)T * heads * 4 * splits * (dp + 2) * sizeof(float);  // at most heads (group) units of four records
+}
+uint32_t kv_attn_counters(uint32_t T, uint32_t heads) { return T * heads; }
+
+cudaError_t launch_kv_attention(const KvAttn &p, bool f32, cudaStream_t s) {
+  if (!p.T || !p.kv_heads || p.heads % p.kv_heads || p.dp % 16 || p.dp > 256 || !p.splits) return cudaErrorInvalidValue;
+  if (!f32 && p.T >= kTileRows) {
+    if (p.dp <= 32) return launch_tile<32>(p, s);
+    if (p.dp <= 48) return launch_tile<48>(p, s);
+    if (p.dp <= 64) return launch_tile<64>(p, s);
+    if (p.dp <= 96) return launch_tile<96>(p, s);
+    if (p.dp <= 128) return launch_tile<128>(p, s);
+    if (p.dp <= 192) return launch_tile<192>(p, s);
+    return launch_tile<256>(p, s);
+  }
+  if (p.T > 65535) return cudaErrorInvalidValue;
+  return f32 ? launch_row_d<float>(p, s) : launch_row_d<bf16>(p, s);
+}
+
+}  // namespace vkl
