@@ -318,8 +318,113 @@ def run_gemm(args):
                       "roofline": roof, "gpu_launches": int(vk.kernel_launches() - launches0)}))
 
 
+# Layer shapes of --design: width, heads, feed-forward, layers, vocabulary
+DESIGN_SIZES = {"1b": (2048, 16, 5632, 12, 32000), "7b": (4096, 32, 11008, 8, 32000), "13b": (5120, 40, 13824, 6, 32000)}
+
+
+def design_config(name, size, variant):
+    """A config of the design at a size: 'dense' has the closest model's layers (as many key heads as heads), 'gqa' a
+    quarter of the key heads, 'moe' 16 experts of a quarter of the width (two per token) in every other layer and a loop."""
+    d, h, f, nl, v = DESIGN_SIZES[size]
+    mix = {"heads": h, "kv_heads": h if variant == "dense" else h // 4, "dim": d // h, "vdim": d // h, "scale": (d // h) ** -0.5,
+           "bias_max": 1024, "q_temp": {"coef": 0.1, "every": 512}}
+    dense = {"kind": "dense", "ff": f, "limit": 7.0}
+    moe = {"kind": "moe", "expert": {"ff": f // 4}, "router": {"experts": 16, "top": 2}}
+    return {"architecture": name, "vocab": v, "width": d, "logit_scale": 1.0, "norm": {"eps": 1e-6},
+            "loop": {"start": 0, "stop": nl // 2, "times": 2} if variant == "moe" else None,
+            "layers": [{"type": "attention", "mixer": mix, "mlp": moe if variant == "moe" and i % 2 else dense} for i in range(nl)]}
+
+
+def design_work(size, variant, T):
+    """Algorithmic bytes of one decode token and FLOPs of a T-token prompt pass, per kernel class (the classes of
+    vkl_model_decode_profile / vkl_model_prefill_profile), for the design's variant or for 'llama'."""
+    d, h, f, nl, v = DESIGN_SIZES[size]
+    hd = d // h
+    b, fl = {"head": 2.0 * v * d}, {}
+    if variant == "llama":
+        b.update({"in": nl * 2.0 * (3 * d * d + 2 * f * d), "out": nl * 2.0 * (d * d + f * d), "attn": nl * 2.0 * 2 * d * T})
+        fl.update({"in": nl * 2.0 * T * (3 * d * d + 2 * f * d), "out": nl * 2.0 * T * (d * d + f * d), "attn": nl * 2.0 * d * T * T})
+        return b, fl
+    kv = h if variant == "dense" else h // 4
+    runs = [i for _ in range(2) for i in range(nl // 2)] + list(range(nl // 2, nl)) if variant == "moe" else list(range(nl))
+    b.update({"in": 0.0, "out": 0.0, "attn": len(runs) * 2.0 * kv * hd * T})
+    fl.update({"in": 0.0, "out": 0.0, "attn": len(runs) * 2.0 * d * T * T, "experts": 0.0})
+    for i in runs:
+        qkg, o = d * (h * hd + kv * hd + h), d * h * hd
+        e = variant == "moe" and i % 2 == 1
+        ff = 2 * (f // 4) * d if e else f * d  # one projection's weights that a token uses
+        b["in"] += 2.0 * (qkg + 2 * ff)
+        b["out"] += 2.0 * (o + ff)
+        fl["in"] += 2.0 * T * (qkg + (0 if e else 2 * ff))
+        fl["out"] += 2.0 * T * (o + (0 if e else ff))
+        fl["experts"] += 2.0 * T * 3 * ff if e else 0.0
+    # a prompt pass streams the weights of every expert that has a token
+    b["experts_prompt"] = sum(2.0 * 16 * 3 * (f // 4) * d for i in runs if variant == "moe" and i % 2 == 1)
+    return b, fl
+
+
+def run_design(args):
+    """Prefill and decode throughput of a decoder design (random weights) at a few layer shapes beside the Llama-2
+    driver with FP16 weights at the same shape (the closest model of the library: 16-bit weights, the same GEMM), with
+    every kernel class's share of its roofline. Weights are larger than L2 and every pass reads all of them."""
+    import vkllama_b200 as vk
+    from vkllama_b200.synth import synth_tokens
+    hbm, hk = peak_hbm()
+    tens, tk = peak_tensor()
+    dev = vk.Device(0)
+    T, n_dec, rows = args.design_prompt, args.design_decode, []
+    sampler = ClockSampler(0)
+    sampler.start()
+    launches0 = vk.kernel_launches()
+    for size in args.design_sizes.split(","):
+        d, h, f, nl, v = DESIGN_SIZES[size]
+        for variant in args.design_variants.split(","):
+            if variant == "llama":
+                m = vk.Model(dev, d, h, f, v, nl, max(4096, T + n_dec + 1), weight_dtype=vk.FP16)
+            else:
+                m = vk.Model.from_config(dev, design_config(args.design, size, variant), max(4096, T + n_dec + 1), vk.BF16)
+            m.synth_weights(17)
+            prompt = synth_tokens(17, 1000, T, v)
+            pre, dec = [], []
+            for i in range(args.warmup + args.steps):
+                _, p_ms, d_ms = m.generate(prompt, n_dec + 1)
+                if i >= args.warmup:
+                    pre.append(p_ms)
+                    dec.append(d_ms / n_dec)
+            reps = 10
+            pp = np.mean([m.prefill_profile(prompt) for _ in range(reps + 2)][2:], axis=0)
+            dp = np.mean([m.decode_profile(int(prompt[i]), T + i) for i in range(reps + 2)][2:], axis=0)
+            b, fl = design_work(size, variant, T)
+            dt = {"in": dp[1] + dp[4], "attn": dp[2], "out": dp[3] + dp[5], "head": dp[6]}
+            if variant == "llama":
+                pt = {"in": pp[1] + pp[4], "attn": pp[2], "out": pp[3] + pp[5]}
+            elif variant == "moe":
+                pt = {"in": pp[1], "attn": pp[2], "out": pp[3], "experts": pp[4] + pp[5]}
+            else:
+                pt = {"in": pp[1], "attn": pp[2], "out": pp[3]}
+            weights = b["in"] + b["out"] + b["head"]
+            rows.append({"size": size, "variant": variant, "prefill_tokens_per_s": T / (np.median(pre) * 1e-3), "decode_tokens_per_s": 1000.0 / np.median(dec),
+                         "prefill_ms": float(np.median(pre)), "decode_ms": float(np.median(dec)),
+                         "decode_frac_of_hbm": (weights + b["attn"]) / (np.median(dec) * 1e-3) / 1e9 / hbm,
+                         "prefill_frac_of_tensor": sum(fl.values()) / (np.median(pre) * 1e-3) / 1e12 / tens,
+                         "decode_kernels": {k: {"us": float(dt[k]), "frac_of_hbm": b[k] / (dt[k] * 1e-6) / 1e9 / hbm} for k in dt},
+                         "prefill_kernels": {k: {"us": float(pt[k]), "frac_of_tensor": fl[k] / (pt[k] * 1e-6) / 1e12 / tens} for k in pt}})
+            if variant == "moe":  # few tokens per expert: the weights' stream is the lower roof
+                rows[-1]["prefill_kernels"]["experts"]["frac_of_hbm"] = b["experts_prompt"] / (pt["experts"] * 1e-6) / 1e9 / hbm
+            m.close()
+    print(json.dumps({"metric": "design_throughput", "design": args.design, "prompt_tokens": T, "decode_tokens": n_dec, "steps": args.steps, "warmup": args.warmup,
+                      "peaks": {"hbm_gbs": hbm, "bf16_tflops": tens, "kind": [hk, tk]}, "data": "synthetic",
+                      "what": "throughputs: CUDA events inside vkl_model_generate, median of steps; kernels: an event after every launch of one pass, mean of 10",
+                      "gpu_launches": int(vk.kernel_launches() - launches0), "clocks": sampler.stop(), "results": rows}))
+
+
 def main():
     ap = argparse.ArgumentParser()
+    ap.add_argument("--design", default=None, help="a registered decoder design: its throughput beside the Llama-2 driver's at equal size, instead of the token loop")
+    ap.add_argument("--design-sizes", default="1b,7b,13b")
+    ap.add_argument("--design-variants", default="llama,dense,gqa,moe")
+    ap.add_argument("--design-prompt", type=int, default=512)
+    ap.add_argument("--design-decode", type=int, default=64)
     ap.add_argument("--micro", default=None, help="'all' or ROWSxK: Q8_0 mat-vec microbenchmark instead of the token loop")
     ap.add_argument("--micro-tokens", default="1,2,4,8,16,64")
     ap.add_argument("--gemm", default=None, help="MxNxK: tensor-core prefill GEMM microbenchmark instead of the token loop")
@@ -349,6 +454,10 @@ def main():
     if args.gemm:
         if rank == 0:
             run_gemm(args)
+        return 0
+    if args.design:
+        if rank == 0:
+            run_design(args)
         return 0
 
     import vkllama_b200 as vk

@@ -323,6 +323,11 @@ int vkl_model_block_forward(vkl_model *m, uint32_t layer, const void *x_fp16, si
  * first CTA; 0 on the multi-kernel path, which is timed with an event after every launch).
  * Appends to the KV cache at `offset`. */
 int vkl_model_decode_profile(vkl_model *m, uint32_t token, size_t offset, float out_us[20]);
+/* The same for one pass over n >= 2 prompt tokens from position 0: out_us[0..7] by the classes above. A
+ * decoder design's classes: 1 everything that reads the norm, 2 attention, 3 out-projection of a prompt pass,
+ * 4 the experts' gate/up rows (with routing gather), 5 out-projection of a decode step, the experts' down rows
+ * and their sum. */
+int vkl_model_prefill_profile(vkl_model *m, const uint32_t *toks, size_t n, float out_us[10]);
 /* The same step with a global-timer stamp (ns) by every CTA of the persistent kernel at six
  * points of every op: out[(op * grid + cta) * 8 + k], k = 0 op entered, 1 input vector
  * complete, 2 the CTA's first warp finished its weight stream, 3 all its warps did,

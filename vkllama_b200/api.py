@@ -98,6 +98,7 @@ def load_library():
         "vkl_model_last_token": [vp, C.POINTER(u32)], "vkl_model_read_kv": [vp, u32, vp, vp], "vkl_model_write_kv": [vp, u32, vp, vp],
         "vkl_model_block_forward": [vp, u32, vp, sz, sz, vp],
         "vkl_model_decode_profile": [vp, u32, sz, C.POINTER(f32)],
+        "vkl_model_prefill_profile": [vp, vp, sz, C.POINTER(f32)],
         "vkl_model_decode_trace": [vp, u32, sz, vp, sz, C.POINTER(u32), C.POINTER(u32), vp],
         "vkl_model_tp_buffer": [vp, pvp, C.POINTER(sz)], "vkl_model_tp_connect": [vp, pvp, i32],
         "vkl_model_set_wait_limit": [vp, u32],
@@ -757,6 +758,12 @@ class Model:
         """Per-kernel-class device microseconds of one decode step (see the header)."""
         out = (f32 * 20)()
         _ck(self.L.vkl_model_decode_profile(self.h, token, offset, out))
+        return list(out)
+
+    def prefill_profile(self, toks):
+        """Per-kernel-class device microseconds of one pass over prompt tokens from position 0 (see the header)."""
+        t, out = np.ascontiguousarray(toks, np.uint32), (f32 * 10)()
+        _ck(self.L.vkl_model_prefill_profile(self.h, _ptr(t), t.size, out))
         return list(out)
 
     def decode_trace(self, token, offset):

@@ -1365,6 +1365,32 @@ int vkl_model_decode_profile(vkl_model *m, uint32_t token, size_t offset, float 
   return VKL_OK;
 }
 
+int vkl_model_prefill_profile(vkl_model *m, const uint32_t *toks, size_t n, float out_us[10]) {
+  VKL_OKAY(check_ready(m));
+  if (!toks || !out_us || n < 2) return fail(VKL_INVALID_ARGUMENT, "model_prefill_profile: needs at least two tokens and an output");
+  if (n > m->cfg.maxlen) return fail(VKL_OUT_OF_RANGE, "model_prefill_profile: %zu tokens exceed the context length %u", n, m->cfg.maxlen);
+  if (m->cfg.tp_size > 1) return fail(VKL_UNIMPLEMENTED, "model_prefill_profile: single-GPU models");
+  VKL_OKAY(check_ids(m, toks, n));
+  VKL_CUDA(cudaSetDevice(m->dev->ordinal));
+  VKL_OKAY(ensure_rows(m, (uint32_t)n));
+  const uint32_t st[2] = {0, 0};
+  VKL_CUDA(cudaMemcpyAsync(m->state->data(), st, 8, cudaMemcpyHostToDevice, m->stream));
+  VKL_CUDA(cudaMemcpyAsync(m->toks->data(), toks, n * 4, cudaMemcpyHostToDevice, m->stream));
+  Marker mk;
+  mk.s = m->stream;
+  const int rc = run_tokens(m, (uint32_t)n, false, &mk);
+  const cudaError_t e = cudaStreamSynchronize(m->stream);
+  for (int i = 0; i < 10; ++i) out_us[i] = 0.f;
+  for (size_t i = 1; i < mk.ev.size(); ++i) {
+    float ms = 0.f;
+    if (rc == VKL_OK && e == cudaSuccess && cudaEventElapsedTime(&ms, mk.ev[i - 1], mk.ev[i]) == cudaSuccess && mk.cls[i] >= 0) out_us[mk.cls[i]] += ms * 1000.f;
+  }
+  for (cudaEvent_t ev : mk.ev) cudaEventDestroy(ev);
+  VKL_OKAY(rc);
+  if (e != cudaSuccess) return fail(VKL_INTERNAL, "model_prefill_profile: %s", cudaGetErrorString(e));
+  return check_gemm(m);
+}
+
 int vkl_model_decode_trace(vkl_model *m, uint32_t token, size_t offset, unsigned long long *out, size_t cap, uint32_t *nops, uint32_t *grid, uint32_t *kinds) {
   VKL_OKAY(check_ready(m));
   if (!nops || !grid) return fail(VKL_INVALID_ARGUMENT, "model_decode_trace: null argument");

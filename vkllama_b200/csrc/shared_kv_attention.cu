@@ -28,6 +28,7 @@ __device__ __forceinline__ float bias_at(const KvAttn &p, uint32_t h, uint32_t n
 }
 
 constexpr int kRowThreads = 128;
+constexpr uint32_t kMaxSplits = 32, kSplitRows = 64;  // a split holds about this many cache rows: a short cache uses fewer splits
 
 template <class T> struct Raw8;
 template <> struct Raw8<bf16> {
@@ -50,6 +51,7 @@ template <> struct Raw8<float> {
 template <class T, int LPR, int NQ> __global__ void __launch_bounds__(kRowThreads) kv_row_kernel(const KvAttn p) {
   constexpr uint32_t NS = kRowThreads / LPR, U = 4, DMAX = LPR * 8;
   __shared__ float sm_o[kRowThreads / 32][NQ][DMAX], sm_m[kRowThreads / 32][NQ], sm_l[kRowThreads / 32][NQ];
+  __shared__ float sm_pm[kMaxSplits][NQ], sm_pl[kMaxSplits][NQ];
   __shared__ uint32_t last_s;
   const uint32_t per = p.heads / p.kv_heads, groups = (per + NQ - 1) / NQ;
   const uint32_t g = blockIdx.x / groups, hg = blockIdx.x % groups, h0 = g * per + hg * NQ, nh = min((uint32_t)NQ, per - hg * NQ);
@@ -57,7 +59,9 @@ template <class T, int LPR, int NQ> __global__ void __launch_bounds__(kRowThread
   const bool ev = e0 < p.dp;
   if (p.use_pdl) asm volatile("griddepcontrol.wait;" ::: "memory");
   const uint32_t pos = *p.pos + m, vis = pos + 1;
-  uint32_t chunk = (vis + p.splits - 1) / p.splits;
+  const uint32_t splits = min(p.splits, (vis + kSplitRows - 1) / kSplitRows);
+  if (split >= splits) return;
+  uint32_t chunk = (vis + splits - 1) / splits;
   chunk = (chunk + 31) & ~31u;
   const uint32_t c0 = min(split * chunk, vis), c1 = min(c0 + chunk, vis);
   const float qs = query_scale(p, pos);
@@ -169,7 +173,7 @@ template <class T, int LPR, int NQ> __global__ void __launch_bounds__(kRowThread
       num += c * sm_o[w][i][d];
       den += c * sm_l[w][i];
     }
-    if (p.splits == 1) {
+    if (splits == 1) {
       write(i, d, num / den);
     } else {
       float *r = part + ((size_t)split * NQ + i) * rec;
@@ -180,23 +184,29 @@ template <class T, int LPR, int NQ> __global__ void __launch_bounds__(kRowThread
       }
     }
   }
-  if (p.splits == 1) return;
+  if (splits == 1) return;
   __threadfence();
   __syncthreads();
-  if (tid == 0) last_s = atomicAdd(&p.counters[unit], 1u) == p.splits - 1;
+  if (tid == 0) last_s = atomicAdd(&p.counters[unit], 1u) == splits - 1;
   __syncthreads();
   if (!last_s) return;
   __threadfence();
+  for (uint32_t x = tid; x < splits * nh; x += kRowThreads) {
+    const float *r = part + ((size_t)(x / nh) * NQ + x % nh) * rec + p.dp;
+    sm_pm[x / nh][x % nh] = __ldcg(r);
+    sm_pl[x / nh][x % nh] = __ldcg(r + 1);
+  }
+  __syncthreads();
   for (uint32_t x = tid; x < nh * p.dp; x += kRowThreads) {
     const uint32_t i = x / p.dp, d = x % p.dp;
-    float M = -INFINITY;
-    for (uint32_t s = 0; s < p.splits; ++s) M = fmaxf(M, __ldcg(part + ((size_t)s * NQ + i) * rec + p.dp));
-    float num = 0.f, den = 0.f;  // split 0 is never empty: M is finite
-    for (uint32_t s = 0; s < p.splits; ++s) {
-      const float *r = part + ((size_t)s * NQ + i) * rec;
-      const float c = exp2f(__ldcg(r + p.dp) - M);
-      num += c * __ldcg(r + d);
-      den += c * __ldcg(r + p.dp + 1);
+    float M = -INFINITY;  // split 0 is never empty: M becomes finite
+    for (uint32_t s = 0; s < splits; ++s) M = fmaxf(M, sm_pm[s][i]);
+    float num = 0.f, den = 0.f;
+#pragma unroll 8
+    for (uint32_t s = 0; s < splits; ++s) {
+      const float c = exp2f(sm_pm[s][i] - M);
+      num += c * __ldcg(part + ((size_t)s * NQ + i) * rec + d);
+      den += c * sm_pl[s][i];
     }
     write(i, d, num / den);
   }
@@ -394,7 +404,7 @@ size_t kv_attn_scratch_bytes(uint32_t T, uint32_t heads, uint32_t dp, uint32_t s
 uint32_t kv_attn_counters(uint32_t T, uint32_t heads) { return T * heads; }
 
 cudaError_t launch_kv_attention(const KvAttn &p, bool f32, cudaStream_t s) {
-  if (!p.T || !p.kv_heads || p.heads % p.kv_heads || p.dp % 16 || p.dp > 256 || !p.splits) return cudaErrorInvalidValue;
+  if (!p.T || !p.kv_heads || p.heads % p.kv_heads || p.dp % 16 || p.dp > 256 || !p.splits || p.splits > kMaxSplits) return cudaErrorInvalidValue;
   if (!f32 && p.T >= kTileRows) {
     if (p.dp <= 32) return launch_tile<32>(p, s);
     if (p.dp <= 48) return launch_tile<48>(p, s);
