@@ -484,6 +484,16 @@ class Model {
     vocab_ = c.vocab;
     return ToStatus(vkl_model_create(gpu_->handle(), &k, &m_));
   }
+  // A registered decoder design from a folder with config.json and model.safetensors (no counterpart in the reference).
+  absl::Status init_folder(const std::string &path, uint32_t context_length, bool in_32bit = false) {
+    gpu_ = new GPUDevice(dev_);
+    VKLLAMA_STATUS_OK(gpu_->init());
+    VKLLAMA_STATUS_OK(ToStatus(vkl_model_load_folder(gpu_->handle(), path.c_str(), context_length, in_32bit ? VKL_FP32 : VKL_BF16, &m_)));
+    uint32_t shape[6];
+    VKLLAMA_STATUS_OK(ToStatus(vkl_model_shape(m_, shape)));
+    vocab_ = shape[0];
+    return absl::OkStatus();
+  }
   absl::Status load_tensor(const std::string &name, uint32_t gguf_type, const void *weights_data, size_t bsize) {
     const int dt = gguf_type == 0 ? FP32 : gguf_type == 1 ? FP16 : gguf_type == 8 ? Q8_0 : INT8;
     return ToStatus(vkl_model_set_weight(m_, name.c_str(), dt, weights_data, bsize));

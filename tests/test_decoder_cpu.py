@@ -85,7 +85,7 @@ def test_loop_order_shows():
     assert U.rel_err(outputs(MIX, V, toks), want) > 2 * U.REL["bfloat16"]
 
 
-@pytest.mark.parametrize("rows,far", [(32, 240), (32, 256), (20, 50), (24, 96), (16, 512), (6, 27), (2, 5), (64, 4096), (9, 30)])
+@pytest.mark.parametrize("rows,far", [(32, 200), (32, 256), (20, 50), (24, 96), (16, 512), (6, 27), (2, 5), (64, 4096), (9, 30)])
 def test_distance_buckets(rows, far):
     got = [vk.distance_bucket(n, rows, far) for n in range(far + 40)]
     assert got == [D.distance_bucket(n, rows, far) for n in range(far + 40)]

@@ -434,7 +434,7 @@ int decoder_ensure_rows(vkl_model *m, uint32_t T) {
   for (size_t i = 0; i < d->L.size(); ++i) {
     const AttnSpec &a = d->spec.layers[i].attn;
     const uint32_t per = a.heads / a.kv_heads, units = a.kv_heads * ((per + 3) / 4);
-    m->splits = std::max(m->splits, std::min(32u, (uint32_t)(2 * m->dev->prop.multiProcessorCount) / units));
+    m->splits = std::max(m->splits, std::min(32u, (uint32_t)(6 * m->dev->prop.multiProcessorCount) / units));
   }
   size_t sc = 0;
   for (size_t i = 0; i < d->L.size(); ++i) sc = std::max(sc, kv_attn_scratch_bytes(1, d->spec.layers[i].attn.heads, d->L[i].dp, m->splits));

@@ -17,7 +17,7 @@ struct Marker;
 struct AttnSpec {
   uint32_t heads = 0, kv_heads = 0, dim = 0;
   float scale = 1.f;
-  float temp_coef = 0.f;      // query temperature 1 + coef * ln(floor((p + 1) / every) + 1)
+  float temp_coef = 0.f;      // query temperature, see KvAttn
   uint32_t temp_every = 1;
   uint32_t bias_max = 0;      // distance at which the bucketed bias saturates; the buckets' number is the table's
 };

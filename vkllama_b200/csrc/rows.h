@@ -24,8 +24,8 @@ enum RowKind : uint32_t {
   ROW_STORE       // * scale -> f32 [tokens, f32_ld]
 };
 enum GluAct : uint32_t {
-  GLU_SILU,     // silu(g) * u
-  GLU_CLAMPED   // g = min(g, limit), u = clamp(u, +-limit); g * sigmoid(1.702 g) * (u + 1)
+  GLU_SILU,     // the gate's SiLU times up
+  GLU_CLAMPED   // gate cut off above the limit, up at both ends; quick-GELU of the gate times (1 + up)
 };
 struct RowSeg {
   uint32_t n0, n1;  // rows [n0, n1), multiples of 32
@@ -114,7 +114,7 @@ struct KvAttn {
   uint32_t bias_n;
   const uint32_t *pos;      // position of row 0
   float scale;
-  float temp_coef, temp_every;  // q is multiplied by 1 + coef * ln(floor((p + 1) / every) + 1); coef 0: not
+  float temp_coef, temp_every;  // query temperature at p: 1 + temp_coef log(1 + k), k = whole temp_every-s in p + 1; temp_coef 0: none
   uint32_t T, heads, kv_heads, dp, maxlen, splits;
   float *scratch;           // kv_attn_scratch_bytes
   uint32_t *counters;       // one per (row, head group), zero before and after

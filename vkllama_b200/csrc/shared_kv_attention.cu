@@ -88,12 +88,13 @@ template <class T, int LPR, int NQ> __global__ void __launch_bounds__(kRowThread
     for (int u = 0; u < U; ++u) {
       const uint32_t j = jb + u * NS + sub;
       if (ev && j < c1) kr[u].load(base + (size_t)j * p.dp);
+#pragma unroll
+      for (int i = 0; i < NQ; ++i) s[u][i] = (j < c1 && i < nh) ? bias_at(p, h0 + i, pos - j) : -INFINITY;
     }
 #pragma unroll
     for (int u = 0; u < U; ++u) {
       float k[8];
       kr[u].get(k);
-      const uint32_t j = jb + u * NS + sub;
 #pragma unroll
       for (int i = 0; i < NQ; ++i) {
         float d = 0.f;
@@ -101,7 +102,7 @@ template <class T, int LPR, int NQ> __global__ void __launch_bounds__(kRowThread
         for (int e = 0; e < 8; ++e) d = fmaf(q[i][e], k[e], d);
 #pragma unroll
         for (int o = LPR / 2; o > 0; o >>= 1) d += __shfl_xor_sync(0xffffffffu, d, o);
-        s[u][i] = (j < c1 && i < nh) ? d + bias_at(p, h0 + i, pos - j) : -INFINITY;
+        s[u][i] += d;
       }
     }
 #pragma unroll
@@ -154,8 +155,8 @@ template <class T, int LPR, int NQ> __global__ void __launch_bounds__(kRowThread
   __syncthreads();
   if (p.use_pdl) asm volatile("griddepcontrol.launch_dependents;");
   const size_t unit = (size_t)m * gridDim.x + blockIdx.x;
-  const uint32_t rec = p.dp + 2;
-  float *part = p.scratch + unit * p.splits * NQ * rec;  // [split][NQ][dp + 2]
+  const uint32_t rec = p.dp + 4;
+  float *part = p.scratch + unit * p.splits * NQ * rec;  // [split][NQ][dp + 4]: output, max, sum
   auto write = [&](uint32_t i, uint32_t d, float v) {
     if (p.gate) v *= p.gate[(size_t)m * p.gate_ld + h0 + i];
     store1(static_cast<T *>(p.out) + (size_t)m * p.out_ld + (size_t)(h0 + i) * p.dp + d, v);
@@ -197,18 +198,26 @@ template <class T, int LPR, int NQ> __global__ void __launch_bounds__(kRowThread
     sm_pl[x / nh][x % nh] = __ldcg(r + 1);
   }
   __syncthreads();
-  for (uint32_t x = tid; x < nh * p.dp; x += kRowThreads) {
-    const uint32_t i = x / p.dp, d = x % p.dp;
+  for (uint32_t x = tid; x < nh * (p.dp / 4); x += kRowThreads) {
+    const uint32_t i = x / (p.dp / 4), d = x % (p.dp / 4) * 4;
     float M = -INFINITY;  // split 0 is never empty: M becomes finite
     for (uint32_t s = 0; s < splits; ++s) M = fmaxf(M, sm_pm[s][i]);
-    float num = 0.f, den = 0.f;
+    float4 num = make_float4(0.f, 0.f, 0.f, 0.f);
+    float den = 0.f;
 #pragma unroll 8
     for (uint32_t s = 0; s < splits; ++s) {
       const float c = exp2f(sm_pm[s][i] - M);
-      num += c * __ldcg(part + ((size_t)s * NQ + i) * rec + d);
-      den += c * sm_pl[s][i];
+      const float4 v = __ldcg(reinterpret_cast<const float4 *>(part + ((size_t)s * NQ + i) * rec + d));
+      num.x = fmaf(c, v.x, num.x);
+      num.y = fmaf(c, v.y, num.y);
+      num.z = fmaf(c, v.z, num.z);
+      num.w = fmaf(c, v.w, num.w);
+      den = fmaf(c, sm_pl[s][i], den);
     }
-    write(i, d, num / den);
+    write(i, d, num.x / den);
+    write(i, d + 1, num.y / den);
+    write(i, d + 2, num.z / den);
+    write(i, d + 3, num.w / den);
   }
   if (tid == 0) p.counters[unit] = 0;
 }
@@ -399,7 +408,7 @@ constexpr uint32_t kTileRows = 16;  // from this many query rows the tile kernel
 }  // namespace
 
 size_t kv_attn_scratch_bytes(uint32_t T, uint32_t heads, uint32_t dp, uint32_t splits) {
-  return splits < 2 ? 0 : (size_t)T * heads * 4 * splits * (dp + 2) * sizeof(float);  // at most heads (group) units of four records
+  return splits < 2 ? 0 : (size_t)T * heads * 4 * splits * (dp + 4) * sizeof(float);  // at most heads (group) units of four records
 }
 uint32_t kv_attn_counters(uint32_t T, uint32_t heads) { return T * heads; }
 
