@@ -275,8 +275,15 @@ int vkl_model_forward_rows(vkl_model *m, const uint32_t *toks, size_t n, size_t 
 int vkl_model_trace_layers(vkl_model *m, const uint32_t *toks, size_t n, size_t offset, float *out);
 /* vocabulary, width, layers (layer runs of a decoder design), maxlen, compute dtype, heads. */
 int vkl_model_shape(const vkl_model *m, uint32_t out6[6]);
-/* One layer's (layer run's) key cache: heads, maxlen, head width in memory, dtype. */
+/* One layer's (layer run's) key cache: heads, maxlen, head width in memory, dtype; all 0 where a
+ * layer has none (a recurrent layer, or one that uses another's). */
 int vkl_model_kv_shape(const vkl_model *m, uint32_t layer, uint32_t out4[4]);
+/* All that a layer (layer run) keeps of a sequence: key heads, maxlen, key width, value width (0: the
+ * keys are the values), dtype; of a recurrent layer, states (fp32): heads, rows, columns, and the ring
+ * of past projections: rows, columns. 0 for what a layer does not have. */
+int vkl_model_cache_info(const vkl_model *m, uint32_t layer, uint32_t out10[10]);
+/* A recurrent layer's states [heads][value][key], padded widths. */
+int vkl_model_read_state(vkl_model *m, uint32_t layer, float *state);
 /* A model from a checkpoint folder: config.json names the architecture and its sizes,
  * model.safetensors holds the weights (bfloat16, integer tables int32). The architecture is looked
  * up in the library's registry; maxlen is the context length, compute_dtype VKL_BF16 or VKL_FP32
@@ -285,6 +292,9 @@ int vkl_model_load_folder(vkl_device *dev, const char *path, uint32_t maxlen, in
 /* The same from the text of a config.json, without weights (vkl_model_set_weight by the
  * checkpoint's tensor names, BF16 or UINT32, or vkl_model_synth_weights). */
 int vkl_model_create_config(vkl_device *dev, const char *config_json, uint32_t maxlen, int compute_dtype, vkl_model **out);
+/* The same for a design whose config leaves sizes to its tensors: shapes_json gives them as a
+ * safetensors header does, {"name": {"shape": [rows, cols]}, ...}; NULL for none. */
+int vkl_model_create_config_shapes(vkl_device *dev, const char *config_json, const char *shapes_json, uint32_t maxlen, int compute_dtype, vkl_model **out);
 /* Names of the registered architectures, separated by commas. */
 const char *vkl_model_architectures(void);
 /* Row of a distance-bias table with `rows` rows for a key n positions back; -1 when the table

@@ -107,20 +107,27 @@ def distance_bias(table, far, n_max):
     return np.stack([table[distance_bucket(n, table.shape[0], far)] for n in range(n_max + 1)])
 
 
-def causal_attention(q, k, v, scale, bias=None):
-    """q [T,H,d], k [T,G,d], v [T,G,e]; bias [distance, H] or None -> [T,H,e]."""
+def causal_attention(q, k, v, scale, bias=None, window=None, sink=None):
+    """q [T,H,d], k [T,G,d], v [T,G,e]; bias [distance, H] or None; window: keys a query sees, itself included, or
+    None; sink [H] or None: one more term of each head's denominator, without a value -> [T,H,e]."""
     T, H, _ = q.shape
     per = H // k.shape[1]
     out = np.zeros((T, H, v.shape[2]), q.dtype)
     back = np.arange(T)[:, None] - np.arange(T)[None, :]
-    seen = back >= 0
+    seen = (back >= 0) & (back < window) if window else back >= 0
     for h in range(H):
         s = (q[:, h] @ k[:, h // per].T) * scale
         if bias is not None:
             s = s + bias[np.maximum(back, 0), h]
         s = np.where(seen, s, -np.inf)
-        p = np.exp(s - s.max(1, keepdims=True))
-        out[:, h] = (p / p.sum(1, keepdims=True)) @ v[:, h // per]
+        top = s.max(1, keepdims=True)
+        if sink is not None:
+            top = np.maximum(top, sink[h])
+        p = np.exp(s - top)
+        den = p.sum(1, keepdims=True)
+        if sink is not None:
+            den = den + np.exp(sink[h] - top)
+        out[:, h] = (p / den) @ v[:, h // per]
     return out
 
 
@@ -165,6 +172,135 @@ def feed_forward(h, W, p, mlp, tokens):
     return table_experts(h, W, p, tokens)
 
 
+def rms(x, eps):
+    """x over its root mean square."""
+    return x / np.sqrt((x * x).mean(-1, keepdims=True) + eps)
+
+
+def centred_rms_norm(x, w, eps):
+    """The weight is stored as its difference from one."""
+    return rms(x, eps) * (1.0 + w)
+
+
+def rotation_frequencies(base, dims, scaling=None):
+    """Angle per position of every pair; scaling stretches long wavelengths by a factor, short ones not at all, with
+    a linear passage between original/high and original/low."""
+    f = np.asarray(base, np.float64) ** (-np.arange(0, dims, 2) / dims)
+    if not scaling:
+        return f
+    out = np.empty_like(f)
+    for i, fi in enumerate(f):
+        wave = 2 * math.pi / fi
+        if wave < scaling["original"] / scaling["high"]:
+            out[i] = fi
+        elif wave > scaling["original"] / scaling["low"]:
+            out[i] = fi / scaling["factor"]
+        else:
+            s = (scaling["original"] / wave - scaling["low"]) / (scaling["high"] - scaling["low"])
+            out[i] = (1 - s) * fi / scaling["factor"] + s * fi
+    return out
+
+
+def rotate_pairs(x, pos, freq):
+    """x [T,H,d]: neighbours (2i, 2i+1) turn by pos * freq[i]; dimensions beyond the pairs stay."""
+    n = 2 * len(freq)
+    a = np.asarray(pos, np.float64)[:, None, None] * freq
+    c, s = np.cos(a).astype(x.dtype), np.sin(a).astype(x.dtype)
+    u, v = x[..., 0:n:2], x[..., 1:n:2]
+    y = x.copy()
+    y[..., 0:n:2], y[..., 1:n:2] = u * c - v * s, v * c + u * s
+    return y
+
+
+def windowed_mixer(h, W, p, mix, eps, kv=None, attend=causal_attention, turn=rotate_pairs, freq_of=rotation_frequencies):
+    """Norm over the whole query and key projection, rotation, a window and a sink per head. kv: the keys (after norm
+    and rotation) and values of an earlier layer, which this one uses instead of its own. Returns output, keys, values."""
+    T, H, G, d, e = h.shape[0], mix["heads"], mix["kv_heads"], mix["dim"], mix["vdim"]
+    freq, pos = freq_of(mix["rot"]["base"], mix["rot"]["dims"], mix["rot"].get("scaling")), np.arange(T)
+
+    def side(name, heads):
+        y = rms(linear(W["%s.%s" % (p, name)], h), eps) * W["%s.%s.norm" % (p, name)]
+        return turn(y.reshape(T, heads, d), pos, freq)
+
+    q = side("q", H)
+    k, v = kv if kv is not None else (side("k", G), linear(W[p + ".v"], h).reshape(T, G, e))
+    o = attend(q, k, v, mix["scale"], window=mix["mask"]["size"], sink=W[p + ".sink"])
+    return linear(W[p + ".o"], o.reshape(T, H * e)), k, v
+
+
+def silu(z):
+    return z * sigmoid(z)
+
+
+def short_convolution(x, taps):
+    """x [T,C], taps [C,n]: causal, the last column is the current token's."""
+    T, n = x.shape[0], taps.shape[1]
+    y = np.zeros_like(x)
+    for j in range(n):
+        back = n - 1 - j
+        y[back:] += x[:T - back] * taps[:, j] if back else x * taps[:, j]
+    return y
+
+
+def unit(x):
+    return x / np.sqrt((x * x).sum(-1, keepdims=True) + 1e-6)
+
+
+def softplus(z):
+    return np.logaddexp(0.0, z)
+
+
+def delta_recurrence(q, k, v, g, beta, S=None):
+    """q, k, g [T,H,d], v [T,H,e], beta [T,H]: one token after the other, the read-out after the write."""
+    T, H, d = q.shape
+    S = np.zeros((H, d, v.shape[2]), q.dtype) if S is None else S
+    out = np.zeros(v.shape, q.dtype)
+    for t in range(T):
+        S = g[t][:, :, None] * S
+        u = beta[t][:, None] * (v[t] - np.einsum("hde,hd->he", S, k[t]))
+        S = S + k[t][:, :, None] * u[:, None, :]
+        out[t] = np.einsum("hde,hd->he", S, q[t])
+    return out
+
+
+def delta_mixer(h, W, p, mix, eps, conv=short_convolution, recur=delta_recurrence, unit_of=unit):
+    """Gated delta rule with a decay per head and key channel."""
+    T, H, G, d, e = h.shape[0], mix["heads"], mix["kv_heads"], mix["dim"], mix["vdim"]
+    side = lambda n: silu(conv(linear(W["%s.%s" % (p, n)], h), W["%s.%s.conv" % (p, n)]))
+    q = np.repeat(unit_of(side("q").reshape(T, G, d)) * d ** -0.5, H // G, 1)
+    k = np.repeat(unit_of(side("k").reshape(T, G, d)), H // G, 1)
+    v = side("v").reshape(T, H, e)
+    beta = sigmoid(linear(W[p + ".b"], h))
+    step = softplus(linear(W[p + ".a2"], linear(W[p + ".a1"], h)) + W[p + ".dt_bias"]).reshape(T, H, d)
+    g = np.exp(-np.exp(W[p + ".A_log"])[:, None] * step)
+    o = rms(recur(q, k, v, g, beta), eps) * W[p + ".norm"]
+    o = o.reshape(T, H * e) * sigmoid(linear(W[p + ".g2"], linear(W[p + ".g1"], h)))
+    return linear(W[p + ".o"], o)
+
+
+def run_kupuzen(config, weights, tokens, dtype=np.float64, layers_out=None, attention=windowed_mixer, delta=delta_mixer, ff=silu_glu):
+    """Both sublayers read the same stream through norms of their own; some attention layers read an earlier one's cache."""
+    W = {k: v.astype(dtype) for k, v in weights.items()}
+    eps, kvs = config["norm"]["eps"], {}
+    x = W["embed"][np.asarray(tokens, np.int64)] * config["embedding"]["scale"]
+    for i, L in enumerate(config["layers"]):
+        p, mix = "l%d" % i, L["mixer"]
+        h = centred_rms_norm(x, W[p + ".norm1"], eps)
+        if L["type"] == "channel_delta":
+            y = delta(h, W, p + ".mix", mix, eps)
+        else:
+            y, k, v = attention(h, W, p + ".mix", mix, eps, kvs.get(mix.get("kv_from")))
+            kvs[i] = (k, v)
+        if L["mlp"] is not None:
+            y = y + ff(centred_rms_norm(x, W[p + ".norm2"], eps), W, p + ".mlp")
+        x = x + config["residual_mult"] * y
+        if layers_out is not None:
+            layers_out.append(x.copy())
+    y = linear(W["head"], centred_rms_norm(x, W["final.norm"], eps))
+    cap = config["logit_softcap"]
+    return cap * np.tanh(y / cap)
+
+
 def layer_runs(config):
     """(layer, pass) of every layer run in order; pass is None outside the loop."""
     n, lp = len(config["layers"]), config.get("loop")
@@ -175,8 +311,13 @@ def layer_runs(config):
             + [(i, None) for i in range(lp["stop"], n)])
 
 
-def run(config, weights, tokens, dtype=np.float64, layers_out=None, mixer=attention_mixer, ff=feed_forward):
-    """Logits [T, vocab] of one sequence; the residual stream after every layer run is appended to layers_out."""
+def run(config, weights, tokens, dtype=np.float64, layers_out=None, **over):
+    """Logits [T, vocab] of one sequence; the residual stream after every layer run is appended to layers_out. `over`
+    replaces mechanisms of the design."""
+    return {"Rumalorn": run_rumalorn, "Kupuzen": run_kupuzen}[config["architecture"]](config, weights, tokens, dtype, layers_out, **over)
+
+
+def run_rumalorn(config, weights, tokens, dtype=np.float64, layers_out=None, mixer=attention_mixer, ff=feed_forward):
     W = {k: (v if v.dtype.kind in "iu" else v.astype(dtype)) for k, v in weights.items()}
     tokens = np.asarray(tokens, np.int64)
     emb = W["embed"][tokens]

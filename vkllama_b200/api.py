@@ -91,8 +91,10 @@ def load_library():
         "vkl_model_forward_rows": [vp, vp, sz, sz, vp, sz, vp],
         "vkl_model_trace_layers": [vp, vp, sz, sz, vp],
         "vkl_model_shape": [vp, C.POINTER(u32)], "vkl_model_kv_shape": [vp, u32, C.POINTER(u32)],
+        "vkl_model_cache_info": [vp, u32, C.POINTER(u32)], "vkl_model_read_state": [vp, u32, vp],
         "vkl_model_load_folder": [vp, C.c_char_p, u32, i32, pvp],
         "vkl_model_create_config": [vp, C.c_char_p, u32, i32, pvp],
+        "vkl_model_create_config_shapes": [vp, C.c_char_p, C.c_char_p, u32, i32, pvp],
         "vkl_distance_bucket": [u32, u32, u32],
         "vkl_model_generate": [vp, vp, sz, sz, vp, C.POINTER(f32), C.POINTER(f32)],
         "vkl_model_last_token": [vp, C.POINTER(u32)], "vkl_model_read_kv": [vp, u32, vp, vp], "vkl_model_write_kv": [vp, u32, vp, vp],
@@ -652,12 +654,14 @@ class Model:
         return self
 
     @classmethod
-    def from_config(cls, dev, config, maxlen, compute=BF16):
-        """The same without weights; `config` is the text of a config.json or the object it holds."""
+    def from_config(cls, dev, config, maxlen, compute=BF16, shapes=None):
+        """The same without weights; `config` is the text of a config.json or the object it holds, `shapes` (name ->
+        shape) those of the checkpoint's tensors, for designs that take sizes from them."""
         self = cls.__new__(cls)
         self.L, self.dev, self.h = load_library(), dev, vp()
         text = config if isinstance(config, str) else json.dumps(config)
-        _ck(self.L.vkl_model_create_config(dev.h, text.encode(), maxlen, compute, C.byref(self.h)))
+        head = json.dumps({k: {"shape": [int(n) for n in v]} for k, v in (shapes or {}).items()})
+        _ck(self.L.vkl_model_create_config_shapes(dev.h, text.encode(), head.encode(), maxlen, compute, C.byref(self.h)))
         self._take_shape()
         return self
 
@@ -688,12 +692,24 @@ class Model:
         return vals, ids
 
     def cache_bytes(self):
-        """Device bytes of all key (and value) caches."""
+        """Device bytes of everything that is kept of a sequence: key and value caches, recurrent states."""
         n = 0
         for layer in range(self.cfg.layers):
-            a, b, c = self.kv_shape(layer)
-            n += a * b * c * (4 if self._kv_dtype == FP32 else 2) * (1 if self.cfg.weight_dtype == BF16 else 2)
+            heads, rows, k, v, dtype, sh, sv, sk, rr, rc = self.cache_info(layer)
+            n += (heads * rows * (k + v) + rr * rc) * (4 if dtype == FP32 else 2) + 4 * sh * sv * sk
         return n
+
+    def cache_info(self, layer):
+        """(key heads, maxlen, key width, value width, dtype, state heads, rows, columns, ring rows, columns)."""
+        o = (u32 * 10)()
+        _ck(self.L.vkl_model_cache_info(self.h, layer, o))
+        return tuple(o)
+
+    def read_state(self, layer):
+        """A recurrent layer's states, fp32 [heads, value, key] with padded widths."""
+        out = np.empty(self.cache_info(layer)[5:8], np.float32)
+        _ck(self.L.vkl_model_read_state(self.h, layer, _ptr(out)))
+        return out
 
     def set_weight(self, name, dtype, data):
         a = np.ascontiguousarray(data)
@@ -736,9 +752,9 @@ class Model:
 
     def read_kv(self, layer):
         """(keys, values) as raw bits. A decoder design whose keys are its values has one cache: values are zeros."""
-        shape = self.kv_shape(layer)
-        k = np.empty(shape, np.uint32 if self._kv_dtype == FP32 else np.uint16)
-        v = np.zeros_like(k)
+        heads, rows, kw, vw, dtype = self.cache_info(layer)[:5]
+        k = np.empty((heads, rows, kw), np.uint32 if dtype == FP32 else np.uint16)
+        v = np.zeros((heads, rows, vw or kw), k.dtype)
         _ck(self.L.vkl_model_read_kv(self.h, layer, _ptr(k), _ptr(v)))
         return k, v
 

@@ -2,7 +2,8 @@
 //
 // The JSON reader takes the whole grammar that config files use; the safetensors reader maps the file and hands
 // every tensor to vkl_model_set_weight by name. An architecture is one entry of kArchitectures: its name as
-// config.json gives it and the function that turns the config into a DecoderSpec.
+// config.json gives it and the function that turns the config (and, where the config leaves a size to a tensor, the
+// tensors' shapes) into a DecoderSpec.
 #include <ctype.h>
 #include <errno.h>
 #include <fcntl.h>
@@ -13,6 +14,7 @@
 #include <sys/stat.h>
 #include <unistd.h>
 
+#include <map>
 #include <memory>
 #include <utility>
 
@@ -187,10 +189,32 @@ int get_object(const Json &o, const char *key, const Json **out) {
 }
 bool absent(const Json *j) { return !j || j->kind == Json::NUL; }
 
+// Shapes of a checkpoint's tensors, for the sizes that a config leaves to them.
+using Shapes = std::map<std::string, std::vector<uint32_t>>;
+int read_shapes(const Json &header, Shapes *out) {
+  for (const auto &t : header.fields) {
+    if (t.first == "__metadata__") continue;
+    const Json *shape = t.second.get("shape");
+    if (!shape || shape->kind != Json::ARRAY) return fail(VKL_INVALID_ARGUMENT, "model: tensor %s has no shape", t.first.c_str());
+    std::vector<uint32_t> &d = (*out)[t.first];
+    for (const Json &k : shape->items) {
+      if (k.kind != Json::NUMBER || k.num < 0 || k.num > 4294967295.0) return fail(VKL_INVALID_ARGUMENT, "model: tensor %s has a malformed shape", t.first.c_str());
+      d.push_back((uint32_t)k.num);
+    }
+  }
+  return VKL_OK;
+}
+int get_rows(const Shapes &shapes, const std::string &name, uint32_t *out) {
+  const auto it = shapes.find(name);
+  if (it == shapes.end() || it->second.size() != 2) return fail(VKL_INVALID_ARGUMENT, "model: the shape of tensor %s is needed", name.c_str());
+  *out = it->second[0];
+  return VKL_OK;
+}
+
 // -------------------------------------------------------------------------------------- Rumalorn
 // Parallel blocks under Dynamic Tanh norms; attention whose keys are its values, with a bucketed distance bias,
 // a query temperature and head gates; dense clamped or table-routed SiLU feed-forwards; a loop over some layers.
-int rumalorn_spec(const Json &c, DecoderSpec *s) {
+int rumalorn_spec(const Json &c, const Shapes &, DecoderSpec *s) {
   VKL_OKAY(get_u32(c, "vocab", &s->vocab));
   VKL_OKAY(get_u32(c, "width", &s->width));
   VKL_OKAY(get_f32(c, "logit_scale", &s->logit_scale));
@@ -251,21 +275,102 @@ int rumalorn_spec(const Json &c, DecoderSpec *s) {
   return VKL_OK;
 }
 
+// --------------------------------------------------------------------------------------- Kupuzen
+// Parallel sublayers under centred RMS norms of their own; windowed attention with sinks, normed and rotated queries
+// and keys and caches that later layers may share; a gated delta rule with a decay per key channel; dense SiLU
+// feed-forwards; scaled embedding and residual, soft-capped logits.
+int kupuzen_attention(const Json &mix, AttnSpec *a) {
+  VKL_OKAY(get_u32(mix, "heads", &a->heads));
+  VKL_OKAY(get_u32(mix, "kv_heads", &a->kv_heads));
+  VKL_OKAY(get_u32(mix, "dim", &a->dim));
+  VKL_OKAY(get_u32(mix, "vdim", &a->vdim));
+  VKL_OKAY(get_f32(mix, "scale", &a->scale));
+  if (!a->vdim) return fail(VKL_INVALID_ARGUMENT, "config: values of width 0");
+  a->qk_norm = a->sink = true;
+  const Json *mask = mix.get("mask"), *rot = mix.get("rot");
+  if (!absent(mask)) {
+    VKL_OKAY(get_u32(*mask, "size", &a->window));
+    if (!a->window) return fail(VKL_INVALID_ARGUMENT, "config: a window of 0 positions");
+  }
+  if (!absent(rot)) {
+    VKL_OKAY(get_u32(*rot, "dims", &a->rot.dims));
+    VKL_OKAY(get_number(*rot, "base", &a->rot.base));
+    const Json *sc = rot->get("scaling");
+    if (!absent(sc)) {
+      a->rot.scaled = true;
+      VKL_OKAY(get_number(*sc, "factor", &a->rot.factor));
+      VKL_OKAY(get_number(*sc, "low", &a->rot.low));
+      VKL_OKAY(get_number(*sc, "high", &a->rot.high));
+      VKL_OKAY(get_number(*sc, "original", &a->rot.original));
+    }
+  }
+  if (!absent(mix.get("kv_from"))) {
+    uint32_t j = 0;
+    VKL_OKAY(get_u32(mix, "kv_from", &j));
+    a->kv_from = (int)j;
+  }
+  return VKL_OK;
+}
+int kupuzen_spec(const Json &c, const Shapes &shapes, DecoderSpec *s) {
+  const Json *norm = nullptr, *emb = c.get("embedding"), *layers = c.get("layers");
+  VKL_OKAY(get_u32(c, "vocab", &s->vocab));
+  VKL_OKAY(get_u32(c, "width", &s->width));
+  VKL_OKAY(get_object(c, "norm", &norm));
+  VKL_OKAY(get_f32(*norm, "eps", &s->norm_eps));
+  VKL_OKAY(get_f32(c, "residual_mult", &s->residual_mult));
+  if (!absent(emb)) VKL_OKAY(get_f32(*emb, "scale", &s->embed_scale));
+  if (!absent(c.get("logit_softcap"))) VKL_OKAY(get_f32(c, "logit_softcap", &s->logit_cap));
+  s->norm = NORM_RMS_CENTRED;
+  s->two_norms = true;
+  if (absent(layers) || layers->kind != Json::ARRAY) return fail(VKL_INVALID_ARGUMENT, "config: 'layers' is missing");
+  for (const Json &j : layers->items) {
+    LayerSpec l;
+    const Json *type = j.get("type"), *mix = nullptr;
+    VKL_OKAY(get_object(j, "mixer", &mix));
+    if (type && type->str == "attention") {
+      VKL_OKAY(kupuzen_attention(*mix, &l.attn));
+    } else if (type && type->str == "channel_delta") {
+      const std::string p = "l" + std::to_string(s->layers.size()) + ".mix.";
+      l.mixer = MIX_DELTA;
+      VKL_OKAY(get_u32(*mix, "heads", &l.delta.heads));
+      VKL_OKAY(get_u32(*mix, "kv_heads", &l.delta.kv_heads));
+      VKL_OKAY(get_u32(*mix, "dim", &l.delta.dim));
+      VKL_OKAY(get_u32(*mix, "vdim", &l.delta.vdim));
+      VKL_OKAY(get_u32(*mix, "conv", &l.delta.taps));
+      VKL_OKAY(get_rows(shapes, p + "a1", &l.delta.decay_rank));
+      VKL_OKAY(get_rows(shapes, p + "g1", &l.delta.gate_rank));
+    } else {
+      return fail(VKL_UNIMPLEMENTED, "config: layer type '%s'", type ? type->str.c_str() : "");
+    }
+    const Json *mlp = j.get("mlp");
+    if (!absent(mlp)) {
+      const Json *kind = mlp->get("kind");
+      if (!kind || kind->str != "dense") return fail(VKL_UNIMPLEMENTED, "config: feed-forward kind '%s'", kind ? kind->str.c_str() : "");
+      l.ffn.kind = FFN_DENSE;
+      l.ffn.act = GLU_SILU;
+      VKL_OKAY(get_u32(*mlp, "ff", &l.ffn.ff));
+    }
+    s->layers.push_back(l);
+  }
+  return VKL_OK;
+}
+
 struct Architecture {
   const char *name;
-  int (*spec)(const Json &config, DecoderSpec *out);
+  int (*spec)(const Json &config, const Shapes &shapes, DecoderSpec *out);
 };
 const Architecture kArchitectures[] = {
     {"Rumalorn", rumalorn_spec},
+    {"Kupuzen", kupuzen_spec},
 };
 
-int spec_of(const char *text, size_t n, DecoderSpec *out) {
+int spec_of(const char *text, size_t n, const Shapes &shapes, DecoderSpec *out) {
   Json c;
   VKL_OKAY(parse_json(text, n, "config", &c));
   const Json *name = c.get("architecture");
   if (!name || name->kind != Json::STRING) return fail(VKL_INVALID_ARGUMENT, "config: 'architecture' is missing");
   for (const Architecture &a : kArchitectures)
-    if (name->str == a.name) return a.spec(c, out);
+    if (name->str == a.name) return a.spec(c, shapes, out);
   return fail(VKL_UNIMPLEMENTED, "config: architecture '%s' is not registered (%s)", name->str.c_str(), vkl_model_architectures());
 }
 
@@ -289,31 +394,46 @@ struct Mapping {
   }
 };
 
-int load_safetensors(vkl_model *m, const std::string &path) {
+// A safetensors file: its header, and every tensor by name.
+struct Safetensors {
+  std::string path;
   Mapping f;
-  VKL_OKAY(f.open_file(path));
-  uint64_t hn = 0;
-  if (f.n < 8) return fail(VKL_INVALID_ARGUMENT, "model_load: %s is too short", path.c_str());
-  memcpy(&hn, f.p, 8);
-  if (hn > f.n - 8) return fail(VKL_INVALID_ARGUMENT, "model_load: %s: the header runs past the end", path.c_str());
   Json head;
-  VKL_OKAY(parse_json((const char *)f.p + 8, (size_t)hn, path.c_str(), &head));
-  const uint8_t *data = f.p + 8 + hn;
-  const size_t left = f.n - 8 - (size_t)hn;
-  for (const auto &t : head.fields) {
-    if (t.first == "__metadata__") continue;
-    const Json *dt = t.second.get("dtype"), *off = t.second.get("data_offsets"), *shape = t.second.get("shape");
-    if (!dt || !off || !shape || off->items.size() != 2) return fail(VKL_INVALID_ARGUMENT, "model_load: %s: entry %s is malformed", path.c_str(), t.first.c_str());
-    const double a = off->items[0].num, b = off->items[1].num;
-    if (!(a >= 0 && a <= b && b <= (double)left)) return fail(VKL_OUT_OF_RANGE, "model_load: tensor %s runs past the end of %s", t.first.c_str(), path.c_str());
-    const int dtype = dt->str == "BF16" ? VKL_BF16 : dt->str == "I32" ? VKL_UINT32 : -1;
-    if (dtype < 0) return fail(VKL_UNIMPLEMENTED, "model_load: tensor %s has dtype %s (BF16 or I32)", t.first.c_str(), dt->str.c_str());
-    std::vector<uint32_t> dims;
-    for (const Json &d : shape->items) dims.push_back((uint32_t)d.num);
-    VKL_OKAY(decoder_check_shape(m, t.first.c_str(), dims));
-    VKL_OKAY(vkl_model_set_weight(m, t.first.c_str(), dtype, data + (size_t)a, (size_t)(b - a)));
+  size_t data = 0;
+  int open_file(const std::string &p) {
+    path = p;
+    VKL_OKAY(f.open_file(path));
+    uint64_t hn = 0;
+    if (f.n < 8) return fail(VKL_INVALID_ARGUMENT, "model_load: %s is too short", path.c_str());
+    memcpy(&hn, f.p, 8);
+    if (hn > f.n - 8) return fail(VKL_INVALID_ARGUMENT, "model_load: %s: the header runs past the end", path.c_str());
+    data = 8 + (size_t)hn;
+    return parse_json((const char *)f.p + 8, (size_t)hn, path.c_str(), &head);
   }
-  return VKL_OK;
+  int load(vkl_model *m) const {
+    Shapes shapes;
+    VKL_OKAY(read_shapes(head, &shapes));
+    for (const auto &t : head.fields) {
+      if (t.first == "__metadata__") continue;
+      const Json *dt = t.second.get("dtype"), *off = t.second.get("data_offsets");
+      if (!dt || !off || off->items.size() != 2) return fail(VKL_INVALID_ARGUMENT, "model_load: %s: entry %s is malformed", path.c_str(), t.first.c_str());
+      const double a = off->items[0].num, b = off->items[1].num;
+      if (!(a >= 0 && a <= b && b <= (double)(f.n - data))) return fail(VKL_OUT_OF_RANGE, "model_load: tensor %s runs past the end of %s", t.first.c_str(), path.c_str());
+      const int dtype = dt->str == "BF16" ? VKL_BF16 : dt->str == "I32" ? VKL_UINT32 : -1;
+      if (dtype < 0) return fail(VKL_UNIMPLEMENTED, "model_load: tensor %s has dtype %s (BF16 or I32)", t.first.c_str(), dt->str.c_str());
+      VKL_OKAY(decoder_check_shape(m, t.first.c_str(), shapes[t.first]));
+      VKL_OKAY(vkl_model_set_weight(m, t.first.c_str(), dtype, f.p + data + (size_t)a, (size_t)(b - a)));
+    }
+    return VKL_OK;
+  }
+};
+
+int create(vkl_device *dev, const char *config_json, const Shapes &shapes, uint32_t maxlen, int compute_dtype, vkl_model **out) {
+  if (compute_dtype != VKL_BF16 && compute_dtype != VKL_FP32) return fail(VKL_INVALID_ARGUMENT, "model_create_config: compute dtype %d (BF16 or FP32)", compute_dtype);
+  DecoderSpec s;
+  VKL_OKAY(spec_of(config_json, strlen(config_json), shapes, &s));
+  if (!dev) return fail(VKL_INVALID_ARGUMENT, "model_create_config: null device");
+  return decoder_create(dev, s, maxlen, compute_dtype == VKL_FP32, out);
 }
 
 }  // namespace
@@ -330,12 +450,18 @@ const char *vkl_model_architectures(void) {
 }
 
 int vkl_model_create_config(vkl_device *dev, const char *config_json, uint32_t maxlen, int compute_dtype, vkl_model **out) {
+  return vkl_model_create_config_shapes(dev, config_json, nullptr, maxlen, compute_dtype, out);
+}
+
+int vkl_model_create_config_shapes(vkl_device *dev, const char *config_json, const char *shapes_json, uint32_t maxlen, int compute_dtype, vkl_model **out) {
   if (!config_json || !out) return fail(VKL_INVALID_ARGUMENT, "model_create_config: null argument");
-  if (compute_dtype != VKL_BF16 && compute_dtype != VKL_FP32) return fail(VKL_INVALID_ARGUMENT, "model_create_config: compute dtype %d (BF16 or FP32)", compute_dtype);
-  DecoderSpec s;
-  VKL_OKAY(spec_of(config_json, strlen(config_json), &s));
-  if (!dev) return fail(VKL_INVALID_ARGUMENT, "model_create_config: null device");
-  return decoder_create(dev, s, maxlen, compute_dtype == VKL_FP32, out);
+  Shapes shapes;
+  if (shapes_json) {
+    Json j;
+    VKL_OKAY(parse_json(shapes_json, strlen(shapes_json), "shapes", &j));
+    VKL_OKAY(read_shapes(j, &shapes));
+  }
+  return create(dev, config_json, shapes, maxlen, compute_dtype, out);
 }
 
 int vkl_model_load_folder(vkl_device *dev, const char *path, uint32_t maxlen, int compute_dtype, vkl_model **out) {
@@ -347,9 +473,13 @@ int vkl_model_load_folder(vkl_device *dev, const char *path, uint32_t maxlen, in
     VKL_OKAY(f.open_file(dir + "/config.json"));
     text.assign((const char *)f.p, f.n);
   }
+  Safetensors f;
+  VKL_OKAY(f.open_file(dir + "/model.safetensors"));
+  Shapes shapes;
+  VKL_OKAY(read_shapes(f.head, &shapes));
   vkl_model *m = nullptr;
-  VKL_OKAY(vkl_model_create_config(dev, text.c_str(), maxlen, compute_dtype, &m));
-  int st = load_safetensors(m, dir + "/model.safetensors");
+  VKL_OKAY(create(dev, text.c_str(), shapes, maxlen, compute_dtype, &m));
+  int st = f.load(m);
   if (st == VKL_OK) st = decoder_ready(m);
   if (st != VKL_OK) {
     vkl_model_destroy(m);

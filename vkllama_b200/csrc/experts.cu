@@ -50,14 +50,14 @@ template <class T> __global__ void combine_kernel(const float *__restrict__ y, u
   for (uint32_t n = threadIdx.x; n < r.ldw; n += blockDim.x) {
     float v = 0.f;
     for (uint32_t j = 0; j < top; ++j) v += y[(size_t)slot[m * top + j] * y_ld + n];
-    finish_residual<T>(r, m, n, r.x[(size_t)m * r.ldw + n] + v);
+    finish_residual<T>(r, m, n, r.x[(size_t)m * r.ldw + n] + r.mult * v);
   }
 }
 
-template <class T> __global__ void embed_rows_kernel(const bf16 *__restrict__ emb, const uint32_t *__restrict__ toks, const Residual r) {
+template <class T> __global__ void embed_rows_kernel(const bf16 *__restrict__ emb, const uint32_t *__restrict__ toks, float scale, const Residual r) {
   const uint32_t m = blockIdx.x;
   const bf16 *e = emb + (size_t)toks[m] * r.ldw;
-  for (uint32_t n = threadIdx.x; n < r.ldw; n += blockDim.x) finish_residual<T>(r, m, n, __bfloat162float(e[n]));
+  for (uint32_t n = threadIdx.x; n < r.ldw; n += blockDim.x) finish_residual<T>(r, m, n, __bfloat162float(e[n]) * scale);
 }
 
 __global__ void pack_rows_kernel(const bf16 *__restrict__ src, uint32_t rows, uint32_t cols, bf16 *__restrict__ dst, uint32_t ld, const PackMap m) {
@@ -93,9 +93,9 @@ cudaError_t launch_combine(const float *y, uint32_t y_ld, const int32_t *slot, u
   else combine_kernel<bf16><<<T, 256, 0, s>>>(y, y_ld, slot, top, r);
   return cudaGetLastError();
 }
-cudaError_t launch_embed_rows(const bf16 *emb, const uint32_t *toks, uint32_t T, const Residual &r, bool f32, cudaStream_t s) {
-  if (f32) embed_rows_kernel<float><<<T, 256, 0, s>>>(emb, toks, r);
-  else embed_rows_kernel<bf16><<<T, 256, 0, s>>>(emb, toks, r);
+cudaError_t launch_embed_rows(const bf16 *emb, const uint32_t *toks, uint32_t T, float scale, const Residual &r, bool f32, cudaStream_t s) {
+  if (f32) embed_rows_kernel<float><<<T, 256, 0, s>>>(emb, toks, scale, r);
+  else embed_rows_kernel<bf16><<<T, 256, 0, s>>>(emb, toks, scale, r);
   return cudaGetLastError();
 }
 cudaError_t launch_pack_rows(const bf16 *src, uint32_t rows, uint32_t cols, bf16 *dst, uint32_t ld, const PackMap &m, cudaStream_t s) {

@@ -19,7 +19,7 @@ __global__ void __launch_bounds__(128) gemm_f32_kernel(const GemmRows p) {
     if (e < 0) return;
     w0 += (size_t)e * p.N;
   }
-  const float *a = static_cast<const float *>(p.a);
+  const float *a = static_cast<const float *>(p.a) + (p.n2 && n0 >= p.n2 ? (size_t)p.M * p.K : 0);
   float acc[32];
 #pragma unroll
   for (int i = 0; i < 32; ++i) acc[i] = 0.f;
@@ -52,7 +52,7 @@ __global__ void __launch_bounds__(128) gemm_f32_kernel(const GemmRows p) {
 }  // namespace
 
 cudaError_t launch_gemm_rows_f32(const GemmRows &p, cudaStream_t s) {
-  if (!p.M || !p.N || p.N % 32 || p.K % 64) return cudaErrorInvalidValue;
+  if (!p.M || !p.N || p.N % 32 || p.K % 64 || p.n2 % kInputAlign) return cudaErrorInvalidValue;
   gemm_f32_kernel<<<dim3((p.M + TM - 1) / TM, (p.N + TN - 1) / TN), 128, 0, s>>>(p);
   return cudaGetLastError();
 }

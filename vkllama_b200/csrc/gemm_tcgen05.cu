@@ -224,8 +224,9 @@ __global__ void __launch_bounds__(KIND == GK_Q8 ? GEMM_THREADS_Q8 : GEMM_THREADS
   const uint32_t warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const uint32_t m0 = blockIdx.x * BM, n0 = blockIdx.y * BN;
   const uint32_t nkb = p.K / BK;
-  uint32_t w_row = n0;  // first weight row of the tile
+  uint32_t w_row = n0, a_row = m0;  // first weight and input row of the tile
   if constexpr (KIND == GK_ROWS) {
+    if (p.n2 && n0 >= p.n2) a_row += p.M;  // rows beyond an input's M are read (the next one's, or zeros) and dropped by the epilogue
     if (p.tile_expert) {
       const int32_t e = p.tile_expert[blockIdx.x];
       if (e < 0) return;  // uniform over the CTA
@@ -273,7 +274,7 @@ __global__ void __launch_bounds__(KIND == GK_Q8 ? GEMM_THREADS_Q8 : GEMM_THREADS
 #endif
         asm volatile("mbarrier.arrive.expect_tx.shared::cta.b64 _, [%0], %1;" ::"r"(bar), "r"(Q8 ? A_TILE_BYTES : C::STAGE_BYTES) : "memory");
         unsigned char *st = stages + (size_t)s * C::STAGE_BYTES;
-        tma_load_2d(sa(st), &map_a, kb * BK, m0, bar);
+        tma_load_2d(sa(st), &map_a, kb * BK, a_row, bar);
         if (!Q8) tma_load_2d(sa(st + A_TILE_BYTES), &map_w, kb * BK, w_row, bar);
       }
     }
@@ -534,7 +535,9 @@ bool make_map(CUtensorMap *map, const void *base, uint32_t rows, uint32_t K, uin
 template <int BN, int KIND> cudaError_t launch_bn(const typename GemmArgs<KIND>::Type &p, cudaStream_t s, uint32_t w_rows) {
   constexpr bool Q8 = KIND == GK_Q8;
   CUtensorMap ma, mw;
-  if (!make_map(&ma, p.a, p.M, p.K, BM, KIND == GK_ROWS)) return cudaErrorInvalidValue;
+  uint32_t a_rows = p.M;
+  if constexpr (KIND == GK_ROWS) a_rows *= p.n2 ? 2 : 1;
+  if (!make_map(&ma, p.a, a_rows, p.K, BM, KIND == GK_ROWS)) return cudaErrorInvalidValue;
   if constexpr (Q8) {
     mw = ma;  // unused: the W tile is written by the dequantising warps
   } else if (!make_map(&mw, p.w, w_rows, p.K, BN, KIND == GK_ROWS)) {
@@ -603,7 +606,7 @@ cudaError_t launch_gemm_q8_tcgen05(const GemmParams &p, cudaStream_t s) {
 }
 
 cudaError_t launch_gemm_rows_bf16(const GemmRows &p, cudaStream_t s) {
-  if (!gemm_tcgen05_supported(p.M, p.N, p.K) || p.N % 32 || (p.tile_expert && p.M % BM)) return cudaErrorInvalidValue;
+  if (!gemm_tcgen05_supported(p.M, p.N, p.K) || p.N % 32 || (p.tile_expert && (p.M % BM || p.n2)) || p.n2 % kInputAlign) return cudaErrorInvalidValue;
   if ((reinterpret_cast<uintptr_t>(p.a) | reinterpret_cast<uintptr_t>(p.w)) & 15) return cudaErrorMisalignedAddress;
   // grouped: a tile's weight rows beyond its expert's N are read (the next expert's, or zeros) and dropped by the epilogue
   const uint32_t w_rows = p.tile_expert ? p.w_rows : p.N;

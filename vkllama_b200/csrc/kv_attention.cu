@@ -1,14 +1,15 @@
-// Causal attention over a cache in which one row per key head is both key and value, grouped queries, no
-// rotation: a position enters as a temperature of its query and as a bias by distance; a gate per head scales
-// the output. Scores, softmax and accumulation are fp32 (scores in units of log2).
+// Causal attention over a cache with grouped queries, of keys and values or of rows that are both, optionally only
+// over the last `window` positions. A position may also enter as a temperature of its query and as a bias by
+// distance (rotations are in the cache already); a head may have a sink in its denominator and a gate on its
+// output. Scores, softmax and accumulation are fp32 (scores in units of log2).
 //
 // row kernel   one token (decode), few tokens, and every call of the 32-bit mode. A CTA takes a query row, a
 //              key head and a range of the cache, and up to four of the head's query heads: every cache row is
-//              read once, and the registers that held it for the score are added to the outputs. Ranges are
-//              merged by the CTA that finishes last.
+//              read once (where the keys are the values, the registers that held a row for the score are added
+//              to the outputs). Ranges are merged by the CTA that finishes last.
 // tile kernel  64 query rows of a head per CTA on mma.sync m16n8k16 (bf16, fp32 accumulate): a 64-row cache tile
-//              is copied to shared memory once (cp.async, double buffered) and serves Q.K^T directly and P.K
-//              through transposing loads. The 127 biases that a tile pair can need travel with the tile.
+//              is copied to shared memory once (cp.async, double buffered) and serves Q.K^T directly; it, or the
+//              value tile beside it, serves P.V through transposing loads. The 127 biases that a tile pair can need travel with the tile.
 #include <algorithm>
 
 #include "rows.cuh"
@@ -26,6 +27,10 @@ __device__ __forceinline__ float query_scale(const KvAttn &p, uint32_t pos) {
 __device__ __forceinline__ float bias_at(const KvAttn &p, uint32_t h, uint32_t n) {
   return p.bias ? p.bias[(size_t)h * p.bias_n + min(n, p.bias_n - 1)] : 0.f;
 }
+
+// First position that a query at `pos` sees.
+__device__ __forceinline__ uint32_t first_seen(const KvAttn &p, uint32_t pos) { return p.window && pos >= p.window ? pos + 1 - p.window : 0u; }
+__device__ __forceinline__ float sink_log2(const KvAttn &p, uint32_t h) { return p.sink ? p.sink[h] * kLog2e : -INFINITY; }
 
 constexpr int kRowThreads = 128;
 constexpr uint32_t kMaxSplits = 32, kSplitRows = 64;  // a split holds about this many cache rows: a short cache uses fewer splits
@@ -47,23 +52,24 @@ template <> struct Raw8<float> {
   }
 };
 
-// LPR lanes hold one cache row (8 values each), NQ query heads per CTA. grid (kv heads x head groups, rows, splits)
-template <class T, int LPR, int NQ> __global__ void __launch_bounds__(kRowThreads) kv_row_kernel(const KvAttn p) {
-  constexpr uint32_t NS = kRowThreads / LPR, U = 4, DMAX = LPR * 8;
+// LPR lanes hold one cache row (8 values each), NQ query heads per CTA, SEP: values in a cache of their own.
+// grid (kv heads x head groups, rows, splits)
+template <class T, int LPR, int NQ, bool SEP> __global__ void __launch_bounds__(kRowThreads) kv_row_kernel(const KvAttn p) {
+  constexpr uint32_t NS = kRowThreads / LPR, U = SEP && sizeof(T) == 4 ? 2 : 4, DMAX = LPR * 8;
   __shared__ float sm_o[kRowThreads / 32][NQ][DMAX], sm_m[kRowThreads / 32][NQ], sm_l[kRowThreads / 32][NQ];
   __shared__ float sm_pm[kMaxSplits][NQ], sm_pl[kMaxSplits][NQ];
   __shared__ uint32_t last_s;
   const uint32_t per = p.heads / p.kv_heads, groups = (per + NQ - 1) / NQ;
   const uint32_t g = blockIdx.x / groups, hg = blockIdx.x % groups, h0 = g * per + hg * NQ, nh = min((uint32_t)NQ, per - hg * NQ);
   const uint32_t m = blockIdx.y, split = blockIdx.z, tid = threadIdx.x, sub = tid / LPR, l = tid % LPR, e0 = l * 8, warp = tid >> 5;
-  const bool ev = e0 < p.dp;
+  const bool ev = e0 < p.dp, vv = SEP && e0 < p.vp;
   if (p.use_pdl) asm volatile("griddepcontrol.wait;" ::: "memory");
-  const uint32_t pos = *p.pos + m, vis = pos + 1;
-  const uint32_t splits = min(p.splits, (vis + kSplitRows - 1) / kSplitRows);
+  const uint32_t pos = *p.pos + m, vis = pos + 1, lo = first_seen(p, pos);
+  const uint32_t splits = min(p.splits, (vis - lo + kSplitRows - 1) / kSplitRows);
   if (split >= splits) return;
-  uint32_t chunk = (vis + splits - 1) / splits;
+  uint32_t chunk = (vis - lo + splits - 1) / splits;
   chunk = (chunk + 31) & ~31u;
-  const uint32_t c0 = min(split * chunk, vis), c1 = min(c0 + chunk, vis);
+  const uint32_t c0 = min(lo + split * chunk, vis), c1 = min(c0 + chunk, vis);
   const float qs = query_scale(p, pos);
 
   float q[NQ][8], acc[NQ][8], mx[NQ], sum[NQ];
@@ -81,13 +87,17 @@ template <class T, int LPR, int NQ> __global__ void __launch_bounds__(kRowThread
     sum[i] = 0.f;
   }
   const T *base = static_cast<const T *>(p.cache) + (size_t)g * p.maxlen * p.dp + e0;
+  const T *vbase = SEP ? static_cast<const T *>(p.vcache) + (size_t)g * p.maxlen * p.vp + e0 : nullptr;
   for (uint32_t jb = c0; jb < c1; jb += NS * U) {  // the same trip count for every thread
-    Raw8<T> kr[U];
+    Raw8<T> kr[U], vr[SEP ? U : 1];
     float s[U][NQ];
 #pragma unroll
     for (int u = 0; u < U; ++u) {
       const uint32_t j = jb + u * NS + sub;
       if (ev && j < c1) kr[u].load(base + (size_t)j * p.dp);
+      if constexpr (SEP) {
+        if (vv && j < c1) vr[u].load(vbase + (size_t)j * p.vp);
+      }
 #pragma unroll
       for (int i = 0; i < NQ; ++i) s[u][i] = (j < c1 && i < nh) ? bias_at(p, h0 + i, pos - j) : -INFINITY;
     }
@@ -123,12 +133,13 @@ template <class T, int LPR, int NQ> __global__ void __launch_bounds__(kRowThread
     }
 #pragma unroll
     for (int u = 0; u < U; ++u) {
-      float k[8];
-      kr[u].get(k);
+      float v[8];
+      if constexpr (SEP) vr[u].get(v);
+      else kr[u].get(v);
 #pragma unroll
       for (int i = 0; i < NQ; ++i)
 #pragma unroll
-        for (int e = 0; e < 8; ++e) acc[i][e] = fmaf(s[u][i], k[e], acc[i][e]);
+        for (int e = 0; e < 8; ++e) acc[i][e] = fmaf(s[u][i], v[e], acc[i][e]);
     }
   }
   // merge the warp's row streams, then the warps, in a fixed order
@@ -155,19 +166,20 @@ template <class T, int LPR, int NQ> __global__ void __launch_bounds__(kRowThread
   __syncthreads();
   if (p.use_pdl) asm volatile("griddepcontrol.launch_dependents;");
   const size_t unit = (size_t)m * gridDim.x + blockIdx.x;
-  const uint32_t rec = p.dp + 4;
-  float *part = p.scratch + unit * p.splits * NQ * rec;  // [split][NQ][dp + 4]: output, max, sum
+  const uint32_t rec = p.vp + 4;
+  float *part = p.scratch + unit * p.splits * NQ * rec;  // [split][NQ][vp + 4]: output, max, sum
   auto write = [&](uint32_t i, uint32_t d, float v) {
     if (p.gate) v *= p.gate[(size_t)m * p.gate_ld + h0 + i];
-    store1(static_cast<T *>(p.out) + (size_t)m * p.out_ld + (size_t)(h0 + i) * p.dp + d, v);
+    store1(static_cast<T *>(p.out) + (size_t)m * p.out_ld + (size_t)(h0 + i) * p.vp + d, v);
   };
-  for (uint32_t x = tid; x < nh * p.dp; x += kRowThreads) {
-    const uint32_t i = x / p.dp, d = x % p.dp;
-    float M = -INFINITY;
+  for (uint32_t x = tid; x < nh * p.vp; x += kRowThreads) {
+    const uint32_t i = x / p.vp, d = x % p.vp;
+    const float sink = splits == 1 ? sink_log2(p, h0 + i) : -INFINITY;  // counts once: here, or in the merge
+    float M = sink;
 #pragma unroll
     for (int w = 0; w < kRowThreads / 32; ++w) M = fmaxf(M, sm_m[w][i]);
     const float ref = M == -INFINITY ? 0.f : M;
-    float num = 0.f, den = 0.f;
+    float num = 0.f, den = exp2f(sink - ref);
 #pragma unroll
     for (int w = 0; w < kRowThreads / 32; ++w) {
       const float c = exp2f(sm_m[w][i] - ref);
@@ -180,8 +192,8 @@ template <class T, int LPR, int NQ> __global__ void __launch_bounds__(kRowThread
       float *r = part + ((size_t)split * NQ + i) * rec;
       r[d] = num;
       if (d == 0) {
-        r[p.dp] = M;
-        r[p.dp + 1] = den;
+        r[p.vp] = M;
+        r[p.vp + 1] = den;
       }
     }
   }
@@ -193,17 +205,18 @@ template <class T, int LPR, int NQ> __global__ void __launch_bounds__(kRowThread
   if (!last_s) return;
   __threadfence();
   for (uint32_t x = tid; x < splits * nh; x += kRowThreads) {
-    const float *r = part + ((size_t)(x / nh) * NQ + x % nh) * rec + p.dp;
+    const float *r = part + ((size_t)(x / nh) * NQ + x % nh) * rec + p.vp;
     sm_pm[x / nh][x % nh] = __ldcg(r);
     sm_pl[x / nh][x % nh] = __ldcg(r + 1);
   }
   __syncthreads();
-  for (uint32_t x = tid; x < nh * (p.dp / 4); x += kRowThreads) {
-    const uint32_t i = x / (p.dp / 4), d = x % (p.dp / 4) * 4;
-    float M = -INFINITY;  // split 0 is never empty: M becomes finite
+  for (uint32_t x = tid; x < nh * (p.vp / 4); x += kRowThreads) {
+    const uint32_t i = x / (p.vp / 4), d = x % (p.vp / 4) * 4;
+    const float sink = sink_log2(p, h0 + i);
+    float M = sink;  // split 0 is never empty: M becomes finite
     for (uint32_t s = 0; s < splits; ++s) M = fmaxf(M, sm_pm[s][i]);
     float4 num = make_float4(0.f, 0.f, 0.f, 0.f);
-    float den = 0.f;
+    float den = exp2f(sink - M);
 #pragma unroll 8
     for (uint32_t s = 0; s < splits; ++s) {
       const float c = exp2f(sm_pm[s][i] - M);
@@ -222,9 +235,9 @@ template <class T, int LPR, int NQ> __global__ void __launch_bounds__(kRowThread
   if (tid == 0) p.counters[unit] = 0;
 }
 
-template <class T, int LPR> cudaError_t launch_row(const KvAttn &p, cudaStream_t s) {
+template <class T, int LPR, bool SEP> cudaError_t launch_row(const KvAttn &p, cudaStream_t s) {
   const uint32_t per = p.heads / p.kv_heads;
-  auto kern = per >= 3 ? kv_row_kernel<T, LPR, 4> : per == 2 ? kv_row_kernel<T, LPR, 2> : kv_row_kernel<T, LPR, 1>;
+  auto kern = per >= 3 ? kv_row_kernel<T, LPR, 4, SEP> : per == 2 ? kv_row_kernel<T, LPR, 2, SEP> : kv_row_kernel<T, LPR, 1, SEP>;
   const uint32_t nq = per >= 3 ? 4 : per;
   cudaLaunchConfig_t cfg = {};
   cfg.gridDim = dim3(p.kv_heads * ((per + nq - 1) / nq), p.T, p.splits);
@@ -237,10 +250,11 @@ template <class T, int LPR> cudaError_t launch_row(const KvAttn &p, cudaStream_t
   cfg.numAttrs = p.use_pdl ? 1 : 0;
   return cudaLaunchKernelEx(&cfg, kern, p);
 }
-template <class T> cudaError_t launch_row_d(const KvAttn &p, cudaStream_t s) {
-  if (p.dp <= 64) return launch_row<T, 8>(p, s);
-  if (p.dp <= 128) return launch_row<T, 16>(p, s);
-  return launch_row<T, 32>(p, s);
+template <class T, bool SEP> cudaError_t launch_row_d(const KvAttn &p, cudaStream_t s) {
+  const uint32_t d = std::max(p.dp, p.vp);
+  if (d <= 64) return launch_row<T, 8, SEP>(p, s);
+  if (d <= 128) return launch_row<T, 16, SEP>(p, s);
+  return launch_row<T, 32, SEP>(p, s);
 }
 
 // ------------------------------------------------------------------------------------------ tiles
@@ -257,28 +271,37 @@ __device__ __forceinline__ void cp_async4(void *dst, const void *src) {
 }
 
 constexpr int QT = 64, KT = 64;
-template <int D> struct TileSmem {
+template <int D, bool SEP> struct TileSmem {
   static constexpr int LD = D + 8;  // padded rows: conflict-free fragment loads
   bf16 q[QT * LD];
   bf16 k[2][KT * LD];
+  bf16 v[SEP ? 2 : 1][SEP ? KT * LD : 8];
   float bias[2][128];
 };
 
-// D: head width rounded up to what is instantiated; dp the width in memory.
-template <int D> __global__ void __launch_bounds__(128) kv_tile_kernel(const KvAttn p) {
-  constexpr int LD = TileSmem<D>::LD;
+// D: the wider of key and value rounded up to what is instantiated; dp, vp the widths in memory.
+template <int D, bool SEP> __global__ void __launch_bounds__(128) kv_tile_kernel(const KvAttn p) {
+  constexpr int LD = TileSmem<D, SEP>::LD;
   extern __shared__ __align__(16) unsigned char raw[];
-  TileSmem<D> &sm = *reinterpret_cast<TileSmem<D> *>(raw);
+  TileSmem<D, SEP> &sm = *reinterpret_cast<TileSmem<D, SEP> *>(raw);
   const uint32_t h = blockIdx.x, g = h / (p.heads / p.kv_heads), tiles = gridDim.y, m0 = (tiles - 1 - blockIdx.y) * QT;  // longest rows first
   const uint32_t tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, gq = lane >> 2, t = lane & 3;
   const uint32_t T = p.T, pos0 = *p.pos, vecs = p.dp / 8;
   const bf16 *cache = static_cast<const bf16 *>(p.cache) + (size_t)g * p.maxlen * p.dp;
-  const uint32_t jmax = pos0 + min(m0 + QT, T);  // cache rows that some row of the tile sees
+  const uint32_t jmax = pos0 + min(m0 + QT, T), jmin = first_seen(p, pos0 + m0) / KT * KT;  // cache rows that some row of the tile sees
   auto fetch = [&](uint32_t j0, uint32_t b) {
     for (uint32_t i = tid; i < KT * (D / 8); i += 128) {
       const uint32_t r = i / (D / 8), c = i % (D / 8);
       const bool ok = j0 + r < jmax && c < vecs;
       cp_async16(&sm.k[b][r * LD + c * 8], cache + (ok ? (size_t)(j0 + r) * p.dp + c * 8 : 0), ok);
+    }
+    if constexpr (SEP) {
+      const bf16 *vc = static_cast<const bf16 *>(p.vcache) + (size_t)g * p.maxlen * p.vp;
+      for (uint32_t i = tid; i < KT * (D / 8); i += 128) {
+        const uint32_t r = i / (D / 8), c = i % (D / 8);
+        const bool ok = j0 + r < jmax && c < p.vp / 8;
+        cp_async16(&sm.v[b][r * LD + c * 8], vc + (ok ? (size_t)(j0 + r) * p.vp + c * 8 : 0), ok);
+      }
     }
     if (p.bias && tid < 127) {  // distance of (row r, column c): pos0 + m0 + r - j0 - c = entry r - c + 63
       const int n = (int)(pos0 + m0) - (int)j0 + (int)tid - 63;
@@ -293,9 +316,10 @@ template <int D> __global__ void __launch_bounds__(128) kv_tile_kernel(const KvA
   }
   if (!p.bias)
     for (uint32_t i = tid; i < 256; i += 128) sm.bias[i >> 7][i & 127] = 0.f;
-  fetch(0, 0);
+  fetch(jmin, 0);
   const uint32_t rl = warp * 16 + gq, rh = rl + 8;                                       // rows in the tile
   const uint32_t vis_lo = m0 + rl < T ? pos0 + m0 + rl + 1 : 0u, vis_hi = m0 + rh < T ? pos0 + m0 + rh + 1 : 0u;
+  const uint32_t see_lo = first_seen(p, pos0 + m0 + rl), see_hi = first_seen(p, pos0 + m0 + rh);
   const float qs_lo = query_scale(p, pos0 + m0 + rl), qs_hi = query_scale(p, pos0 + m0 + rh);
   float o[D / 8][4];
 #pragma unroll
@@ -303,7 +327,7 @@ template <int D> __global__ void __launch_bounds__(128) kv_tile_kernel(const KvA
   float mx_lo = -INFINITY, mx_hi = -INFINITY, l_lo = 0.f, l_hi = 0.f;
   const bf16 *qw = sm.q + rl * LD + 2 * t;
   uint32_t b = 0;
-  for (uint32_t j0 = 0; j0 < jmax; j0 += KT, b ^= 1) {
+  for (uint32_t j0 = jmin; j0 < jmax; j0 += KT, b ^= 1) {
     asm volatile("cp.async.wait_group 0;" ::: "memory");
     __syncthreads();  // tile b has landed for everyone, tile b ^ 1 is consumed
     if (j0 + KT < jmax) fetch(j0 + KT, b ^ 1);
@@ -327,10 +351,10 @@ template <int D> __global__ void __launch_bounds__(128) kv_tile_kernel(const KvA
     for (int nt = 0; nt < KT / 8; ++nt) {
       const int c = nt * 8 + 2 * t;
       const uint32_t j = j0 + c;
-      sc[nt][0] = j < vis_lo ? fmaf(sc[nt][0], qs_lo, bs[(int)rl - c]) : -INFINITY;
-      sc[nt][1] = j + 1 < vis_lo ? fmaf(sc[nt][1], qs_lo, bs[(int)rl - c - 1]) : -INFINITY;
-      sc[nt][2] = j < vis_hi ? fmaf(sc[nt][2], qs_hi, bs[(int)rh - c]) : -INFINITY;
-      sc[nt][3] = j + 1 < vis_hi ? fmaf(sc[nt][3], qs_hi, bs[(int)rh - c - 1]) : -INFINITY;
+      sc[nt][0] = j < vis_lo && j >= see_lo ? fmaf(sc[nt][0], qs_lo, bs[(int)rl - c]) : -INFINITY;
+      sc[nt][1] = j + 1 < vis_lo && j + 1 >= see_lo ? fmaf(sc[nt][1], qs_lo, bs[(int)rl - c - 1]) : -INFINITY;
+      sc[nt][2] = j < vis_hi && j >= see_hi ? fmaf(sc[nt][2], qs_hi, bs[(int)rh - c]) : -INFINITY;
+      sc[nt][3] = j + 1 < vis_hi && j + 1 >= see_hi ? fmaf(sc[nt][3], qs_hi, bs[(int)rh - c - 1]) : -INFINITY;
       tm_lo = fmaxf(tm_lo, fmaxf(sc[nt][0], sc[nt][1]));
       tm_hi = fmaxf(tm_hi, fmaxf(sc[nt][2], sc[nt][3]));
     }
@@ -367,7 +391,7 @@ template <int D> __global__ void __launch_bounds__(128) kv_tile_kernel(const KvA
     for (int j16 = 0; j16 < KT / 16; ++j16) {
       const uint32_t a0 = pack_bf2(sc[2 * j16][0], sc[2 * j16][1]), a1 = pack_bf2(sc[2 * j16][2], sc[2 * j16][3]);
       const uint32_t a2 = pack_bf2(sc[2 * j16 + 1][0], sc[2 * j16 + 1][1]), a3 = pack_bf2(sc[2 * j16 + 1][2], sc[2 * j16 + 1][3]);
-      const bf16 *vrow = ks + (j16 * 16 + (lane & 7) + ((lane >> 3) & 1) * 8) * LD + ((lane >> 4) & 1) * 8;
+      const bf16 *vrow = (SEP ? sm.v[b] : ks) + (j16 * 16 + (lane & 7) + ((lane >> 3) & 1) * 8) * LD + ((lane >> 4) & 1) * 8;
 #pragma unroll
       for (int dt = 0; dt < D / 16; ++dt) {
         uint32_t b0, b1, b2, b3;
@@ -384,47 +408,59 @@ template <int D> __global__ void __launch_bounds__(128) kv_tile_kernel(const KvA
     l_hi += __shfl_xor_sync(0xffffffffu, l_hi, w);
   }
   const uint32_t ml = m0 + rl, mh = m0 + rh;
-  const float f_lo = ml < T ? (p.gate ? p.gate[(size_t)ml * p.gate_ld + h] : 1.f) / l_lo : 0.f;
-  const float f_hi = mh < T ? (p.gate ? p.gate[(size_t)mh * p.gate_ld + h] : 1.f) / l_hi : 0.f;
-  bf16 *out = static_cast<bf16 *>(p.out) + (size_t)h * p.dp;
+  float k_lo = 1.f, k_hi = 1.f;  // the sink may be the largest term: the outputs are rescaled to it
+  if (p.sink) {
+    const float sink = sink_log2(p, h), M_lo = fmaxf(mx_lo, sink), M_hi = fmaxf(mx_hi, sink);
+    k_lo = exp2f(mx_lo - M_lo);
+    k_hi = exp2f(mx_hi - M_hi);
+    l_lo = l_lo * k_lo + exp2f(sink - M_lo);
+    l_hi = l_hi * k_hi + exp2f(sink - M_hi);
+  }
+  const float f_lo = ml < T ? (p.gate ? p.gate[(size_t)ml * p.gate_ld + h] : 1.f) * k_lo / l_lo : 0.f;
+  const float f_hi = mh < T ? (p.gate ? p.gate[(size_t)mh * p.gate_ld + h] : 1.f) * k_hi / l_hi : 0.f;
+  bf16 *out = static_cast<bf16 *>(p.out) + (size_t)h * p.vp;
 #pragma unroll
   for (int nt = 0; nt < D / 8; ++nt) {
     const uint32_t d = nt * 8 + 2 * t;
-    if (d >= p.dp) continue;
+    if (d >= p.vp) continue;
     if (ml < T) *reinterpret_cast<uint32_t *>(out + (size_t)ml * p.out_ld + d) = pack_bf2(o[nt][0] * f_lo, o[nt][1] * f_lo);
     if (mh < T) *reinterpret_cast<uint32_t *>(out + (size_t)mh * p.out_ld + d) = pack_bf2(o[nt][2] * f_hi, o[nt][3] * f_hi);
   }
 }
 
-template <int D> cudaError_t launch_tile(const KvAttn &p, cudaStream_t s) {
-  cudaError_t e = cudaFuncSetAttribute(kv_tile_kernel<D>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)sizeof(TileSmem<D>));
+template <int D, bool SEP> cudaError_t launch_tile(const KvAttn &p, cudaStream_t s) {
+  cudaError_t e = cudaFuncSetAttribute(kv_tile_kernel<D, SEP>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)sizeof(TileSmem<D, SEP>));
   if (e != cudaSuccess) return e;
-  kv_tile_kernel<D><<<dim3(p.heads, (p.T + QT - 1) / QT), 128, sizeof(TileSmem<D>), s>>>(p);
+  kv_tile_kernel<D, SEP><<<dim3(p.heads, (p.T + QT - 1) / QT), 128, sizeof(TileSmem<D, SEP>), s>>>(p);
   return cudaGetLastError();
+}
+template <bool SEP> cudaError_t launch_tile_d(const KvAttn &p, cudaStream_t s) {
+  const uint32_t d = std::max(p.dp, p.vp);
+  if (d <= 32) return launch_tile<32, SEP>(p, s);
+  if (d <= 48) return launch_tile<48, SEP>(p, s);
+  if (d <= 64) return launch_tile<64, SEP>(p, s);
+  if (d <= 96) return launch_tile<96, SEP>(p, s);
+  if (d <= 128) return launch_tile<128, SEP>(p, s);
+  if (d <= 192) return launch_tile<192, SEP>(p, s);
+  return launch_tile<256, SEP>(p, s);
 }
 
 constexpr uint32_t kTileRows = 16;  // from this many query rows the tile kernel is used
 
 }  // namespace
 
-size_t kv_attn_scratch_bytes(uint32_t T, uint32_t heads, uint32_t dp, uint32_t splits) {
-  return splits < 2 ? 0 : (size_t)T * heads * 4 * splits * (dp + 4) * sizeof(float);  // at most heads (group) units of four records
+size_t kv_attn_scratch_bytes(uint32_t T, uint32_t heads, uint32_t vp, uint32_t splits) {
+  return splits < 2 ? 0 : (size_t)T * heads * 4 * splits * (vp + 4) * sizeof(float);  // at most heads (group) units of four records
 }
 uint32_t kv_attn_counters(uint32_t T, uint32_t heads) { return T * heads; }
 
 cudaError_t launch_kv_attention(const KvAttn &p, bool f32, cudaStream_t s) {
-  if (!p.T || !p.kv_heads || p.heads % p.kv_heads || p.dp % 16 || p.dp > 256 || !p.splits || p.splits > kMaxSplits) return cudaErrorInvalidValue;
-  if (!f32 && p.T >= kTileRows) {
-    if (p.dp <= 32) return launch_tile<32>(p, s);
-    if (p.dp <= 48) return launch_tile<48>(p, s);
-    if (p.dp <= 64) return launch_tile<64>(p, s);
-    if (p.dp <= 96) return launch_tile<96>(p, s);
-    if (p.dp <= 128) return launch_tile<128>(p, s);
-    if (p.dp <= 192) return launch_tile<192>(p, s);
-    return launch_tile<256>(p, s);
-  }
+  if (!p.T || !p.kv_heads || p.heads % p.kv_heads || p.dp % 16 || p.dp > 256 || p.vp % 16 || p.vp > 256 || (!p.vcache && p.vp != p.dp) || !p.splits || p.splits > kMaxSplits)
+    return cudaErrorInvalidValue;
+  if (!f32 && p.T >= kTileRows) return p.vcache ? launch_tile_d<true>(p, s) : launch_tile_d<false>(p, s);
   if (p.T > 65535) return cudaErrorInvalidValue;
-  return f32 ? launch_row_d<float>(p, s) : launch_row_d<bf16>(p, s);
+  if (p.vcache) return f32 ? launch_row_d<float, true>(p, s) : launch_row_d<bf16, true>(p, s);
+  return f32 ? launch_row_d<float, false>(p, s) : launch_row_d<bf16, false>(p, s);
 }
 
 }  // namespace vkl

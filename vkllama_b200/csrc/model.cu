@@ -957,6 +957,7 @@ int vkl_model_forward(vkl_model *m, const uint32_t *toks, size_t n, size_t offse
     return fail(VKL_OUT_OF_RANGE, "model_forward: position %zu is beyond %s", offset + n, m->dec ? "the context length" : "the RoPE table (2*maxlen)");
   VKL_OKAY(check_ids(m, toks, n));
   VKL_CUDA(cudaSetDevice(m->dev->ordinal));
+  if (m->dec) VKL_OKAY(decoder_begin(m, offset));
   VKL_OKAY(ensure_rows(m, (uint32_t)n));
   if (n == 1 || m->cfg.tp_size > 1) VKL_OKAY(prepare_decode(m));
   if (n > 1 && m->cfg.tp_size > 1) {
@@ -1010,6 +1011,7 @@ int vkl_model_forward(vkl_model *m, const uint32_t *toks, size_t n, size_t offse
     memcpy(logits_out, m->pin, lb);
     if (*errw) VKL_OKAY(check_mega(m));  // (reads the word again, resets the kernel's state, reports)
     VKL_OKAY(check_gemm(m));
+    if (m->dec) decoder_end(m, offset + 1);
     return VKL_OK;
   }
   VKL_CUDA(cudaMemsetAsync((uint32_t *)m->state->data() + 5, 0, 4, m->stream));
@@ -1025,6 +1027,7 @@ int vkl_model_forward(vkl_model *m, const uint32_t *toks, size_t n, size_t offse
   VKL_CUDA(cudaStreamSynchronize(m->stream));
   if (n == 1) VKL_OKAY(check_mega(m));
   VKL_OKAY(check_gemm(m));
+  if (m->dec) decoder_end(m, offset + n);
   return VKL_OK;
 }
 
@@ -1060,6 +1063,7 @@ int vkl_model_trace_layers(vkl_model *m, const uint32_t *toks, size_t n, size_t 
   VKL_OKAY(check_ids(m, toks, n));
   VKL_CUDA(cudaSetDevice(m->dev->ordinal));
   Decoder *d = m->dec.get();
+  VKL_OKAY(decoder_begin(m, offset));
   VKL_OKAY(ensure_rows(m, (uint32_t)n));
   const size_t R = d->runs.size();
   VKL_OKAY(ensure_tensor(m->dev, &d->trace, R, n, d->ldw, VKL_FP32));
@@ -1072,7 +1076,9 @@ int vkl_model_trace_layers(vkl_model *m, const uint32_t *toks, size_t n, size_t 
   VKL_OKAY(rc);
   VKL_CUDA(cudaMemcpy2DAsync(out, (size_t)m->cfg.dim * 4, d->trace->data(), (size_t)d->ldw * 4, (size_t)m->cfg.dim * 4, R * n, cudaMemcpyDeviceToHost, m->stream));
   VKL_CUDA(cudaStreamSynchronize(m->stream));
-  return check_gemm(m);
+  VKL_OKAY(check_gemm(m));
+  decoder_end(m, offset + n);
+  return VKL_OK;
 }
 
 int vkl_model_shape(const vkl_model *m, uint32_t out6[6]) {
@@ -1089,10 +1095,46 @@ int vkl_model_shape(const vkl_model *m, uint32_t out6[6]) {
 int vkl_model_kv_shape(const vkl_model *m, uint32_t layer, uint32_t out4[4]) {
   if (!m || !out4 || layer >= m->cfg.layers) return fail(VKL_INVALID_ARGUMENT, "model_kv_shape: bad model or layer");
   const vkl_tensor *k = m->L[layer].kcache;
+  if (!k) {
+    memset(out4, 0, 4 * sizeof(uint32_t));
+    return VKL_OK;
+  }
   out4[0] = (uint32_t)k->c;
   out4[1] = (uint32_t)k->h;
   out4[2] = (uint32_t)k->w;
   out4[3] = (uint32_t)k->dtype;
+  return VKL_OK;
+}
+
+int vkl_model_cache_info(const vkl_model *m, uint32_t layer, uint32_t out10[10]) {
+  if (!m || !out10 || layer >= m->cfg.layers) return fail(VKL_INVALID_ARGUMENT, "model_cache_info: bad model or layer");
+  const Layer &y = m->L[layer];
+  memset(out10, 0, 10 * sizeof(uint32_t));
+  if (y.kcache) {
+    out10[0] = (uint32_t)y.kcache->c;
+    out10[1] = (uint32_t)y.kcache->h;
+    out10[2] = (uint32_t)y.kcache->w;
+    out10[3] = y.vcache ? (uint32_t)y.vcache->w : 0u;
+    out10[4] = (uint32_t)y.kcache->dtype;
+  }
+  if (y.state) {
+    out10[5] = (uint32_t)y.state->c;
+    out10[6] = (uint32_t)y.state->h;
+    out10[7] = (uint32_t)y.state->w;
+    out10[8] = (uint32_t)y.ring->h;
+    out10[9] = (uint32_t)y.ring->w;
+    out10[4] = (uint32_t)y.ring->dtype;
+  }
+  return VKL_OK;
+}
+
+int vkl_model_read_state(vkl_model *m, uint32_t layer, float *state) {
+  if (!m || !state || layer >= m->cfg.layers) return fail(VKL_INVALID_ARGUMENT, "model_read_state: bad model or layer");
+  Layer &y = m->L[layer];
+  if (!y.state) return fail(VKL_FAILED_PRECONDITION, "model_read_state: layer %u is not recurrent", layer);
+  VKL_CUDA(cudaSetDevice(m->dev->ordinal));
+  VKL_CUDA(cudaMemcpyAsync(state, y.state->data(), y.state->device_bytes(), cudaMemcpyDeviceToHost, m->stream));
+  VKL_CUDA(cudaStreamSynchronize(m->stream));
   return VKL_OK;
 }
 
@@ -1106,6 +1148,7 @@ int vkl_model_generate(vkl_model *m, const uint32_t *prompt, size_t n_prompt, si
     return fail(VKL_OUT_OF_RANGE, "model_generate: %zu + %zu tokens run past %s", n_prompt, n_gen, m->dec ? "the context length" : "the RoPE table (2*maxlen)");
   VKL_OKAY(check_ids(m, prompt, n_prompt));
   VKL_CUDA(cudaSetDevice(m->dev->ordinal));
+  if (m->dec) VKL_OKAY(decoder_begin(m, 0));
   VKL_OKAY(ensure_rows(m, (uint32_t)n_prompt));
   VKL_OKAY(prepare_decode(m));
   const uint32_t st[2] = {0, 0};
@@ -1165,6 +1208,7 @@ int vkl_model_generate(vkl_model *m, const uint32_t *prompt, size_t n_prompt, si
     *decode_ms = ms;
   }
   VKL_OKAY(check_gemm(m));
+  if (m->dec) decoder_end(m, n_prompt + n_gen - 1);
   return check_mega(m);
 }
 
@@ -1199,6 +1243,7 @@ int vkl_model_read_kv(vkl_model *m, uint32_t layer, void *kcache, void *vcache) 
   if (!m || layer >= m->cfg.layers) return fail(VKL_INVALID_ARGUMENT, "model_read_kv: bad model or layer");
   VKL_CUDA(cudaSetDevice(m->dev->ordinal));
   Layer &y = m->L[layer];
+  if ((kcache || vcache) && !y.kcache) return fail(VKL_FAILED_PRECONDITION, "model_read_kv: layer %u has no cache of its own", layer);
   if (kcache) VKL_CUDA(cudaMemcpyAsync(kcache, y.kcache->data(), y.kcache->device_bytes(), cudaMemcpyDeviceToHost, m->stream));
   if (vcache && y.vcache) VKL_CUDA(cudaMemcpyAsync(vcache, y.vcache->data(), y.vcache->device_bytes(), cudaMemcpyDeviceToHost, m->stream));
   VKL_CUDA(cudaStreamSynchronize(m->stream));
@@ -1208,6 +1253,7 @@ int vkl_model_write_kv(vkl_model *m, uint32_t layer, const void *kcache, const v
   if (!m || layer >= m->cfg.layers) return fail(VKL_INVALID_ARGUMENT, "model_write_kv: bad model or layer");
   VKL_CUDA(cudaSetDevice(m->dev->ordinal));
   Layer &y = m->L[layer];
+  if ((kcache || vcache) && !y.kcache) return fail(VKL_FAILED_PRECONDITION, "model_write_kv: layer %u has no cache of its own", layer);
   if (kcache) VKL_CUDA(cudaMemcpyAsync(y.kcache->data(), kcache, y.kcache->device_bytes(), cudaMemcpyHostToDevice, m->stream));
   if (vcache && y.vcache) VKL_CUDA(cudaMemcpyAsync(y.vcache->data(), vcache, y.vcache->device_bytes(), cudaMemcpyHostToDevice, m->stream));
   VKL_CUDA(cudaStreamSynchronize(m->stream));
@@ -1282,6 +1328,7 @@ int vkl_model_decode_profile(vkl_model *m, uint32_t token, size_t offset, float 
   if (offset + 1 > max_positions(m)) return fail(VKL_OUT_OF_RANGE, "model_decode_profile: position out of range");
   VKL_CUDA(cudaSetDevice(m->dev->ordinal));
   VKL_OKAY(prepare_decode(m));
+  if (m->dec) m->dec->filled = Decoder::kNowhere;  // a token at any position: what the recurrent states hold is no sequence
   const uint32_t st[2] = {(uint32_t)offset, 0};
   VKL_CUDA(cudaMemcpyAsync(m->state->data(), st, 8, cudaMemcpyHostToDevice, m->stream));
   VKL_CUDA(cudaMemcpyAsync(m->toks->data(), &token, 4, cudaMemcpyHostToDevice, m->stream));
@@ -1373,6 +1420,7 @@ int vkl_model_prefill_profile(vkl_model *m, const uint32_t *toks, size_t n, floa
   VKL_OKAY(check_ids(m, toks, n));
   VKL_CUDA(cudaSetDevice(m->dev->ordinal));
   VKL_OKAY(ensure_rows(m, (uint32_t)n));
+  if (m->dec) VKL_OKAY(decoder_begin(m, 0));
   const uint32_t st[2] = {0, 0};
   VKL_CUDA(cudaMemcpyAsync(m->state->data(), st, 8, cudaMemcpyHostToDevice, m->stream));
   VKL_CUDA(cudaMemcpyAsync(m->toks->data(), toks, n * 4, cudaMemcpyHostToDevice, m->stream));
@@ -1388,7 +1436,9 @@ int vkl_model_prefill_profile(vkl_model *m, const uint32_t *toks, size_t n, floa
   for (cudaEvent_t ev : mk.ev) cudaEventDestroy(ev);
   VKL_OKAY(rc);
   if (e != cudaSuccess) return fail(VKL_INTERNAL, "model_prefill_profile: %s", cudaGetErrorString(e));
-  return check_gemm(m);
+  VKL_OKAY(check_gemm(m));
+  if (m->dec) decoder_end(m, n);
+  return VKL_OK;
 }
 
 int vkl_model_decode_trace(vkl_model *m, uint32_t token, size_t offset, unsigned long long *out, size_t cap, uint32_t *nops, uint32_t *grid, uint32_t *kinds) {

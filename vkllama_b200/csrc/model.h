@@ -15,11 +15,13 @@ struct Layer {
   vkl_tensor *wq = nullptr, *wk = nullptr, *wv = nullptr, *wo = nullptr;
   vkl_tensor *gate = nullptr, *up = nullptr, *down = nullptr;
   vkl_tensor *kcache = nullptr, *vcache = nullptr;
+  // recurrent layers: state per head [heads][value][key] in fp32, the last projections before the convolution
+  vkl_tensor *state = nullptr, *ring = nullptr;
 };
 
 // Optional per-kernel timing of a pass: an event after every launch, tagged with
 // the kernel's class (0 embedding, 1 norm+QKV, 2 attention, 3 o_proj, 4 gate/up,
-// 5 down, 6 lm head, 7 arg-max).
+// 5 down, 6 lm head, 7 arg-max, 8 recurrent layers' steps between the projections, 9 norms of their own).
 struct Marker {
   std::vector<cudaEvent_t> ev;
   std::vector<int> cls;
@@ -39,7 +41,7 @@ struct vkl_model {
   vkl_model_config cfg;
   cudaStream_t stream = nullptr;
   uint32_t head_dim = 0, heads_l = 0, dim_l = 0, ffn_l = 0, vocab_l = 0;
-  std::vector<vkl::Layer> L;  // Llama-2: blocks; a decoder design: layer runs, of which only the key caches live here
+  std::vector<vkl::Layer> L;  // Llama-2: blocks; a decoder design: layer runs, of which only caches and states live here
   std::unique_ptr<vkl::Decoder> dec;  // set for the layer-list decoder designs
   vkl_tensor *tok_embd = nullptr, *output_norm = nullptr, *output = nullptr;
   vkl_tensor *fc = nullptr, *fs = nullptr;
@@ -89,7 +91,7 @@ struct vkl_model {
     if (tp_buf) cudaFree(tp_buf);
     if (pin) cudaFreeHost(pin);
     for (auto &l : L)
-      for (vkl_tensor *p : {l.attn_norm, l.ffn_norm, l.wq, l.wk, l.wv, l.wo, l.gate, l.up, l.down, l.kcache, l.vcache}) vkl_tensor_release(p);
+      for (vkl_tensor *p : {l.attn_norm, l.ffn_norm, l.wq, l.wk, l.wv, l.wo, l.gate, l.up, l.down, l.kcache, l.vcache, l.state, l.ring}) vkl_tensor_release(p);
     for (vkl_tensor *p : mega_packed) vkl_tensor_release(p);
     for (vkl_tensor *p : {tok_embd, output_norm, output, fc, fs, x, xn, q, k, v, ao, t, gu32, logits16, logits32, toks, state, out_ids, forced, argpart, attn_scratch, attn_counters, mega_ops, mega_sync, mega_arg, mega_attn, mega_stages, mega_counts, mega_ll})
       vkl_tensor_release(p);

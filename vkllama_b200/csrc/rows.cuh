@@ -42,6 +42,9 @@ __device__ __forceinline__ float glu_act(uint32_t act, float limit, float g, flo
 }
 __device__ __forceinline__ float tanh_norm(float x, float alpha, float w, float b) { return tanhf(alpha * x) * w + b; }
 
+__device__ __forceinline__ float softplus_f(float z) { return fmaxf(z, 0.f) + log1pf(expf(-fabsf(z))); }
+__device__ __forceinline__ float soft_cap(float v, float cap) { return cap > 0.f ? cap * tanhf(v / cap) : v; }
+
 // x (already summed) of token m, column n: what follows a layer run (struct Residual).
 template <class T> __device__ __forceinline__ void finish_residual(const Residual &r, uint32_t m, uint32_t n, float x) {
   const size_t o = (size_t)m * r.ldw + n;
@@ -57,8 +60,12 @@ __device__ __forceinline__ const RowSeg &find_seg(const RowsOut &o, uint32_t n) 
   while (i + 1 < o.nseg && n >= o.seg[i].n1) ++i;
   return o.seg[i];
 }
-template <class T> __device__ __forceinline__ T *key_slot(const RowsOut &o, uint32_t pos, uint32_t c) {  // c: padded key column
-  return static_cast<T *>(o.kcache) + ((size_t)(c / o.dp) * o.maxlen + pos) * o.dp + c % o.dp;
+// c: padded column of a key or value row of width d
+template <class T> __device__ __forceinline__ T *cache_slot(void *cache, uint32_t d, uint32_t maxlen, uint32_t pos, uint32_t c) {
+  return static_cast<T *>(cache) + ((size_t)(c / d) * maxlen + pos) * d + c % d;
+}
+template <class T> __device__ __forceinline__ T *low_slot(const RowsOut &o, uint32_t m, uint32_t c) {
+  return static_cast<T *>(o.low) + (c / o.low_ld) * o.low_stride + (size_t)m * o.low_ld + c % o.low_ld;
 }
 
 // 32 consecutive results (rows n0 .. n0 + 31 of the weights, one segment) of token m.
@@ -83,9 +90,31 @@ template <class T> __device__ __forceinline__ void rows_chunk(const RowsOut &o, 
       const uint32_t pos = *o.pos + m;
 #pragma unroll
       for (int j = 0; j < 32; j += 8)
-        if (c0 + j < o.kv_heads * o.dp) store8(key_slot<T>(o, pos, c0 + j), v + j);
+        if (c0 + j < o.kv_heads * o.dp) store8(cache_slot<T>(o.kcache, o.dp, o.maxlen, pos, c0 + j), v + j);
       break;
     }
+    case ROW_VALUE: {
+      const uint32_t pos = *o.pos + m;
+#pragma unroll
+      for (int j = 0; j < 32; j += 8)
+        if (c0 + j < o.kv_heads * o.vp) store8(cache_slot<T>(o.vcache, o.vp, o.maxlen, pos, c0 + j), v + j);
+      break;
+    }
+    case ROW_LOW: {
+      T *p = low_slot<T>(o, m, c0);  // low_ld is a multiple of 32
+#pragma unroll
+      for (int j = 0; j < 32; j += 8) store8(p + j, v + j);
+      break;
+    }
+    case ROW_DECAY: {
+      float *p = o.f32 + (size_t)m * o.f32_ld + c0;
+#pragma unroll
+      for (int j = 0; j < 32; ++j) v[j] = expf(-__ldg(o.rate + n0 + j) * softplus_f(v[j]));
+#pragma unroll
+      for (int j = 0; j < 32; j += 8) store8(p + j, v + j);
+      break;
+    }
+    case ROW_NONE: break;
     case ROW_HEAD_GATE: {
       float *p = o.gate + (size_t)m * o.gate_ld + c0;
 #pragma unroll
@@ -111,7 +140,7 @@ template <class T> __device__ __forceinline__ void rows_chunk(const RowsOut &o, 
         float x[8];
         load8(r.x + at + j, x);
 #pragma unroll
-        for (int i = 0; i < 8; ++i) x[i] += v[j + i] + (r.bias ? __ldg(r.bias + n0 + j + i) : 0.f);
+        for (int i = 0; i < 8; ++i) x[i] += r.mult * (v[j + i] + (r.bias ? __ldg(r.bias + n0 + j + i) : 0.f));
         if (r.trace) store8(r.trace + at + j, x);
         if (r.emb) {
           float e[8];
@@ -136,7 +165,8 @@ template <class T> __device__ __forceinline__ void rows_chunk(const RowsOut &o, 
       float *p = o.f32 + (size_t)m * o.f32_ld + c0;
 #pragma unroll
       for (int j = 0; j < 32; j += 4)
-        *reinterpret_cast<float4 *>(p + j) = make_float4(v[j] * o.scale, v[j + 1] * o.scale, v[j + 2] * o.scale, v[j + 3] * o.scale);
+        *reinterpret_cast<float4 *>(p + j) =
+            make_float4(soft_cap(v[j] * o.scale, o.cap), soft_cap(v[j + 1] * o.scale, o.cap), soft_cap(v[j + 2] * o.scale, o.cap), soft_cap(v[j + 3] * o.scale, o.cap));
     }
   }
 }
@@ -148,11 +178,17 @@ template <class T> __device__ __forceinline__ void rows_one(const RowsOut &o, co
   switch (sg.kind) {
     case ROW_QUERY: store1(static_cast<T *>(o.q) + c, v); break;
     case ROW_KEY:
-      if (c < o.kv_heads * o.dp) store1(key_slot<T>(o, *o.pos, c), v);
+      if (c < o.kv_heads * o.dp) store1(cache_slot<T>(o.kcache, o.dp, o.maxlen, *o.pos, c), v);
       break;
+    case ROW_VALUE:
+      if (c < o.kv_heads * o.vp) store1(cache_slot<T>(o.vcache, o.vp, o.maxlen, *o.pos, c), v);
+      break;
+    case ROW_LOW: store1(low_slot<T>(o, 0, c), v); break;
+    case ROW_DECAY: o.f32[c] = expf(-o.rate[n] * softplus_f(v)); break;
+    case ROW_NONE: break;
     case ROW_HEAD_GATE: o.gate[c] = sigmoid_f(v); break;
-    case ROW_RESIDUAL: finish_residual<T>(o.res, 0, n, o.res.x[n] + (v + (o.res.bias ? o.res.bias[n] : 0.f))); break;
-    default: o.f32[c] = v * o.scale;
+    case ROW_RESIDUAL: finish_residual<T>(o.res, 0, n, o.res.x[n] + o.res.mult * (v + (o.res.bias ? o.res.bias[n] : 0.f))); break;
+    default: o.f32[c] = soft_cap(v * o.scale, o.cap);
   }
 }
 

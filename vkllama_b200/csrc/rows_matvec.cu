@@ -5,7 +5,8 @@
 // warp's lanes hold 8 columns each: four coalesced 128-bit weight loads per step and lane, eight inputs, 32
 // fp32 FMAs. What becomes of a row is in its segment (rows.h), so one launch runs everything that reads the
 // same input: keys, queries, head gates and the feed-forward's gate/up rows of a parallel block, and the
-// gate/up rows of the experts that the token's id names. The out-projection form sums, per output row, the
+// gate/up rows of the experts that the token's id names. Rows may be split between two inputs (two norms of one
+// stream). The out-projection form sums, per output row, the
 // attention's columns, the dense feed-forward's columns (one matrix, side by side) or the chosen experts'
 // rows, and leaves the residual stream and the next norm's output behind.
 #include <algorithm>
@@ -68,7 +69,9 @@ template <class T, int KS, bool OUT> __global__ void __launch_bounds__(kThreads)
   __shared__ float red[2][kWarps][4];
   const uint32_t warp = threadIdx.x >> 5, lane = threadIdx.x & 31, wg = warp / KS, ws = warp % KS;
   const uint32_t k0 = (ws * 32 + lane) * 8, step = KS * 256;
-  const uint32_t u_main = p.N / 4, u_exp = p.ne / 4, units = u_main + (OUT ? 0u : p.top * u_exp);
+  const uint32_t gap = p.n2 - p.gap0;  // rows without a result
+  const uint32_t u_main = (p.N - gap) / 4, u_exp = p.ne / 4, units = u_main + (OUT ? 0u : p.top * u_exp);
+  auto first_row = [&](uint32_t u) { return u * 4 + (u * 4 >= p.gap0 ? gap : 0u); };
   const uint32_t rounds = (units + gridDim.x * UPC - 1) / (gridDim.x * UPC);
   // rows of unit u of a segment: four in a row, or two gate rows and the up rows of the same two outputs
   auto glu_row = [](uint32_t u) { return (u / 8) * 32 + (u % 8) * 2; };
@@ -76,7 +79,7 @@ template <class T, int KS, bool OUT> __global__ void __launch_bounds__(kThreads)
     // the weights do not depend on the kernel before: ask for the first unit's rows, then wait for it
     const uint32_t u = blockIdx.x * UPC + wg;
     if (u < u_main) {
-      const bf16 *w = p.w + (size_t)(u * 4) * p.K;
+      const bf16 *w = p.w + (size_t)first_row(u) * p.K;
       for (uint32_t k = k0, i = 0; k < p.K && i < 2; k += step, ++i)
         for (int r = 0; r < 4; ++r) prefetch_l2(w + (size_t)r * p.K + k);
     }
@@ -93,9 +96,11 @@ template <class T, int KS, bool OUT> __global__ void __launch_bounds__(kThreads)
     if (active) {
       const T *x = static_cast<const T *>(p.x);
       if (u < u_main) {
-        sg = find_seg(p.out, u * 4);
+        n = first_row(u);
+        if (p.x2 && n >= p.n2) x = static_cast<const T *>(p.x2);
+        sg = find_seg(p.out, n);
         glu = !OUT && sg.kind == ROW_GLU;
-        n = glu ? sg.n0 + glu_row(u - sg.n0 / 4) : u * 4;
+        if (glu) n = sg.n0 + glu_row((n - sg.n0) / 4);
         const bf16 *w = p.w + (size_t)n * p.K, *w2 = w + (size_t)(glu ? 16 : 2) * p.K;
         dot4<T>(acc, w, w + p.K, w2, w2 + p.K, x, k0, step, p.K, 1.f);
         if (OUT) {
@@ -169,7 +174,7 @@ template <class T, int KS, bool OUT> cudaError_t launch_t(const MvRows &p, uint3
 }
 
 template <class T, bool OUT> cudaError_t launch_ks(const MvRows &p, int sms, cudaStream_t s) {
-  const uint32_t units = p.N / 4 + (OUT ? 0u : p.top * (p.ne / 4));
+  const uint32_t units = (p.N - (p.n2 - p.gap0)) / 4 + (OUT ? 0u : p.top * (p.ne / 4));
   // enough warps to keep the memory system busy, as long as each has a step of K of its own
   uint32_t ks = 1;
   while (ks < 8 && units * ks < (uint32_t)sms * 24 && p.K >= 512 * ks) ks *= 2;
@@ -184,7 +189,7 @@ template <class T, bool OUT> cudaError_t launch_ks(const MvRows &p, int sms, cud
 }  // namespace
 
 cudaError_t launch_rows_matvec(const MvRows &p, bool f32, int sms, cudaStream_t s) {
-  if (!p.N || p.N % 32 || p.K % 64 || (p.top && (p.ke % 64 || p.ne % 32))) return cudaErrorInvalidValue;
+  if (!p.N || p.N % 32 || p.K % 64 || p.gap0 % 32 || p.n2 % 32 || p.gap0 > p.n2 || p.n2 > p.N || (p.top && (p.ke % 64 || p.ne % 32))) return cudaErrorInvalidValue;
   if (f32) return p.out_proj ? launch_ks<float, true>(p, sms, s) : launch_ks<float, false>(p, sms, s);
   return p.out_proj ? launch_ks<bf16, true>(p, sms, s) : launch_ks<bf16, false>(p, sms, s);
 }
