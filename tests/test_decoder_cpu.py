@@ -130,7 +130,7 @@ def create(text):
 
 
 def test_config_reader():
-    assert vk.architectures() == ["Rumalorn"]
+    assert vk.architectures() == ["Rumalorn", "Kupuzen"]
     for cfg in U.CASES.values():
         st, msg = create(json.dumps(cfg))
         assert st == 3 and "null device" in msg  # the config itself was taken

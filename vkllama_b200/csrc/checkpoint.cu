@@ -234,6 +234,7 @@ int rumalorn_spec(const Json &c, const Shapes &, DecoderSpec *s) {
     VKL_OKAY(get_object(j, "mixer", &mix));
     AttnSpec &a = l.attn;
     uint32_t vdim = 0;
+    a.proj_bias = a.head_gate = true;
     VKL_OKAY(get_u32(*mix, "heads", &a.heads));
     VKL_OKAY(get_u32(*mix, "kv_heads", &a.kv_heads));
     VKL_OKAY(get_u32(*mix, "dim", &a.dim));
