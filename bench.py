@@ -322,20 +322,45 @@ def run_gemm(args):
 DESIGN_SIZES = {"1b": (2048, 16, 5632, 12, 32000), "7b": (4096, 32, 11008, 8, 32000), "13b": (5120, 40, 13824, 6, 32000)}
 
 
+FP32_FLOPS = 148 * 128 * 2 * 1.965e9  # nominal
+DESIGN_VARIANTS = {"Rumalorn": "llama,dense,gqa,moe", "Kupuzen": "llama,rumalorn,delta,window,mixed"}
+DELTA_RANK, WINDOW = 128, 1024
+
+
+def design_layers(variant, nl):
+    """Kupuzen's layers by variant: 'd' delta rule, 'a' windowed attention, 's' the same with the cache of the layer before."""
+    return {"delta": "d", "window": "a", "mixed": "ddas"}[variant] * nl
+
+
 def design_config(name, size, variant):
-    """A config of the design at a size: 'dense' has the closest model's layers (as many key heads as heads), 'gqa' a
-    quarter of the key heads, 'moe' 16 experts of a quarter of the width (two per token) in every other layer and a loop."""
+    """A config of a design at a size, and the tensor shapes that it leaves open.
+    Rumalorn: 'dense' has the Llama layers (as many key heads as heads), 'gqa' a quarter of the key heads, 'moe' 16
+    experts of a quarter of the width (two per token) in every other layer and a loop. Kupuzen: 'delta' and 'window' have
+    one kind of layer (as many key heads as heads), 'mixed' two delta-rule layers, then two that share a windowed cache."""
     d, h, f, nl, v = DESIGN_SIZES[size]
-    mix = {"heads": h, "kv_heads": h if variant == "dense" else h // 4, "dim": d // h, "vdim": d // h, "scale": (d // h) ** -0.5,
+    hd = d // h
+    if name == "Kupuzen":
+        mix = {"heads": h, "kv_heads": h, "dim": hd, "vdim": hd}
+        attn = dict(mix, scale=hd ** -0.5, mask={"size": WINDOW},
+                    rot={"base": 500000.0, "dims": hd, "scaling": {"factor": 8.0, "low": 1.0, "high": 4.0, "original": 8192}})
+        layers, shapes = [], {}
+        for i, k in enumerate(design_layers(variant, nl)[:nl]):
+            layers.append({"type": "channel_delta" if k == "d" else "attention", "mlp": {"kind": "dense", "ff": f},
+                           "mixer": dict(mix, conv=4) if k == "d" else dict(attn, kv_from=i - 1) if k == "s" else attn})
+            if k == "d":
+                shapes.update({"l%d.mix.a1" % i: (DELTA_RANK, d), "l%d.mix.g1" % i: (DELTA_RANK, d)})
+        return {"architecture": name, "vocab": v, "width": d, "embedding": {"scale": 1.0}, "residual_mult": 1.0, "logit_softcap": 30.0,
+                "norm": {"eps": 1e-6}, "layers": layers}, shapes
+    mix = {"heads": h, "kv_heads": h if variant == "dense" else h // 4, "dim": hd, "vdim": hd, "scale": hd ** -0.5,
            "bias_max": 1024, "q_temp": {"coef": 0.1, "every": 512}}
     dense = {"kind": "dense", "ff": f, "limit": 7.0}
     moe = {"kind": "moe", "expert": {"ff": f // 4}, "router": {"experts": 16, "top": 2}}
     return {"architecture": name, "vocab": v, "width": d, "logit_scale": 1.0, "norm": {"eps": 1e-6},
             "loop": {"start": 0, "stop": nl // 2, "times": 2} if variant == "moe" else None,
-            "layers": [{"type": "attention", "mixer": mix, "mlp": moe if variant == "moe" and i % 2 else dense} for i in range(nl)]}
+            "layers": [{"type": "attention", "mixer": mix, "mlp": moe if variant == "moe" and i % 2 else dense} for i in range(nl)]}, {}
 
 
-def design_work(size, variant, T):
+def design_work(name, size, variant, T):
     """Algorithmic bytes of one decode token and FLOPs of a T-token prompt pass, per kernel class (the classes of
     vkl_model_decode_profile / vkl_model_prefill_profile), for the design's variant or for 'llama'."""
     d, h, f, nl, v = DESIGN_SIZES[size]
@@ -345,7 +370,20 @@ def design_work(size, variant, T):
         b.update({"in": nl * 2.0 * (3 * d * d + 2 * f * d), "out": nl * 2.0 * (d * d + f * d), "attn": nl * 2.0 * 2 * d * T})
         fl.update({"in": nl * 2.0 * T * (3 * d * d + 2 * f * d), "out": nl * 2.0 * T * (d * d + f * d), "attn": nl * 2.0 * d * T * T})
         return b, fl
-    kv = h if variant == "dense" else h // 4
+    if name == "Kupuzen" and variant != "rumalorn":
+        kinds = design_layers(variant, nl)[:nl]
+        rows = {"d": 3 * d + 2 * DELTA_RANK + h, "a": 3 * d, "s": d}
+        na, nd, seen = sum(k != "d" for k in kinds), kinds.count("d"), min(T, WINDOW)
+        pairs = sum(min(i + 1, WINDOW) for i in range(T))  # a query's visible keys, over a prompt
+        b.update({"in": sum(2.0 * d * (rows[k] + 2 * f) for k in kinds), "out": nl * 2.0 * (d * d + f * d)})
+        fl.update({"in": T * b["in"], "out": T * b["out"]})
+        if na:
+            b["attn"], fl["attn"] = na * 2.0 * 2 * d * seen, na * 2.0 * 2 * d * pairs
+        if nd:  # state in and out, the second steps of decay and gate; a prompt: those, and seven operations per state element and token
+            b["delta"] = nd * (2 * 4.0 * d * hd + 2.0 * 2 * d * DELTA_RANK)
+            fl["delta"] = nd * T * (7.0 * d * hd + 2.0 * 2 * d * DELTA_RANK)
+        return b, fl
+    kv = h if variant in ("dense", "rumalorn") else h // 4
     runs = [i for _ in range(2) for i in range(nl // 2)] + list(range(nl // 2, nl)) if variant == "moe" else list(range(nl))
     b.update({"in": 0.0, "out": 0.0, "attn": len(runs) * 2.0 * kv * hd * T})
     fl.update({"in": 0.0, "out": 0.0, "attn": len(runs) * 2.0 * d * T * T, "experts": 0.0})
@@ -365,7 +403,7 @@ def design_work(size, variant, T):
 
 def run_design(args):
     """Prefill and decode throughput of a decoder design (random weights) at a few layer shapes beside the Llama-2
-    driver with FP16 weights at the same shape (the closest model of the library: 16-bit weights, the same GEMM), with
+    driver with FP16 weights at the same shape (16-bit weights, the same GEMM; for Kupuzen also beside Rumalorn), with
     every kernel class's share of its roofline. Weights are larger than L2 and every pass reads all of them."""
     import vkllama_b200 as vk
     from vkllama_b200.synth import synth_tokens
@@ -378,11 +416,12 @@ def run_design(args):
     launches0 = vk.kernel_launches()
     for size in args.design_sizes.split(","):
         d, h, f, nl, v = DESIGN_SIZES[size]
-        for variant in args.design_variants.split(","):
+        for variant in (args.design_variants or DESIGN_VARIANTS[args.design]).split(","):
             if variant == "llama":
                 m = vk.Model(dev, d, h, f, v, nl, max(4096, T + n_dec + 1), weight_dtype=vk.FP16)
             else:
-                m = vk.Model.from_config(dev, design_config(args.design, size, variant), max(4096, T + n_dec + 1), vk.BF16)
+                cfg, shapes = design_config("Rumalorn", size, "dense") if variant == "rumalorn" else design_config(args.design, size, variant)
+                m = vk.Model.from_config(dev, cfg, max(4096, T + n_dec + 1), vk.BF16, shapes=shapes)
             m.synth_weights(17)
             prompt = synth_tokens(17, 1000, T, v)
             pre, dec = [], []
@@ -394,7 +433,7 @@ def run_design(args):
             reps = 10
             pp = np.mean([m.prefill_profile(prompt) for _ in range(reps + 2)][2:], axis=0)
             dp = np.mean([m.decode_profile(int(prompt[i]), T + i) for i in range(reps + 2)][2:], axis=0)
-            b, fl = design_work(size, variant, T)
+            b, fl = design_work(args.design, size, variant, T)
             dt = {"in": dp[1] + dp[4], "attn": dp[2], "out": dp[3] + dp[5], "head": dp[6]}
             if variant == "llama":
                 pt = {"in": pp[1] + pp[4], "attn": pp[2], "out": pp[3] + pp[5]}
@@ -402,13 +441,20 @@ def run_design(args):
                 pt = {"in": pp[1], "attn": pp[2], "out": pp[3], "experts": pp[4] + pp[5]}
             else:
                 pt = {"in": pp[1], "attn": pp[2], "out": pp[3]}
-            weights = b["in"] + b["out"] + b["head"]
+            if "delta" in b:
+                dt["delta"], pt["delta"] = dp[8], pp[8]
+            for times in (dt, pt):
+                if "attn" not in b:
+                    del times["attn"]
+            other = {"decode_norms_us": float(dp[9]), "prefill_norms_us": float(pp[9])}
             rows.append({"size": size, "variant": variant, "prefill_tokens_per_s": T / (np.median(pre) * 1e-3), "decode_tokens_per_s": 1000.0 / np.median(dec),
                          "prefill_ms": float(np.median(pre)), "decode_ms": float(np.median(dec)),
-                         "decode_frac_of_hbm": (weights + b["attn"]) / (np.median(dec) * 1e-3) / 1e9 / hbm,
+                         "decode_frac_of_hbm": sum(b[k] for k in dt) / (np.median(dec) * 1e-3) / 1e9 / hbm,
                          "prefill_frac_of_tensor": sum(fl.values()) / (np.median(pre) * 1e-3) / 1e12 / tens,
                          "decode_kernels": {k: {"us": float(dt[k]), "frac_of_hbm": b[k] / (dt[k] * 1e-6) / 1e9 / hbm} for k in dt},
-                         "prefill_kernels": {k: {"us": float(pt[k]), "frac_of_tensor": fl[k] / (pt[k] * 1e-6) / 1e12 / tens} for k in pt}})
+                         "prefill_kernels": {k: {"us": float(pt[k]), "frac_of_tensor": fl[k] / (pt[k] * 1e-6) / 1e12 / tens} for k in pt}, **other})
+            if "delta" in b:  # the recurrence is fp32: its roof is the FMA units'
+                rows[-1]["prefill_kernels"]["delta"]["frac_of_fp32"] = fl["delta"] / (pt["delta"] * 1e-6) / FP32_FLOPS
             if variant == "moe":  # few tokens per expert: the weights' stream is the lower roof
                 rows[-1]["prefill_kernels"]["experts"]["frac_of_hbm"] = b["experts_prompt"] / (pt["experts"] * 1e-6) / 1e9 / hbm
             m.close()
@@ -422,7 +468,7 @@ def main():
     ap = argparse.ArgumentParser()
     ap.add_argument("--design", default=None, help="a registered decoder design: its throughput beside the Llama-2 driver's at equal size, instead of the token loop")
     ap.add_argument("--design-sizes", default="1b,7b,13b")
-    ap.add_argument("--design-variants", default="llama,dense,gqa,moe")
+    ap.add_argument("--design-variants", default=None, help="default: the design's own, see DESIGN_VARIANTS")
     ap.add_argument("--design-prompt", type=int, default=512)
     ap.add_argument("--design-decode", type=int, default=64)
     ap.add_argument("--micro", default=None, help="'all' or ROWSxK: Q8_0 mat-vec microbenchmark instead of the token loop")

@@ -42,7 +42,7 @@ double rotation_frequency(const RotSpec &r, uint32_t i) {
 Decoder::~Decoder() {
   for (DecLayer &l : L)
     for (vkl_tensor *t : {l.norm.w, l.norm.b, l.norm2.w, l.norm2.b, l.qw, l.kw, l.freq, l.sink, l.taps, l.wl, l.biasl, l.rate, l.onorm, l.w1, l.bias1, l.w2, l.bias_o, l.rel, l.we1, l.we2, l.table, l.slot, l.token, l.tile_expert}) vkl_tensor_release(t);
-  for (vkl_tensor *t : {emb, head, step, final_norm.w, final_norm.b, x, h, q, gate, a2, low, dq, dk, dv, dg, ogate, xe, hp, tp, y, want, hw, logits_rows, trace, attn_scratch, attn_counters}) vkl_tensor_release(t);
+  for (vkl_tensor *t : {emb, head, step, final_norm.w, final_norm.b, x, h, q, gate, a2, low, dv, dz, dblocks, xe, hp, tp, y, want, hw, logits_rows, trace, attn_scratch, attn_counters}) vkl_tensor_release(t);
 }
 
 namespace {
@@ -442,8 +442,7 @@ int build_attention(vkl_model *m, DecLayer &l, const AttnSpec &a) {
 int build_delta(vkl_model *m, DecLayer &l, const DeltaSpec &p) {
   Decoder *d = m->dec.get();
   d->recurrent = true;
-  l.lgap0 = up_to(p.heads * l.dp, 32);
-  l.ln2 = up_to(l.lgap0, kInputAlign);
+  l.ln2 = up_to(p.heads * l.dp, kInputAlign);
   l.nl = l.ln2 + up_to(p.heads * l.vp, 32);
   VKL_OKAY(zeros(m, &l.taps, 1, l.qcols, p.taps, VKL_FP32));
   VKL_OKAY(zeros(m, &l.wl, 1, l.nl, l.lowp, VKL_BF16));
@@ -451,10 +450,8 @@ int build_delta(vkl_model *m, DecLayer &l, const DeltaSpec &p) {
   VKL_OKAY(zeros(m, &l.rate, 1, 1, l.ln2, VKL_FP32));
   VKL_OKAY(zeros(m, &l.onorm, 1, 1, l.vp, VKL_FP32));
   d->low_max = std::max(d->low_max, l.lowp);
-  d->dqk_max = std::max(d->dqk_max, p.kv_heads * l.dp);
   d->dv_max = std::max(d->dv_max, p.heads * l.vp);
-  d->dg_max = std::max(d->dg_max, l.lgap0);
-  d->og_max = std::max(d->og_max, up_to(p.heads * l.vp, 32));
+  d->dz_max = std::max(d->dz_max, l.nl);
   d->gld_max = std::max(d->gld_max, up_to(p.heads, 32));
   return VKL_OK;
 }
@@ -668,11 +665,14 @@ int decoder_ensure_rows(vkl_model *m, uint32_t T) {
   VKL_OKAY(zeros(m, &d->gate, 1, T, d->gld_max, VKL_FP32));
   if (d->recurrent) {
     VKL_OKAY(zeros(m, &d->low, 2, T, d->low_max, ct));
-    VKL_OKAY(zeros(m, &d->dq, 1, T, d->dqk_max, VKL_FP32));
-    VKL_OKAY(zeros(m, &d->dk, 1, T, d->dqk_max, VKL_FP32));
-    VKL_OKAY(zeros(m, &d->dv, 1, T, d->dv_max, VKL_FP32));
-    VKL_OKAY(zeros(m, &d->dg, 1, T, d->dg_max, VKL_FP32));
-    VKL_OKAY(zeros(m, &d->ogate, 1, T, d->og_max, VKL_FP32));
+    if (T > 1) {
+      VKL_OKAY(zeros(m, &d->dv, 1, T, d->dv_max, VKL_FP32));
+      VKL_OKAY(zeros(m, &d->dz, 1, T, d->dz_max, VKL_FP32));
+      size_t most = 0;
+      for (size_t i = 0; i < d->L.size(); ++i)
+        if (d->spec.layers[i].mixer == MIX_DELTA) most = std::max(most, delta_block_floats(T, d->spec.layers[i].delta.heads, d->L[i].dp));
+      VKL_OKAY(zeros(m, &d->dblocks, 1, 1, most, VKL_FP32));
+    }
   }
   VKL_OKAY(zeros(m, &d->a2, 1, T, d->k2_max, ct));
   VKL_OKAY(zeros(m, &m->toks, 1, 1, T, VKL_UINT32));
@@ -848,6 +848,7 @@ int decoder_begin(vkl_model *m, size_t offset) {
 void decoder_end(vkl_model *m, size_t end) { m->dec->filled = end; }
 
 #define MARK(c) do { if (mk) mk->mark(c); } while (0)
+#define MARK_NORM() do { if (d->spec.norm != NORM_TANH) MARK(9); } while (0)
 
 namespace {
 // The delta rule's steps between the projections of layer run r.
@@ -855,45 +856,8 @@ int run_delta(vkl_model *m, size_t r, uint32_t T, bool pdl) {
   Decoder *d = m->dec.get();
   DecLayer &l = d->L[d->runs[r].layer];
   const DeltaSpec &a = d->spec.layers[d->runs[r].layer].delta;
-  const bool one = T == 1, f32 = d->f32;
+  const bool f32 = d->f32;
   cudaStream_t s = m->stream;
-  // decays and output gates: the second steps of their projections, one matrix over two inputs
-  RowsOut out = {};
-  out.seg[0] = RowSeg{0, l.lgap0, ROW_DECAY};
-  out.seg[1] = RowSeg{l.lgap0, l.ln2, ROW_NONE};
-  out.seg[2] = RowSeg{l.ln2, l.nl, ROW_HEAD_GATE};
-  out.nseg = 3;
-  out.bias = (const float *)l.biasl->data();
-  out.rate = (const float *)l.rate->data();
-  out.f32 = (float *)d->dg->data();
-  out.f32_ld = l.lgap0;
-  out.gate = (float *)d->ogate->data();
-  out.gate_ld = l.nl - l.ln2;
-  if (one) {
-    MvRows p = {};
-    p.w = (const bf16 *)l.wl->data();
-    p.N = l.nl;
-    p.K = l.lowp;
-    p.x = d->low->data();
-    p.x2 = d->low->data() + (size_t)l.lowp * elem(d);
-    p.n2 = l.ln2;
-    p.gap0 = l.lgap0;
-    p.out = out;
-    p.use_pdl = pdl;
-    VKL_LAUNCH(1, launch_rows_matvec(p, f32, m->dev->prop.multiProcessorCount, s));
-  } else {
-    GemmRows g = {};
-    g.a = d->low->data();
-    g.w = (const bf16 *)l.wl->data();
-    g.M = T;
-    g.N = l.nl;
-    g.K = l.lowp;
-    g.n2 = l.ln2;
-    g.out = out;
-    g.error = (uint32_t *)m->state->data() + 6;
-    m->gemm_used = true;
-    VKL_LAUNCH(1, f32 ? launch_gemm_rows_f32(g, s) : launch_gemm_rows_bf16(g, s));
-  }
   DeltaRows p = {};
   p.raw = d->q->data();
   p.raw_ld = l.qcols;
@@ -910,24 +874,45 @@ int run_delta(vkl_model *m, size_t r, uint32_t T, bool pdl) {
   p.vdim = a.vdim;
   p.dp = l.dp;
   p.vp = l.vp;
-  p.q = (float *)d->dq->data();
-  p.k = (float *)d->dk->data();
-  p.v = (float *)d->dv->data();
-  p.g = out.f32;
-  p.g_ld = out.f32_ld;
+  p.bias = (const float *)l.biasl->data();
+  p.rate = (const float *)l.rate->data();
   p.beta = (const float *)d->gate->data();
   p.beta_ld = d->gld_max;
   p.state = (float *)m->L[r].state->data();
   p.norm = (const float *)l.onorm->data();
   p.eps = d->spec.norm_eps;
-  p.gate = out.gate;
-  p.gate_ld = out.gate_ld;
   p.out = d->a2->data();
   p.out_ld = l.k2;
   p.use_pdl = pdl;
-  VKL_LAUNCH(1, launch_delta_prepare(p, f32, s));
-  VKL_LAUNCH(1, launch_delta_recurrence(p, s));
-  VKL_LAUNCH(1, launch_delta_finish(p, f32, s));
+  p.z_gate = l.ln2;
+  if (T == 1) {
+    p.wl = (const bf16 *)l.wl->data();
+    p.low = d->low->data();
+    p.low_ld = l.lowp;
+    VKL_LAUNCH(1, launch_delta_step(p, f32, s));
+    return VKL_OK;
+  }
+  // the second steps of the decays' and the gates' projections: one matrix over two inputs
+  GemmRows g = {};
+  g.a = d->low->data();
+  g.w = (const bf16 *)l.wl->data();
+  g.M = T;
+  g.N = l.nl;
+  g.K = l.lowp;
+  g.n2 = l.ln2;
+  g.out.seg[0] = RowSeg{0, l.nl, ROW_STORE};
+  g.out.nseg = 1;
+  g.out.f32 = (float *)d->dz->data();
+  g.out.f32_ld = l.nl;
+  g.out.scale = 1.f;
+  g.error = (uint32_t *)m->state->data() + 6;
+  m->gemm_used = true;
+  VKL_LAUNCH(1, f32 ? launch_gemm_rows_f32(g, s) : launch_gemm_rows_bf16(g, s));
+  p.z = g.out.f32;
+  p.z_ld = l.nl;
+  p.v = (float *)d->dv->data();
+  p.blocks = (float *)d->dblocks->data();
+  VKL_LAUNCH(delta_launches(T), launch_delta_rows(p, f32, s));
   return VKL_OK;
 }
 }  // namespace
@@ -960,7 +945,7 @@ int decoder_run(vkl_model *m, uint32_t T, bool pdl, Marker *mk) {
   VKL_LAUNCH(1, launch_embed_rows((const bf16 *)d->emb->data(), toks, T, d->spec.embed_scale, residual_after(m, -1), f32, s));
   MARK(0);
   VKL_OKAY(norm_after(m, -1, T, false));
-  MARK(9);
+  MARK_NORM();
   for (size_t r = 0; r < d->runs.size(); ++r) {
     const uint32_t i = d->runs[r].layer;
     DecLayer &l = d->L[i];
@@ -1113,7 +1098,7 @@ int decoder_run(vkl_model *m, uint32_t T, bool pdl, Marker *mk) {
       VKL_LAUNCH(1, launch_rows_matvec(p, f32, sms, s));
       MARK(5);
       VKL_OKAY(norm_after(m, (int)r, T, pdl));
-      MARK(9);
+      MARK_NORM();
       continue;
     }
     if (moe) {
@@ -1171,7 +1156,7 @@ int decoder_run(vkl_model *m, uint32_t T, bool pdl, Marker *mk) {
       MARK(5);
     }
     VKL_OKAY(norm_after(m, (int)r, T, false));
-    MARK(9);
+    MARK_NORM();
   }
   // --- output layer: the last row for the token loop, and the rows a caller asked for
   MvRows p = {};

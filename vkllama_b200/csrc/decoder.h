@@ -95,7 +95,7 @@ struct DecLayer {
   vkl_tensor *qw = nullptr, *kw = nullptr, *freq = nullptr, *sink = nullptr;  // query and key norm, angles, sinks
   // delta rule: convolution taps, second steps of decay and gate (one matrix, two inputs), its bias, the decays' rates, norm
   vkl_tensor *taps = nullptr, *wl = nullptr, *biasl = nullptr, *rate = nullptr, *onorm = nullptr;
-  uint32_t lowp = 0, nl = 0, lgap0 = 0, ln2 = 0;
+  uint32_t lowp = 0, nl = 0, ln2 = 0;
   vkl_tensor *we1 = nullptr, *we2 = nullptr, *table = nullptr;  // experts: gate/up rows, down rows, token table
   vkl_tensor *slot = nullptr, *token = nullptr, *tile_expert = nullptr;  // routing of the current pass's tokens
 };
@@ -120,10 +120,10 @@ struct Decoder {
   std::set<std::string> loaded;
   // activations for vkl_model::cap_T rows
   vkl_tensor *x = nullptr, *h = nullptr, *q = nullptr, *gate = nullptr, *a2 = nullptr;
-  vkl_tensor *low = nullptr, *dq = nullptr, *dk = nullptr, *dv = nullptr, *dg = nullptr, *ogate = nullptr;  // delta rule
+  vkl_tensor *low = nullptr, *dv = nullptr, *dz = nullptr, *dblocks = nullptr;  // delta rule
   vkl_tensor *xe = nullptr, *hp = nullptr, *tp = nullptr, *y = nullptr;  // experts: one token; grouped rows
   vkl_tensor *want = nullptr, *hw = nullptr, *logits_rows = nullptr, *trace = nullptr;
-  uint32_t low_max = 0, dqk_max = 0, dv_max = 0, dg_max = 0, og_max = 0;
+  uint32_t low_max = 0, dv_max = 0, dz_max = 0;
   uint32_t qld_max = 0, gld_max = 0, k2_max = 0, top_max = 0, ffe_max = 0, experts_max = 0, heads_max = 0;
   vkl_tensor *attn_scratch = nullptr, *attn_counters = nullptr;
   uint32_t counters_n = 0;

@@ -1,245 +1,599 @@
-// Gated delta rule with a decay per head and key channel, for prompts and portions of any length: the steps between
-// the in-projection and the out-projection. Everything is fp32 except the projections that come in and the rows
-// that go out.
+// Gated delta rule with a decay per head and key channel: everything between the in-projection and the out-projection
+// of a recurrent layer. All arithmetic is fp32 except the projections that come in and the rows that go out.
 //
-//   prepare     a warp per token and row (query, key or value head): short causal convolution over time, SiLU, unit
-//               norm of queries and keys. Tokens before the call come from the ring of past projections.
-//   recurrence  the columns of a state do not depend on each other: a CTA owns 16 columns of a head in registers,
-//               eight lanes per column, and walks over the tokens. Queries, keys, decays and values travel through a
-//               ring of shared-memory stages. A column's arithmetic is the same however a prompt is cut.
-//   finish      a warp per token and head: RMS norm of the head's outputs, gate; and the call's last projections
-//               go to the ring.
+// Many tokens, in blocks of eight. Inside a block the recurrence is unrolled: with P_t the product of the block's decays
+// up to token t, and S the state before the block,
+//   w_t = v_t - S^T (P_t k_t)                          how far the state is from each value,
+//   u   = M w, M = (1 + beta A)^-1 beta                A_ts = k_t . (decays s+1 .. t) k_s for s < t, the writes' overlap,
+//   o_t = S^T (P_t q_t) + (N w)_t, N = B M             B_ts = q_t . (decays s+1 .. t) k_s for s <= t,
+//   S  <- P_8 S + sum_s (decays s+1 .. 8) k_s u_s^T.
+// Decays only ever multiply (no quotient of products), so nothing overflows and a decay of zero is exact.
+//   blocks      a CTA per head and block: convolution, SiLU, unit norms, decays, and from them the rows P k, P q,
+//               (later decays) k, the product of the decays, M and N. Depends on no state: all blocks at once.
+//   scan        the columns of a state do not depend on each other: 16 lanes hold four columns in registers and walk
+//               over the blocks, whose rows travel through a ring of shared-memory stages. A column's arithmetic within
+//               a block is all independent dot products.
+//   finish      a warp per token and head: RMS norm of the head's outputs, gate; and the call's last projections go to
+//               the ring of past projections.
+// One token: a cluster of CTAs per head, 32 columns each, does all of it in one kernel; what does not depend on the
+// kernel before (weights, state) is requested before waiting for it, and the norm's sum crosses the cluster.
+#include <cooperative_groups.h>
+
 #include <algorithm>
+#include <type_traits>
 
 #include "rows.cuh"
 
 namespace vkl {
 namespace {
 
-constexpr int kThreads = 256, kWarps = kThreads / 32;
+namespace cg = cooperative_groups;
+
 constexpr float kUnitEps = 1e-6f;
+constexpr uint32_t kBlock = 8, kPairsA = 28, kPairs = 64;  // token pairs s < t, and those plus s <= t
 
 __device__ __forceinline__ float load1(const bf16 *p) { return __bfloat162float(*p); }
 __device__ __forceinline__ float load1(const float *p) { return *p; }
 __device__ __forceinline__ float silu_f(float z) { return z * sigmoid_f(z); }
 
-// Channel c of token m after convolution and SiLU; pos0: position of token 0.
-template <class T> __device__ __forceinline__ float convolved(const DeltaRows &p, uint32_t m, uint32_t pos0, uint32_t c) {
-  const float *w = p.taps + (size_t)c * p.ntaps;
-  float a = 0.f;
-  for (uint32_t j = 0; j < p.ntaps; ++j) {
-    const uint32_t back = p.ntaps - 1 - j;
-    if (back > pos0 + m) continue;  // before the sequence's start
-    const T *x = back <= m ? static_cast<const T *>(p.raw) + (size_t)(m - back) * p.raw_ld : static_cast<const T *>(p.ring) + (size_t)((pos0 + m - back) % p.ntaps) * p.raw_ld;
-    a = fmaf(load1(x + c), w[j], a);
-  }
-  return silu_f(a);
+// Projection c of token m, which may lie before the call's first token (position pos0) or the sequence's.
+template <class T> __device__ __forceinline__ float projection(const DeltaRows &p, int m, uint32_t pos0, uint32_t c) {
+  if (m >= 0) return load1(static_cast<const T *>(p.raw) + (size_t)m * p.raw_ld + c);
+  const int at = (int)pos0 + m;
+  return at < 0 ? 0.f : load1(static_cast<const T *>(p.ring) + (size_t)((uint32_t)at % p.ntaps) * p.raw_ld + c);
 }
 
-template <class T> __global__ void __launch_bounds__(kThreads) delta_prepare_kernel(const DeltaRows p) {
-  if (p.use_pdl) asm volatile("griddepcontrol.wait;" ::: "memory");
-  const uint32_t m = blockIdx.x, lane = threadIdx.x & 31, unit = blockIdx.y * kWarps + (threadIdx.x >> 5);
-  const uint32_t pos0 = *p.pos;
-  if (unit >= 2 * p.kv_heads + p.heads) return;
-  if (unit >= 2 * p.kv_heads) {
-    const uint32_t h = unit - 2 * p.kv_heads;
-    float *v = p.v + ((size_t)m * p.heads + h) * p.vp;
-    for (uint32_t d = lane; d < p.vp; d += 32) v[d] = convolved<T>(p, m, pos0, p.v_col + h * p.vp + d);
-    return;
-  }
-  const bool key = unit >= p.kv_heads;
-  const uint32_t g = key ? unit - p.kv_heads : unit;
-  float y[8], ss = 0.f;
+// Channel c of tokens t0 .. t0 + 7 after convolution and SiLU; 0 from token n on. TAPS: 0 for any number.
+template <class T, int TAPS> __device__ __forceinline__ void convolve8(const DeltaRows &p, uint32_t t0, uint32_t n, uint32_t pos0, uint32_t c, float (&y)[kBlock]) {
+  const float *w = p.taps + (size_t)c * p.ntaps;
+  if constexpr (TAPS > 0) {
+    float x[kBlock + TAPS - 1], wr[TAPS];
 #pragma unroll
-  for (int i = 0; i < 8; ++i) {
-    const uint32_t d = i * 32 + lane;
-    y[i] = d < p.dp ? convolved<T>(p, m, pos0, (key ? p.k_col : 0u) + g * p.dp + d) : 0.f;
-    ss = fmaf(y[i], y[i], ss);
-  }
-  ss = warp_sum(ss);
-  const float r = 1.0f / sqrtf(ss + kUnitEps) * (key ? 1.f : 1.0f / sqrtf((float)p.dim));
-  float *o = (key ? p.k : p.q) + ((size_t)m * p.kv_heads + g) * p.dp;
+    for (int i = 0; i < (int)kBlock + TAPS - 1; ++i) x[i] = (int)n > i - (TAPS - 1) ? projection<T>(p, (int)t0 + i - (TAPS - 1), pos0, c) : 0.f;
 #pragma unroll
-  for (int i = 0; i < 8; ++i)
-    if (i * 32 < p.dp) o[i * 32 + lane] = y[i] * r;
+    for (int j = 0; j < TAPS; ++j) wr[j] = w[j];
+#pragma unroll
+    for (int t = 0; t < (int)kBlock; ++t) {
+      float a = 0.f;
+#pragma unroll
+      for (int j = 0; j < TAPS; ++j) a = fmaf(x[t + j], wr[j], a);
+      y[t] = t < (int)n ? silu_f(a) : 0.f;
+    }
+  } else {
+#pragma unroll
+    for (int t = 0; t < (int)kBlock; ++t) {
+      float a = 0.f;
+      if (t < (int)n)
+        for (uint32_t j = 0; j < p.ntaps; ++j) a = fmaf(projection<T>(p, (int)(t0 + t + j) - (int)(p.ntaps - 1), pos0, c), w[j], a);
+      y[t] = silu_f(a);
+    }
+  }
+}
+
+// Sums N values over the warp; lane i ends with the sums of values (i * N / 32) ... (N >= 32), or of value i / (32 / N).
+template <int N, int BIT> __device__ __forceinline__ void scatter_sum(float *v, uint32_t lane) {
+  if constexpr (BIT > 0) {
+    const bool up = lane & BIT;
+    if constexpr (N > 1) {
+#pragma unroll
+      for (int i = 0; i < N / 2; ++i) {
+        const float send = up ? v[i] : v[N / 2 + i], keep = up ? v[N / 2 + i] : v[i];
+        v[i] = keep + __shfl_xor_sync(0xffffffffu, send, BIT);
+      }
+      scatter_sum<N / 2, BIT / 2>(v, lane);
+    } else {
+      v[0] += __shfl_xor_sync(0xffffffffu, v[0], BIT);
+      scatter_sum<1, BIT / 2>(v, lane);
+    }
+  }
+}
+
+// A block's record, in floats: P k [8][dp], P q [8][dp], (later decays) k [8][dp], P_8 [dp], M [8][8], N [8][8].
+__host__ __device__ constexpr uint32_t block_floats(uint32_t dp) { return 25 * dp + 128; }
+__device__ __forceinline__ uint32_t pair_a(uint32_t t, uint32_t s) { return s * 7 - s * (s - 1) / 2 + t - s - 1; }   // s < t
+__device__ __forceinline__ uint32_t pair_b(uint32_t t, uint32_t s) { return kPairsA + s * 8 - s * (s - 1) / 2 + t - s; }  // s <= t
+
+// NT threads, one per key channel and one per value channel. first: token of block 0 of this launch.
+template <class T, int TAPS, int NT> __global__ void __launch_bounds__(NT) delta_blocks_kernel(const DeltaRows p, uint32_t first) {
+  constexpr int NW = NT / 32;
+  __shared__ float sums[NW][2 * kBlock], pairs[NW][kPairs], ab[kPairs], minv[kBlock][kBlock], beta_s[kBlock];
+  const uint32_t h = blockIdx.x, t0 = first + blockIdx.y * kBlock, n = min(kBlock, p.T - t0), tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+  const uint32_t kv = h / (p.heads / p.kv_heads), pos0 = *p.pos;
+  float *rec = p.blocks + ((size_t)blockIdx.y * p.heads + h) * block_floats(p.dp);
+  if (tid < kBlock) beta_s[tid] = tid < n ? p.beta[(size_t)(t0 + tid) * p.beta_ld + h] : 0.f;
+  if (tid < p.vp) {
+    float v[kBlock];
+    convolve8<T, TAPS>(p, t0, n, pos0, p.v_col + h * p.vp + tid, v);
+#pragma unroll
+    for (uint32_t t = 0; t < kBlock; ++t)
+      if (t < n) p.v[((size_t)(t0 + t) * p.heads + h) * p.vp + tid] = v[t];
+  }
+  const bool on = tid < p.dp;
+  float q[kBlock], k[kBlock], g[kBlock];
+#pragma unroll
+  for (uint32_t t = 0; t < kBlock; ++t) {
+    q[t] = k[t] = 0.f;
+    g[t] = 1.f;
+  }
+  if (on) {
+    convolve8<T, TAPS>(p, t0, n, pos0, kv * p.dp + tid, q);
+    convolve8<T, TAPS>(p, t0, n, pos0, p.k_col + kv * p.dp + tid, k);
+    const uint32_t c = h * p.dp + tid;
+    const float rate = p.rate[c], bias = p.bias[c];
+#pragma unroll
+    for (uint32_t t = 0; t < kBlock; ++t)
+      if (t < n) g[t] = expf(-rate * softplus_f(p.z[(size_t)(t0 + t) * p.z_ld + c] + bias));
+  }
+  float ss[2 * kBlock];
+#pragma unroll
+  for (uint32_t t = 0; t < kBlock; ++t) {
+    ss[t] = q[t] * q[t];
+    ss[kBlock + t] = k[t] * k[t];
+  }
+  scatter_sum<2 * kBlock, 16>(ss, lane);  // lane: value lane / 2
+  if (!(lane & 1)) sums[warp][lane >> 1] = ss[0];
+  __syncthreads();
+  const float qscale = 1.0f / sqrtf((float)p.dim);
+#pragma unroll
+  for (uint32_t t = 0; t < kBlock; ++t) {
+    float a = 0.f, b = 0.f;
+#pragma unroll
+    for (int w = 0; w < NW; ++w) {
+      a += sums[w][t];
+      b += sums[w][kBlock + t];
+    }
+    q[t] *= 1.0f / sqrtf(a + kUnitEps) * qscale;
+    k[t] *= 1.0f / sqrtf(b + kUnitEps);
+  }
+  if (on) {
+    float d = 1.f;
+#pragma unroll
+    for (uint32_t t = 0; t < kBlock; ++t) {
+      d *= g[t];
+      rec[t * p.dp + tid] = d * k[t];
+      rec[(kBlock + t) * p.dp + tid] = d * q[t];
+    }
+    rec[3 * kBlock * p.dp + tid] = d;
+    d = 1.f;
+#pragma unroll
+    for (int t = kBlock - 1; t >= 0; --t) {
+      rec[(2 * kBlock + t) * p.dp + tid] = d * k[t];
+      d *= g[t];
+    }
+  }
+  float pr[kPairs];
+  int ia = 0, ib = kPairsA;
+#pragma unroll
+  for (int s = 0; s < (int)kBlock; ++s) {
+    float d = k[s];
+    pr[ib++] = d * q[s];
+#pragma unroll
+    for (int t = s + 1; t < (int)kBlock; ++t) {
+      d *= g[t];
+      pr[ia++] = d * k[t];
+      pr[ib++] = d * q[t];
+    }
+  }
+  scatter_sum<kPairs, 16>(pr, lane);  // lane: values 2 lane, 2 lane + 1
+  pairs[warp][2 * lane] = pr[0];
+  pairs[warp][2 * lane + 1] = pr[1];
+  __syncthreads();
+  if (tid < kPairs) {
+    float a = 0.f;
+#pragma unroll
+    for (int w = 0; w < NW; ++w) a += pairs[w][tid];
+    ab[tid] = a;
+  }
+  __syncthreads();
+  float *mn = rec + 25 * p.dp;
+  if (tid < kBlock) {  // column tid of M
+    float m[kBlock];
+#pragma unroll
+    for (int t = 0; t < (int)kBlock; ++t) {
+      float a = t == (int)tid ? 1.f : 0.f;
+#pragma unroll
+      for (int s = 0; s < t; ++s) a = fmaf(-ab[pair_a(t, s)], m[s], a);
+      m[t] = beta_s[t] * a;
+      minv[t][tid] = m[t];
+      mn[t * kBlock + tid] = m[t];
+    }
+  }
+  __syncthreads();
+  if (tid < kBlock * kBlock) {
+    const uint32_t t = tid / kBlock, j = tid % kBlock;
+    float a = 0.f;
+    for (uint32_t s = 0; s <= t; ++s) a = fmaf(ab[pair_b(t, s)], minv[s][j], a);
+    mn[kBlock * kBlock + tid] = a;
+  }
 }
 
 __device__ __forceinline__ void copy16(void *dst, const void *src) {
   asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"((uint32_t)__cvta_generic_to_shared(dst)), "l"(src) : "memory");
 }
-
-constexpr uint32_t kCols = 16, kLanes = 8, kRecThreads = kCols * kLanes;
-constexpr uint32_t kStageTokens = 8, kStages = 3;
-// A stage: [token][q | k | g | v | beta], floats.
-__host__ __device__ constexpr uint32_t rec_token_floats(uint32_t E) { return 3 * E * 32 + kCols + 4; }
-
-// E: 32-element steps of the key width. Lane l of a column holds elements 32 i + 4 l .. + 3, i < E.
-template <int E> __global__ void __launch_bounds__(kRecThreads) delta_recurrence_kernel(const DeltaRows p) {
-  constexpr uint32_t DP = E * 32, TF = rec_token_floats(E);
-  extern __shared__ __align__(16) float stage_mem[];
-  if (p.use_pdl) asm volatile("griddepcontrol.wait;" ::: "memory");
-  const uint32_t h = blockIdx.x, c0 = blockIdx.y * kCols, tid = threadIdx.x, col = tid / kLanes, l = tid % kLanes;
-  const uint32_t kv = h / (p.heads / p.kv_heads), T = p.T;
-  float *state = p.state + ((size_t)h * p.vp + c0 + col) * DP + l * 4;
-  float S[E * 4];
-  if (*p.pos == 0) {
-#pragma unroll
-    for (int i = 0; i < E * 4; ++i) S[i] = 0.f;
+// Two fp32 numbers in one register pair.
+using f2 = unsigned long long;
+__device__ __forceinline__ f2 fma2(f2 a, f2 b, f2 c) {
+  f2 d;
+  asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(d) : "l"(a), "l"(b), "l"(c));
+  return d;
+}
+__device__ __forceinline__ f2 mul2(f2 a, f2 b) {
+  f2 d;
+  asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(d) : "l"(a), "l"(b));
+  return d;
+}
+__device__ __forceinline__ f2 both(float v) {
+  f2 d;
+  asm("mov.b64 %0, {%1, %1};" : "=l"(d) : "f"(v));
+  return d;
+}
+__device__ __forceinline__ float add_halves(f2 a) {
+  float lo, hi;
+  asm("mov.b64 {%0, %1}, %2;" : "=f"(lo), "=f"(hi) : "l"(a));
+  return lo + hi;
+}
+// N consecutive pairs, N = 1 or 2.
+template <int N> __device__ __forceinline__ void load_pairs(const float *p, f2 *o) {
+  if constexpr (N == 2) {
+    const ulonglong2 v = *reinterpret_cast<const ulonglong2 *>(p);
+    o[0] = v.x;
+    o[1] = v.y;
   } else {
-#pragma unroll
-    for (int i = 0; i < E; ++i) {
-      const float4 v = *reinterpret_cast<const float4 *>(state + i * 32);
-      S[4 * i] = v.x; S[4 * i + 1] = v.y; S[4 * i + 2] = v.z; S[4 * i + 3] = v.w;
-    }
+    o[0] = *reinterpret_cast<const f2 *>(p);
   }
-  auto fetch = [&](uint32_t tile) {
-    float *st = stage_mem + (tile % kStages) * kStageTokens * TF;
-    const uint32_t t0 = tile * kStageTokens;
-    constexpr uint32_t V = DP / 4, PER = 3 * V + kCols / 4;  // 16-byte pieces of a token
-    for (uint32_t i = tid; i < kStageTokens * PER; i += kRecThreads) {
-      const uint32_t t = i / PER, x = i % PER, at = t0 + t;
-      if (at >= T) break;
-      float *dst = st + t * TF + x * 4;
-      const float *src;
-      if (x < V) src = p.q + ((size_t)at * p.kv_heads + kv) * DP + x * 4;
-      else if (x < 2 * V) src = p.k + ((size_t)at * p.kv_heads + kv) * DP + (x - V) * 4;
-      else if (x < 3 * V) src = p.g + (size_t)at * p.g_ld + h * DP + (x - 2 * V) * 4;
-      else src = p.v + ((size_t)at * p.heads + h) * p.vp + c0 + (x - 3 * V) * 4;
-      copy16(dst, src);
-    }
-    if (tid < kStageTokens && t0 + tid < T) {
-      const uint32_t dst = (uint32_t)__cvta_generic_to_shared(st + tid * TF + 3 * DP + kCols);
-      asm volatile("cp.async.ca.shared.global [%0], [%1], 4;" ::"r"(dst), "l"(p.beta + (size_t)(t0 + tid) * p.beta_ld + h) : "memory");
-    }
-  };
-  const uint32_t tiles = (T + kStageTokens - 1) / kStageTokens;
-  for (uint32_t i = 0; i < kStages - 1; ++i) {
-    if (i < tiles) fetch(i);
-    asm volatile("cp.async.commit_group;" ::: "memory");
-  }
-  for (uint32_t tile = 0; tile < tiles; ++tile) {
-    asm volatile("cp.async.wait_group %0;" ::"n"(kStages - 2) : "memory");
-    __syncthreads();  // this stage has landed for everyone, the one before is consumed
-    if (tile + kStages - 1 < tiles) fetch(tile + kStages - 1);
-    asm volatile("cp.async.commit_group;" ::: "memory");
-    const float *st = stage_mem + (tile % kStages) * kStageTokens * TF;
-    const uint32_t n = min(kStageTokens, T - tile * kStageTokens);
-    for (uint32_t t = 0; t < n; ++t, st += TF) {
-      float k[E * 4], a = 0.f, b = 0.f;
-#pragma unroll
-      for (int i = 0; i < E; ++i) {
-        const float4 kk = *reinterpret_cast<const float4 *>(st + DP + i * 32 + l * 4), g = *reinterpret_cast<const float4 *>(st + 2 * DP + i * 32 + l * 4);
-        k[4 * i] = kk.x; k[4 * i + 1] = kk.y; k[4 * i + 2] = kk.z; k[4 * i + 3] = kk.w;
-        S[4 * i] *= g.x; S[4 * i + 1] *= g.y; S[4 * i + 2] *= g.z; S[4 * i + 3] *= g.w;
-        a = fmaf(S[4 * i], kk.x, a);
-        b = fmaf(S[4 * i + 1], kk.y, b);
-        a = fmaf(S[4 * i + 2], kk.z, a);
-        b = fmaf(S[4 * i + 3], kk.w, b);
-      }
-      a += b;
-#pragma unroll
-      for (uint32_t o = 1; o < kLanes; o <<= 1) a += __shfl_xor_sync(0xffffffffu, a, o);
-      const float u = st[3 * DP + kCols] * (st[3 * DP + col] - a);
-      float y = 0.f, z = 0.f;
-#pragma unroll
-      for (int i = 0; i < E; ++i) {
-        const float4 q = *reinterpret_cast<const float4 *>(st + i * 32 + l * 4);
-        S[4 * i] = fmaf(k[4 * i], u, S[4 * i]);
-        S[4 * i + 1] = fmaf(k[4 * i + 1], u, S[4 * i + 1]);
-        S[4 * i + 2] = fmaf(k[4 * i + 2], u, S[4 * i + 2]);
-        S[4 * i + 3] = fmaf(k[4 * i + 3], u, S[4 * i + 3]);
-        y = fmaf(S[4 * i], q.x, y);
-        z = fmaf(S[4 * i + 1], q.y, z);
-        y = fmaf(S[4 * i + 2], q.z, y);
-        z = fmaf(S[4 * i + 3], q.w, z);
-      }
-      y += z;
-#pragma unroll
-      for (uint32_t o = 1; o < kLanes; o <<= 1) y += __shfl_xor_sync(0xffffffffu, y, o);
-      if (l == 0) p.v[((size_t)(tile * kStageTokens + t) * p.heads + h) * p.vp + c0 + col] = y;
-    }
-  }
-#pragma unroll
-  for (int i = 0; i < E; ++i) *reinterpret_cast<float4 *>(state + i * 32) = make_float4(S[4 * i], S[4 * i + 1], S[4 * i + 2], S[4 * i + 3]);
-  if (p.use_pdl) asm volatile("griddepcontrol.launch_dependents;");
+}
+template <int N> __device__ __forceinline__ void store_pairs(float *p, const f2 *o) {
+  if constexpr (N == 2) *reinterpret_cast<ulonglong2 *>(p) = make_ulonglong2(o[0], o[1]);
+  else *reinterpret_cast<f2 *>(p) = o[0];
 }
 
-template <class T> __global__ void __launch_bounds__(kThreads) delta_finish_kernel(const DeltaRows p) {
-  if (p.use_pdl) asm volatile("griddepcontrol.wait;" ::: "memory");
-  const uint32_t m = blockIdx.x, lane = threadIdx.x & 31, h = blockIdx.y * kWarps + (threadIdx.x >> 5);
+constexpr uint32_t kScanLanes = 16, kScanCols = 4, kScanThreads = 128, kCtaCols = kScanThreads / kScanLanes * kScanCols, kStages = 3;
+
+// Sums over 16 lanes of [token][column]; lane l ends with token l / 2, columns 2 (l % 2) and the next.
+__device__ __forceinline__ float2 scatter_tokens(const f2 (&acc)[kBlock][kScanCols], uint32_t l) {
+  float a[kBlock * kScanCols];
+#pragma unroll
+  for (int t = 0; t < (int)kBlock; ++t)
+#pragma unroll
+    for (int c = 0; c < (int)kScanCols; ++c) a[t * kScanCols + c] = add_halves(acc[t][c]);
+  scatter_sum<kBlock * kScanCols, 8>(a, l);
+  return make_float2(a[0], a[1]);
+}
+
+// E: 32-element steps of the key width. Lane l holds elements (16 i + l) V .. + V - 1 of each of its columns.
+template <int E> __global__ void __launch_bounds__(kScanThreads) delta_scan_kernel(const DeltaRows p, uint32_t first, uint32_t count) {
+  constexpr uint32_t DP = E * 32, RF = block_floats(DP);
+  constexpr int V = E % 2 ? 2 : 4, NV = 2 * E / V, NP = V / 2;
+  extern __shared__ __align__(16) float stage_mem[];
+  const uint32_t h = blockIdx.x, tid = threadIdx.x, lane = tid & 31, l = lane % kScanLanes;
+  const uint32_t c0 = blockIdx.y * kCtaCols + tid / kScanLanes * kScanCols, blocks = (count + kBlock - 1) / kBlock;
+  const bool active = c0 < p.vp;  // uniform over a warp: vp is a multiple of 16
+  float *state = p.state + ((size_t)h * p.vp + c0) * DP;
+  f2 S[kScanCols][E];
+  const bool fresh = first == 0 && *p.pos == 0;
+#pragma unroll
+  for (int c = 0; c < (int)kScanCols; ++c)
+#pragma unroll
+    for (int i = 0; i < NV; ++i) {
+#pragma unroll
+      for (int j = 0; j < NP; ++j) S[c][i * NP + j] = 0;
+      if (active && !fresh) load_pairs<NP>(state + c * DP + (i * kScanLanes + l) * V, &S[c][i * NP]);
+    }
+  const float *recs = p.blocks + (size_t)h * RF;
+  auto fetch = [&](uint32_t b) {
+    float *st = stage_mem + (b % kStages) * RF;
+    const float *src = recs + (size_t)b * p.heads * RF;
+    for (uint32_t i = tid * 4; i < RF; i += kScanThreads * 4) copy16(st + i, src + i);
+  };
+  const uint32_t tok = l >> 1;
+  float *vrow = p.v + ((size_t)(first + tok) * p.heads + h) * p.vp + c0 + 2 * (l & 1);
+  const size_t vstep = (size_t)kBlock * p.heads * p.vp;
+  auto value = [&](uint32_t b) {
+    return active && b * kBlock + tok < count ? *reinterpret_cast<const float2 *>(vrow + b * vstep) : make_float2(0.f, 0.f);
+  };
+  for (uint32_t i = 0; i < kStages - 1; ++i) {
+    if (i < blocks) fetch(i);
+    asm volatile("cp.async.commit_group;" ::: "memory");
+  }
+  float2 vnext = value(0);
+  for (uint32_t b = 0; b < blocks; ++b) {
+    asm volatile("cp.async.wait_group %0;" ::"n"(kStages - 2) : "memory");
+    __syncthreads();  // this stage has landed for everyone, the one before is consumed
+    if (b + kStages - 1 < blocks) fetch(b + kStages - 1);
+    asm volatile("cp.async.commit_group;" ::: "memory");
+    const float2 v = vnext;
+    if (b + 1 < blocks) vnext = value(b + 1);
+    if (!active) continue;
+    const float *st = stage_mem + (b % kStages) * RF, *mn = st + 25 * DP + tok * kBlock;
+    auto dots = [&](const float *rows) {
+      f2 acc[kBlock][kScanCols];
+#pragma unroll
+      for (int t = 0; t < (int)kBlock; ++t)
+#pragma unroll
+        for (int c = 0; c < (int)kScanCols; ++c) acc[t][c] = 0;
+#pragma unroll
+      for (int i = 0; i < NV; ++i)
+#pragma unroll
+        for (int t = 0; t < (int)kBlock; ++t) {
+          f2 x[NP];
+          load_pairs<NP>(rows + t * DP + (i * kScanLanes + l) * V, x);
+#pragma unroll
+          for (int j = 0; j < NP; ++j)
+#pragma unroll
+            for (int c = 0; c < (int)kScanCols; ++c) acc[t][c] = fma2(S[c][i * NP + j], x[j], acc[t][c]);
+        }
+      return scatter_tokens(acc, l);
+    };
+    const float2 a = dots(st);
+    float2 o = dots(st + kBlock * DP);
+    const float2 w = make_float2(v.x - a.x, v.y - a.y);
+    float2 u = make_float2(0.f, 0.f);
+#pragma unroll
+    for (int s = 0; s < (int)kBlock; ++s) {
+      const float wx = __shfl_sync(0xffffffffu, w.x, 2 * s + (l & 1), kScanLanes), wy = __shfl_sync(0xffffffffu, w.y, 2 * s + (l & 1), kScanLanes);
+      const float m = mn[s], n = mn[kBlock * kBlock + s];
+      u.x = fmaf(m, wx, u.x);
+      u.y = fmaf(m, wy, u.y);
+      o.x = fmaf(n, wx, o.x);
+      o.y = fmaf(n, wy, o.y);
+    }
+    if (b * kBlock + tok < count) *reinterpret_cast<float2 *>(vrow + b * vstep) = o;
+#pragma unroll
+    for (int i = 0; i < NV; ++i) {
+      f2 x[NP];
+      load_pairs<NP>(st + 3 * kBlock * DP + (i * kScanLanes + l) * V, x);
+#pragma unroll
+      for (int j = 0; j < NP; ++j)
+#pragma unroll
+        for (int c = 0; c < (int)kScanCols; ++c) S[c][i * NP + j] = mul2(S[c][i * NP + j], x[j]);
+    }
+#pragma unroll
+    for (int s = 0; s < (int)kBlock; ++s) {
+      f2 us[kScanCols];
+#pragma unroll
+      for (int c = 0; c < (int)kScanCols; ++c) us[c] = both(__shfl_sync(0xffffffffu, c & 1 ? u.y : u.x, 2 * s + (c >> 1), kScanLanes));
+#pragma unroll
+      for (int i = 0; i < NV; ++i) {
+        f2 x[NP];
+        load_pairs<NP>(st + (2 * kBlock + s) * DP + (i * kScanLanes + l) * V, x);
+#pragma unroll
+        for (int j = 0; j < NP; ++j)
+#pragma unroll
+          for (int c = 0; c < (int)kScanCols; ++c) S[c][i * NP + j] = fma2(x[j], us[c], S[c][i * NP + j]);
+      }
+    }
+  }
+  if (!active) return;
+#pragma unroll
+  for (int c = 0; c < (int)kScanCols; ++c)
+#pragma unroll
+    for (int i = 0; i < NV; ++i) store_pairs<NP>(state + c * DP + (i * kScanLanes + l) * V, &S[c][i * NP]);
+}
+
+constexpr int kFinishThreads = 256;
+template <class T> __global__ void __launch_bounds__(kFinishThreads) delta_finish_kernel(const DeltaRows p) {
+  const uint32_t m = blockIdx.x, lane = threadIdx.x & 31, h = blockIdx.y * (kFinishThreads / 32) + (threadIdx.x >> 5);
   if (m + p.ntaps >= p.T) {  // one of the last ntaps tokens: later ones look back at it
     const T *src = static_cast<const T *>(p.raw) + (size_t)m * p.raw_ld;
     T *dst = static_cast<T *>(p.ring) + (size_t)((*p.pos + m) % p.ntaps) * p.raw_ld;
-    for (uint32_t c = blockIdx.y * kThreads + threadIdx.x; c < p.raw_ld; c += gridDim.y * kThreads) dst[c] = src[c];
+    for (uint32_t c = blockIdx.y * kFinishThreads + threadIdx.x; c < p.raw_ld; c += gridDim.y * kFinishThreads) dst[c] = src[c];
   }
-  if (h >= p.heads) return;
-  const float *o = p.v + ((size_t)m * p.heads + h) * p.vp;
-  float y[8], ss = 0.f;
+  if (h >= p.heads || lane * 8 >= p.vp) return;  // a lane holds eight columns
+  const uint32_t lanes = 0xffffffffu >> (32 - p.vp / 8);
+  float y[8], z[8], w[8], ss = 0.f;
+  load8(p.v + ((size_t)m * p.heads + h) * p.vp + lane * 8, y);  // padded columns are zero
+  load8(p.z + (size_t)m * p.z_ld + p.z_gate + h * p.vp + lane * 8, z);
+  load8(p.norm + lane * 8, w);
 #pragma unroll
-  for (int i = 0; i < 8; ++i) {
-    const uint32_t d = i * 32 + lane;
-    y[i] = d < p.vp ? o[d] : 0.f;  // padded columns are zero
-    ss = fmaf(y[i], y[i], ss);
-  }
-  ss = warp_sum(ss);
-  const float r = 1.0f / sqrtf(ss / (float)p.vdim + p.eps);
+  for (int i = 0; i < 8; ++i) ss = fmaf(y[i], y[i], ss);
+  float tot = 0.f;
+  for (uint32_t i = 0; i < p.vp / 8; ++i) tot += __shfl_sync(lanes, ss, i);
+  const float r = 1.0f / sqrtf(tot / (float)p.vdim + p.eps);
 #pragma unroll
-  for (int i = 0; i < 8; ++i) {
-    const uint32_t d = i * 32 + lane;
-    if (d < p.vp) store1(static_cast<T *>(p.out) + (size_t)m * p.out_ld + h * p.vp + d, y[i] * r * p.norm[d] * p.gate[(size_t)m * p.gate_ld + h * p.vp + d]);
-  }
+  for (int i = 0; i < 8; ++i) y[i] *= r * w[i] * sigmoid_f(z[i]);
+  store8(static_cast<T *>(p.out) + (size_t)m * p.out_ld + h * p.vp + lane * 8, y);
 }
 
-cudaError_t launch(void (*kern)(const DeltaRows), const DeltaRows &p, dim3 grid, uint32_t threads, size_t smem, cudaStream_t s) {
-  cudaLaunchConfig_t cfg = {};
-  cfg.gridDim = grid;
-  cfg.blockDim = dim3(threads);
-  cfg.dynamicSmemBytes = smem;
-  cfg.stream = s;
-  cudaLaunchAttribute attr[1];
-  attr[0].id = cudaLaunchAttributeProgrammaticStreamSerialization;
-  attr[0].val.programmaticStreamSerializationAllowed = 1;
-  cfg.attrs = attr;
-  cfg.numAttrs = p.use_pdl ? 1 : 0;
-  return cudaLaunchKernelEx(&cfg, kern, p);
-}
+// ---- one token ----
+constexpr uint32_t kStepThreads = 256, kStepCols = 32, kStepLanes = 8, kRowGroups = kStepThreads / 8, kAhead = 10;
 
-template <int E> cudaError_t launch_recurrence(const DeltaRows &p, cudaStream_t s) {
-  constexpr size_t smem = (size_t)kStages * kStageTokens * rec_token_floats(E) * sizeof(float);
-  if (cudaError_t e = cudaFuncSetAttribute(delta_recurrence_kernel<E>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem)) return e;
-  return launch(delta_recurrence_kernel<E>, p, dim3(p.heads, p.vp / kCols), kRecThreads, smem, s);
+// grid: heads x cluster; a cluster is a head, a CTA 32 of its columns. E: 32-element steps of the key width.
+template <class T, int E> __global__ void __launch_bounds__(kStepThreads) delta_step_kernel(const DeltaRows p, uint32_t cluster) {
+  constexpr uint32_t DP = E * 32;
+  __shared__ float q_s[DP], k_s[DP], g_s[DP], v_s[kStepCols], gate_s[kStepCols], part[kStepThreads / 32], peers[8];
+  const uint32_t h = blockIdx.x / cluster, rank = blockIdx.x % cluster, tid = threadIdx.x, lane = tid & 31, col = tid / kStepLanes, l = tid % kStepLanes;
+  const uint32_t kv = h / (p.heads / p.kv_heads), c0 = rank * kStepCols, cols = c0 < p.vp ? min(kStepCols, p.vp - c0) : 0u;
+  const bool active = col < cols;
+  if (cluster > 1) asm volatile("barrier.cluster.arrive.relaxed.aligned;" ::: "memory");  // waited for before another CTA's memory is touched
+  // Rows of the projections' second steps, 8 lanes each: DP decays, then this CTA's gates. The first ones, and the
+  // state, do not depend on the kernel before.
+  const uint32_t rows = DP + cols, steps = p.low_ld / 64, items = (rows + kRowGroups - 1) / kRowGroups * steps;
+  auto item_row = [&](uint32_t i) { return i / steps * kRowGroups + col; };
+  auto item_weights = [&](uint32_t i, uint32_t row) {
+    const size_t r = row < DP ? (size_t)h * DP + row : (size_t)p.z_gate + h * p.vp + c0 + row - DP;
+    return p.wl + r * p.low_ld + i % steps * 64 + l * 8;
+  };
+  uint4 wa[kAhead];
+#pragma unroll
+  for (uint32_t i = 0; i < kAhead; ++i) {
+    wa[i] = make_uint4(0, 0, 0, 0);
+    if (i < items && item_row(i) < rows) wa[i] = ldg_stream(item_weights(i, item_row(i)));
+  }
+  float4 S[E];
+  float *state = p.state + ((size_t)h * p.vp + c0 + col) * DP + l * 4;
+  const uint32_t pos = *p.pos;
+#pragma unroll
+  for (int i = 0; i < E; ++i) S[i] = active && pos ? *reinterpret_cast<const float4 *>(state + i * 32) : make_float4(0.f, 0.f, 0.f, 0.f);
+  if (p.use_pdl) asm volatile("griddepcontrol.wait;" ::: "memory");
+  // convolution: query and key channels, this CTA's value channels
+  for (uint32_t i = tid; i < 2 * DP + cols; i += kStepThreads) {
+    const uint32_t c = i < DP ? kv * DP + i : i < 2 * DP ? p.k_col + kv * DP + i - DP : p.v_col + h * p.vp + c0 + i - 2 * DP;
+    const T *cur = static_cast<const T *>(p.raw) + c;
+    float a = 0.f;
+    for (uint32_t j = 0; j < p.ntaps; ++j) a = fmaf(projection<T>(p, (int)j - (int)(p.ntaps - 1), pos, c), p.taps[(size_t)c * p.ntaps + j], a);
+    a = silu_f(a);
+    if (i < DP) q_s[i] = a;
+    else if (i < 2 * DP) k_s[i - DP] = a;
+    else v_s[i - 2 * DP] = a;
+    // the slot of this position is read by no one in this step; heads that share a key head write the same number
+    static_cast<T *>(p.ring)[(size_t)(pos % p.ntaps) * p.raw_ld + c] = *cur;
+  }
+  auto finish_row = [&](uint32_t row, float z) {
+#pragma unroll
+    for (uint32_t o = 1; o < 8; o <<= 1) z += __shfl_xor_sync(0xffffffffu, z, o);
+    if (l || row >= rows) return;
+    if (row < DP) g_s[row] = expf(-p.rate[h * DP + row] * softplus_f(z + p.bias[h * DP + row]));
+    else gate_s[row - DP] = sigmoid_f(z);
+  };
+  auto dot8 = [&](uint32_t i, uint32_t row, const uint4 &w) {
+    float wf[8], x[8], a = 0.f;
+    unpack8(w, wf);
+    load8(static_cast<const T *>(p.low) + (row < DP ? 0u : p.low_ld) + i % steps * 64 + l * 8, x);
+#pragma unroll
+    for (int e = 0; e < 8; ++e) a = fmaf(wf[e], x[e], a);
+    return a;
+  };
+  float z = 0.f;
+#pragma unroll
+  for (uint32_t i = 0; i < kAhead; ++i) {
+    if (i >= items) break;
+    const uint32_t row = item_row(i);
+    if (row < rows) z += dot8(i, row, wa[i]);
+    if (i % steps == steps - 1) {
+      finish_row(row, z);
+      z = 0.f;
+    }
+  }
+  for (uint32_t i = kAhead; i < items; ++i) {
+    const uint32_t row = item_row(i);
+    if (row < rows) z += dot8(i, row, ldg_stream(item_weights(i, row)));
+    if (i % steps == steps - 1) {
+      finish_row(row, z);
+      z = 0.f;
+    }
+  }
+  __syncthreads();
+  if (p.use_pdl) asm volatile("griddepcontrol.launch_dependents;");
+  float qq = 0.f, kk = 0.f;  // every warp for itself
+#pragma unroll
+  for (int i = 0; i < E; ++i) {
+    qq = fmaf(q_s[i * 32 + lane], q_s[i * 32 + lane], qq);
+    kk = fmaf(k_s[i * 32 + lane], k_s[i * 32 + lane], kk);
+  }
+  const float rq = 1.0f / sqrtf(warp_sum(qq) + kUnitEps) / sqrtf((float)p.dim), rk = 1.0f / sqrtf(warp_sum(kk) + kUnitEps);
+  float a = 0.f, o = 0.f;
+  float4 k[E];
+#pragma unroll
+  for (int i = 0; i < E; ++i) {
+    const float4 g = *reinterpret_cast<const float4 *>(g_s + i * 32 + l * 4), x = *reinterpret_cast<const float4 *>(k_s + i * 32 + l * 4);
+    k[i] = make_float4(x.x * rk, x.y * rk, x.z * rk, x.w * rk);
+    S[i] = make_float4(S[i].x * g.x, S[i].y * g.y, S[i].z * g.z, S[i].w * g.w);
+    a = fmaf(S[i].x, k[i].x, fmaf(S[i].y, k[i].y, fmaf(S[i].z, k[i].z, fmaf(S[i].w, k[i].w, a))));
+  }
+#pragma unroll
+  for (uint32_t x = 1; x < kStepLanes; x <<= 1) a += __shfl_xor_sync(0xffffffffu, a, x);
+  const float u = active ? p.beta[h] * (v_s[col] - a) : 0.f;
+#pragma unroll
+  for (int i = 0; i < E; ++i) {
+    const float4 x = *reinterpret_cast<const float4 *>(q_s + i * 32 + l * 4);
+    S[i] = make_float4(fmaf(k[i].x, u, S[i].x), fmaf(k[i].y, u, S[i].y), fmaf(k[i].z, u, S[i].z), fmaf(k[i].w, u, S[i].w));
+    o = fmaf(S[i].x, x.x, fmaf(S[i].y, x.y, fmaf(S[i].z, x.z, fmaf(S[i].w, x.w, o))));
+    if (active) *reinterpret_cast<float4 *>(state + i * 32) = S[i];
+  }
+#pragma unroll
+  for (uint32_t x = 1; x < kStepLanes; x <<= 1) o += __shfl_xor_sync(0xffffffffu, o, x);
+  o *= rq;
+  const float ss = warp_sum(active && l == 0 ? o * o : 0.f);
+  if (lane == 0) part[tid >> 5] = ss;
+  __syncthreads();
+  float tot = 0.f;
+#pragma unroll
+  for (uint32_t w = 0; w < kStepThreads / 32; ++w) tot += part[w];
+  if (cluster > 1) {
+    cg::cluster_group cl = cg::this_cluster();
+    asm volatile("barrier.cluster.wait.aligned;" ::: "memory");
+    if (tid < cluster) *cl.map_shared_rank(&peers[rank], tid) = tot;
+    cl.sync();
+    tot = 0.f;
+    for (uint32_t i = 0; i < cluster; ++i) tot += peers[i];
+  }
+  if (active && l == 0) {
+    const float y = o / sqrtf(tot / (float)p.vdim + p.eps) * p.norm[c0 + col] * gate_s[col];
+    store1(static_cast<T *>(p.out) + h * p.vp + c0 + col, y);
+  }
 }
 
 bool sane(const DeltaRows &p) {
-  return p.T && p.heads && p.kv_heads && p.heads % p.kv_heads == 0 && p.ntaps && p.dp % 32 == 0 && p.dp <= 256 && p.vp % kCols == 0 && p.vp <= 256 && p.g_ld % 4 == 0;
+  return p.T && p.heads && p.kv_heads && p.heads % p.kv_heads == 0 && p.ntaps && p.dp % 32 == 0 && p.dp && p.dp <= 256 && p.vp % 16 == 0 && p.vp && p.vp <= 256;
+}
+
+template <class T, int TAPS> cudaError_t launch_blocks(const DeltaRows &p, uint32_t first, uint32_t count, cudaStream_t s) {
+  const dim3 grid(p.heads, (count + kBlock - 1) / kBlock);
+  if (std::max(p.dp, p.vp) <= 128) delta_blocks_kernel<T, TAPS, 128><<<grid, 128, 0, s>>>(p, first);
+  else delta_blocks_kernel<T, TAPS, 256><<<grid, 256, 0, s>>>(p, first);
+  return cudaGetLastError();
+}
+template <int E> cudaError_t launch_scan(const DeltaRows &p, uint32_t first, uint32_t count, cudaStream_t s) {
+  constexpr size_t smem = (size_t)kStages * block_floats(E * 32) * sizeof(float);
+  if (cudaError_t e = cudaFuncSetAttribute(delta_scan_kernel<E>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem)) return e;
+  delta_scan_kernel<E><<<dim3(p.heads, (p.vp + kCtaCols - 1) / kCtaCols), kScanThreads, smem, s>>>(p, first, count);
+  return cudaGetLastError();
+}
+// f<E>() for a key width of 32 E.
+template <class F> cudaError_t by_width(uint32_t dp, F f) {
+  switch (dp / 32) {
+    case 1: return f(std::integral_constant<int, 1>());
+    case 2: return f(std::integral_constant<int, 2>());
+    case 3: return f(std::integral_constant<int, 3>());
+    case 4: return f(std::integral_constant<int, 4>());
+    case 5: return f(std::integral_constant<int, 5>());
+    case 6: return f(std::integral_constant<int, 6>());
+    case 7: return f(std::integral_constant<int, 7>());
+    default: return f(std::integral_constant<int, 8>());
+  }
+}
+template <class T, int E> cudaError_t launch_step(const DeltaRows &p, cudaStream_t s) {
+  uint32_t cluster = 1;
+  while (cluster * kStepCols < p.vp) cluster *= 2;  // at most 8
+  cudaLaunchConfig_t cfg = {};
+  cfg.gridDim = dim3(p.heads * cluster);
+  cfg.blockDim = dim3(kStepThreads);
+  cfg.stream = s;
+  cudaLaunchAttribute attr[2];
+  attr[0].id = cudaLaunchAttributeClusterDimension;
+  attr[0].val.clusterDim.x = cluster;
+  attr[0].val.clusterDim.y = attr[0].val.clusterDim.z = 1;
+  attr[1].id = cudaLaunchAttributeProgrammaticStreamSerialization;
+  attr[1].val.programmaticStreamSerializationAllowed = 1;
+  cfg.attrs = attr;
+  cfg.numAttrs = p.use_pdl ? 2 : 1;
+  return cudaLaunchKernelEx(&cfg, delta_step_kernel<T, E>, p, cluster);
 }
 
 }  // namespace
 
-cudaError_t launch_delta_prepare(const DeltaRows &p, bool f32, cudaStream_t s) {
-  if (!sane(p)) return cudaErrorInvalidValue;
-  const dim3 grid(p.T, (2 * p.kv_heads + p.heads + kWarps - 1) / kWarps);
-  return launch(f32 ? delta_prepare_kernel<float> : delta_prepare_kernel<bf16>, p, grid, kThreads, 0, s);
+size_t delta_block_floats(uint32_t T, uint32_t heads, uint32_t dp) {
+  return (size_t)((std::min(T, kDeltaSlice) + kBlock - 1) / kBlock) * heads * block_floats(dp);
 }
 
-cudaError_t launch_delta_recurrence(const DeltaRows &p, cudaStream_t s) {
-  if (!sane(p)) return cudaErrorInvalidValue;
-  switch (p.dp / 32) {
-    case 1: return launch_recurrence<1>(p, s);
-    case 2: return launch_recurrence<2>(p, s);
-    case 3: return launch_recurrence<3>(p, s);
-    case 4: return launch_recurrence<4>(p, s);
-    case 5: return launch_recurrence<5>(p, s);
-    case 6: return launch_recurrence<6>(p, s);
-    case 7: return launch_recurrence<7>(p, s);
-    default: return launch_recurrence<8>(p, s);
+cudaError_t launch_delta_rows(const DeltaRows &p, bool f32, cudaStream_t s) {
+  if (!sane(p) || p.z_ld % 8 || p.z_gate % 8) return cudaErrorInvalidValue;
+  for (uint32_t first = 0; first < p.T; first += kDeltaSlice) {
+    const uint32_t count = std::min(kDeltaSlice, p.T - first);
+    cudaError_t e = f32 ? (p.ntaps == 4 ? launch_blocks<float, 4>(p, first, count, s) : launch_blocks<float, 0>(p, first, count, s))
+                        : (p.ntaps == 4 ? launch_blocks<bf16, 4>(p, first, count, s) : launch_blocks<bf16, 0>(p, first, count, s));
+    if (e == cudaSuccess) e = by_width(p.dp, [&](auto w) { return launch_scan<decltype(w)::value>(p, first, count, s); });
+    if (e != cudaSuccess) return e;
   }
+  const dim3 grid(p.T, (p.heads + kFinishThreads / 32 - 1) / (kFinishThreads / 32));
+  if (f32) delta_finish_kernel<float><<<grid, kFinishThreads, 0, s>>>(p);
+  else delta_finish_kernel<bf16><<<grid, kFinishThreads, 0, s>>>(p);
+  return cudaGetLastError();
 }
 
-cudaError_t launch_delta_finish(const DeltaRows &p, bool f32, cudaStream_t s) {
-  if (!sane(p)) return cudaErrorInvalidValue;
-  const dim3 grid(p.T, (p.heads + kWarps - 1) / kWarps);
-  return launch(f32 ? delta_finish_kernel<float> : delta_finish_kernel<bf16>, p, grid, kThreads, 0, s);
+cudaError_t launch_delta_step(const DeltaRows &p, bool f32, cudaStream_t s) {
+  if (!sane(p) || p.T != 1 || p.low_ld % 64) return cudaErrorInvalidValue;
+  return by_width(p.dp, [&](auto w) { return f32 ? launch_step<float, decltype(w)::value>(p, s) : launch_step<bf16, decltype(w)::value>(p, s); });
 }
 
 }  // namespace vkl

@@ -106,14 +106,6 @@ template <class T> __device__ __forceinline__ void rows_chunk(const RowsOut &o, 
       for (int j = 0; j < 32; j += 8) store8(p + j, v + j);
       break;
     }
-    case ROW_DECAY: {
-      float *p = o.f32 + (size_t)m * o.f32_ld + c0;
-#pragma unroll
-      for (int j = 0; j < 32; ++j) v[j] = expf(-__ldg(o.rate + n0 + j) * softplus_f(v[j]));
-#pragma unroll
-      for (int j = 0; j < 32; j += 8) store8(p + j, v + j);
-      break;
-    }
     case ROW_NONE: break;
     case ROW_HEAD_GATE: {
       float *p = o.gate + (size_t)m * o.gate_ld + c0;
@@ -184,7 +176,6 @@ template <class T> __device__ __forceinline__ void rows_one(const RowsOut &o, co
       if (c < o.kv_heads * o.vp) store1(cache_slot<T>(o.vcache, o.vp, o.maxlen, *o.pos, c), v);
       break;
     case ROW_LOW: store1(low_slot<T>(o, 0, c), v); break;
-    case ROW_DECAY: o.f32[c] = expf(-o.rate[n] * softplus_f(v)); break;
     case ROW_NONE: break;
     case ROW_HEAD_GATE: o.gate[c] = sigmoid_f(v); break;
     case ROW_RESIDUAL: finish_residual<T>(o.res, 0, n, o.res.x[n] + o.res.mult * (v + (o.res.bias ? o.res.bias[n] : 0.f))); break;

@@ -24,7 +24,6 @@ enum RowKind : uint32_t {
   ROW_STORE,      // * scale, then the soft cap if there is one -> f32 [tokens, f32_ld]
   ROW_VALUE,      // this token's row of the value cache [kv head][position][vp]
   ROW_LOW,        // low_ld rows each of two low-rank inner vectors -> low [2][tokens, low_ld]
-  ROW_DECAY,      // exp(-rate softplus(. + bias)), the decay of a recurrent state's key channel -> f32
   ROW_NONE        // padding between two segments: no result
 };
 enum GluAct : uint32_t {
@@ -66,7 +65,6 @@ struct RowsOut {
   void *low;
   uint32_t low_ld;
   size_t low_stride;    // elements between the two inner vectors of token 0
-  const float *rate;    // ROW_DECAY: per row
   float *gate;
   uint32_t gate_ld;
   void *glu;
@@ -191,8 +189,9 @@ struct QkRows {
 cudaError_t launch_qk_rows(const QkRows &p, bool f32, cudaStream_t s);
 
 // ---- gated delta rule with a decay per key channel (delta_rule.cu) ----
-// Per head a state S [dim, vdim]: S <- g S, u = beta (v - S^T k), S <- S + k u^T, o = S^T q. Query, key and value
-// are projections after a short causal convolution over time and SiLU; query and key are unit vectors.
+// Per head a state S [dim, vdim]: S <- g S, u = beta (v - S^T k), S <- S + k u^T, o = S^T q, then the RMS norm of o and
+// a gate. Query, key and value are projections after a short causal convolution over time and SiLU, query and key unit
+// vectors; decay and gate come from two-step projections, g = exp(-rate softplus(z + bias)), gate = sigmoid(z).
 struct DeltaRows {
   const void *raw;          // [T, raw_ld] compute type: the projections, query | key | value columns
   uint32_t raw_ld, k_col, v_col;
@@ -201,24 +200,30 @@ struct DeltaRows {
   void *ring;               // [ntaps][raw_ld] compute type: the projections at position p in slot p % ntaps
   const uint32_t *pos;      // position of row 0; a sequence that starts at 0 finds state and ring empty
   uint32_t T, heads, kv_heads, dim, vdim, dp, vp;  // dp, vp: widths in memory, multiples of 32 and 16
-  float *q, *k;             // [T][kv_heads * dp]: after convolution and norm
-  float *v;                 // [T][heads * vp]: values, which the recurrence replaces by its outputs
-  const float *g;           // [T, g_ld]: decays, head h at column h * dp
-  uint32_t g_ld;
+  const float *bias, *rate; // [heads * dp]
   const float *beta;        // [T, beta_ld]
   uint32_t beta_ld;
   float *state;             // [heads][vp][dp]
   const float *norm;        // [vp]: weight of the output's RMS norm per head
   float eps;
-  const float *gate;        // [T, gate_ld], head h at column h * vp
-  uint32_t gate_ld;
   void *out;                // [T, out_ld] compute type, head h at column h * vp
   uint32_t out_ld;
   int use_pdl;
+  // many tokens
+  const float *z;           // [T, z_ld]: second steps of the projections, decays from column 0, gates from column z_gate
+  uint32_t z_ld, z_gate;
+  float *v;                 // [T][heads * vp]: values, which the recurrence replaces by its outputs
+  float *blocks;            // delta_block_floats(...): what the recurrence needs of the keys, block by block
+  // one token
+  const bf16 *wl;           // second steps' weights [., low_ld]: decay rows from 0, gate rows from z_gate
+  const void *low;          // [2][low_ld] compute type: the first steps' results
+  uint32_t low_ld;
 };
-cudaError_t launch_delta_prepare(const DeltaRows &p, bool f32, cudaStream_t s);     // raw -> q, k, v
-cudaError_t launch_delta_recurrence(const DeltaRows &p, cudaStream_t s);            // q, k, v, g, beta, state -> v, state
-cudaError_t launch_delta_finish(const DeltaRows &p, bool f32, cudaStream_t s);      // v, gate -> out; raw -> ring
+constexpr uint32_t kDeltaSlice = 1024;  // tokens whose blocks are held at a time
+size_t delta_block_floats(uint32_t T, uint32_t heads, uint32_t dp);
+cudaError_t launch_delta_rows(const DeltaRows &p, bool f32, cudaStream_t s);  // T > 1; launches: delta_launches(T)
+inline uint32_t delta_launches(uint32_t T) { return 2 * ((T + kDeltaSlice - 1) / kDeltaSlice) + 1; }
+cudaError_t launch_delta_step(const DeltaRows &p, bool f32, cudaStream_t s);  // T = 1
 
 // Places a bf16 tensor [rows, cols] into a padded matrix: row r -> (r / ra) * rb + r % ra + r0, columns alike.
 struct PackMap {
