@@ -597,11 +597,12 @@ Residual residual_after(vkl_model *m, int r) {
   return o;
 }
 
-// The norm with statistics that follows layer run `r` (-1: the embedding): of both sublayers' inputs, or the final one.
-int norm_after(vkl_model *m, int r, uint32_t T, bool pdl) {
+// The norm with statistics that follows layer run `r` (-1: the embedding), of both sublayers' inputs or the final one:
+// a kernel of its own for several tokens, for one part of the matrix product that reads it.
+RmsRows norm_of(vkl_model *m, int r, uint32_t T) {
   Decoder *d = m->dec.get();
-  if (d->spec.norm == NORM_TANH) return VKL_OK;
   RmsRows p = {};
+  if (d->spec.norm == NORM_TANH) return p;
   p.x = (const float *)d->x->data();
   p.T = T;
   p.ldw = d->ldw;
@@ -609,20 +610,25 @@ int norm_after(vkl_model *m, int r, uint32_t T, bool pdl) {
   p.eps = d->spec.norm_eps;
   p.h = d->h->data();
   p.w = (const float *)d->final_norm.w->data();
-  p.use_pdl = pdl;
   if ((size_t)(r + 1) < d->runs.size()) {
-    const uint32_t i = d->runs[r + 1].layer;
-    const DecLayer &l = d->L[i];
+    const DecLayer &l = d->L[d->runs[r + 1].layer];
     p.w = (const float *)l.norm.w->data();
     if (l.n2) {
       p.w2 = (const float *)l.norm2.w->data();
       p.h2 = d->h->data() + (size_t)T * d->ldw * elem(d);  // the second input of the in-projection follows the first
     }
   }
+  return p;
+}
+bool norm_in_matvec(const Decoder *d, uint32_t T) { return T == 1 && rows_matvec_takes_norm(d->ldw, d->spec.two_norms, d->f32); }
+int norm_after(vkl_model *m, int r, uint32_t T, bool pdl) {
+  Decoder *d = m->dec.get();
+  RmsRows p = norm_of(m, r, T);
+  if (!p.x || norm_in_matvec(d, T)) return VKL_OK;
+  p.use_pdl = pdl;
   VKL_LAUNCH(1, launch_rms_rows(p, d->f32, m->stream));
   return VKL_OK;
 }
-
 }  // namespace
 
 int decoder_create(vkl_device *dev, const DecoderSpec &spec, uint32_t maxlen, bool f32, vkl_model **out) {
@@ -848,7 +854,7 @@ int decoder_begin(vkl_model *m, size_t offset) {
 void decoder_end(vkl_model *m, size_t end) { m->dec->filled = end; }
 
 #define MARK(c) do { if (mk) mk->mark(c); } while (0)
-#define MARK_NORM() do { if (d->spec.norm != NORM_TANH) MARK(9); } while (0)
+#define MARK_NORM() do { if (d->spec.norm != NORM_TANH && !norm_in_matvec(d, T)) MARK(9); } while (0)
 
 namespace {
 // The delta rule's steps between the projections of layer run r.
@@ -985,6 +991,7 @@ int decoder_run(vkl_model *m, uint32_t T, bool pdl, Marker *mk) {
       p.K = d->ldw;
       p.x = d->h->data();
       if (l.n2) p.x2 = d->h->data() + (size_t)d->ldw * es;
+      if (norm_in_matvec(d, T)) p.norm = norm_of(m, (int)r - 1, T);
       p.n2 = l.n2;
       p.gap0 = l.gap0;
       p.out = in;
@@ -1017,6 +1024,7 @@ int decoder_run(vkl_model *m, uint32_t T, bool pdl, Marker *mk) {
       VKL_OKAY(run_delta(m, r, T, one && pdl));
       MARK(8);
     } else {
+      KvAttn at = {};
       if (a.qk_norm || a.rot.dims) {
         QkRows p = {};
         p.q = d->q->data();
@@ -1035,10 +1043,9 @@ int decoder_run(vkl_model *m, uint32_t T, bool pdl, Marker *mk) {
         p.dp = l.dp;
         p.maxlen = m->cfg.maxlen;
         p.pos = m->pos_dev();
-        p.use_pdl = one && pdl;
-        VKL_LAUNCH(1, launch_qk_rows(p, f32, s));
+        if (one) at.qk = p;  // part of the attention kernel
+        else VKL_LAUNCH(1, launch_qk_rows(p, f32, s));
       }
-      KvAttn at = {};
       at.q = d->q->data();
       at.q_ld = l.qcols;
       at.cache = kv.kcache->data();
@@ -1164,6 +1171,7 @@ int decoder_run(vkl_model *m, uint32_t T, bool pdl, Marker *mk) {
   p.N = d->vocab_p;
   p.K = d->ldw;
   p.x = d->h->data() + (size_t)(T - 1) * d->ldw * es;
+  if (norm_in_matvec(d, T)) p.norm = norm_of(m, (int)d->runs.size() - 1, T);
   p.out.seg[0] = RowSeg{0, d->vocab_p, ROW_STORE};
   p.out.nseg = 1;
   p.out.f32 = (float *)m->logits32->data();

@@ -34,7 +34,6 @@ constexpr uint32_t kBlock = 8, kPairsA = 28, kPairs = 64;  // token pairs s < t,
 
 __device__ __forceinline__ float load1(const bf16 *p) { return __bfloat162float(*p); }
 __device__ __forceinline__ float load1(const float *p) { return *p; }
-__device__ __forceinline__ float silu_f(float z) { return z * sigmoid_f(z); }
 
 // Projection c of token m, which may lie before the call's first token (position pos0) or the sequence's.
 template <class T> __device__ __forceinline__ float projection(const DeltaRows &p, int m, uint32_t pos0, uint32_t c) {
@@ -43,30 +42,42 @@ template <class T> __device__ __forceinline__ float projection(const DeltaRows &
   return at < 0 ? 0.f : load1(static_cast<const T *>(p.ring) + (size_t)((uint32_t)at % p.ntaps) * p.raw_ld + c);
 }
 
-// Channel c of tokens t0 .. t0 + 7 after convolution and SiLU; 0 from token n on. TAPS: 0 for any number.
-template <class T, int TAPS> __device__ __forceinline__ void convolve8(const DeltaRows &p, uint32_t t0, uint32_t n, uint32_t pos0, uint32_t c, float (&y)[kBlock]) {
-  const float *w = p.taps + (size_t)c * p.ntaps;
-  if constexpr (TAPS > 0) {
-    float x[kBlock + TAPS - 1], wr[TAPS];
+__device__ __forceinline__ float fast_sigmoid(float z) { return __fdividef(1.0f, 1.0f + expf(-z)); }
+
+// Projection c of tokens t0 - (TAPS - 1) .. t0 + 7; 0 from token t0 + n on.
+template <class T, int TAPS> __device__ __forceinline__ void load_window(const DeltaRows &p, uint32_t t0, uint32_t n, uint32_t pos0, uint32_t c, float (&x)[kBlock + TAPS - 1]) {
+  constexpr int BACK = TAPS - 1;
+  if (n == kBlock && t0 >= (uint32_t)BACK) {
+    const T *r = static_cast<const T *>(p.raw) + (size_t)(t0 - BACK) * p.raw_ld + c;
 #pragma unroll
-    for (int i = 0; i < (int)kBlock + TAPS - 1; ++i) x[i] = (int)n > i - (TAPS - 1) ? projection<T>(p, (int)t0 + i - (TAPS - 1), pos0, c) : 0.f;
-#pragma unroll
-    for (int j = 0; j < TAPS; ++j) wr[j] = w[j];
-#pragma unroll
-    for (int t = 0; t < (int)kBlock; ++t) {
-      float a = 0.f;
-#pragma unroll
-      for (int j = 0; j < TAPS; ++j) a = fmaf(x[t + j], wr[j], a);
-      y[t] = t < (int)n ? silu_f(a) : 0.f;
-    }
+    for (int i = 0; i < (int)kBlock + BACK; ++i) x[i] = load1(r + (size_t)i * p.raw_ld);
   } else {
 #pragma unroll
-    for (int t = 0; t < (int)kBlock; ++t) {
-      float a = 0.f;
-      if (t < (int)n)
-        for (uint32_t j = 0; j < p.ntaps; ++j) a = fmaf(projection<T>(p, (int)(t0 + t + j) - (int)(p.ntaps - 1), pos0, c), w[j], a);
-      y[t] = silu_f(a);
-    }
+    for (int i = 0; i < (int)kBlock + BACK; ++i) x[i] = (int)n > i - BACK ? projection<T>(p, (int)t0 + i - BACK, pos0, c) : 0.f;
+  }
+}
+// Convolution and SiLU of a window; 0 from token n on.
+template <int TAPS> __device__ __forceinline__ void convolve8(const DeltaRows &p, uint32_t n, uint32_t c, const float (&x)[kBlock + TAPS - 1], float (&y)[kBlock]) {
+  float w[TAPS];
+#pragma unroll
+  for (int j = 0; j < TAPS; ++j) w[j] = p.taps[(size_t)c * TAPS + j];
+#pragma unroll
+  for (int t = 0; t < (int)kBlock; ++t) {
+    float a = 0.f;
+#pragma unroll
+    for (int j = 0; j < TAPS; ++j) a = fmaf(x[t + j], w[j], a);
+    y[t] = t < (int)n ? a * fast_sigmoid(a) : 0.f;
+  }
+}
+// The same for any number of taps, one token after the other.
+template <class T> __device__ __forceinline__ void convolve8_any(const DeltaRows &p, uint32_t t0, uint32_t n, uint32_t pos0, uint32_t c, float (&y)[kBlock]) {
+  const float *w = p.taps + (size_t)c * p.ntaps;
+#pragma unroll
+  for (int t = 0; t < (int)kBlock; ++t) {
+    float a = 0.f;
+    if (t < (int)n)
+      for (uint32_t j = 0; j < p.ntaps; ++j) a = fmaf(projection<T>(p, (int)(t0 + t + j) - (int)(p.ntaps - 1), pos0, c), w[j], a);
+    y[t] = a * fast_sigmoid(a);
   }
 }
 
@@ -94,36 +105,50 @@ __device__ __forceinline__ uint32_t pair_a(uint32_t t, uint32_t s) { return s * 
 __device__ __forceinline__ uint32_t pair_b(uint32_t t, uint32_t s) { return kPairsA + s * 8 - s * (s - 1) / 2 + t - s; }  // s <= t
 
 // NT threads, one per key channel and one per value channel. first: token of block 0 of this launch.
-template <class T, int TAPS, int NT> __global__ void __launch_bounds__(NT) delta_blocks_kernel(const DeltaRows p, uint32_t first) {
+template <class T, int TAPS, int NT> __global__ void __launch_bounds__(NT, 512 / NT) delta_blocks_kernel(const DeltaRows p, uint32_t first) {
   constexpr int NW = NT / 32;
-  __shared__ float sums[NW][2 * kBlock], pairs[NW][kPairs], ab[kPairs], minv[kBlock][kBlock], beta_s[kBlock];
+  __shared__ float sums[NW][2 * kBlock], pairs[NW][kPairs], ab[kPairs], minv[kBlock][kBlock], beta_s[kBlock], scale_s[2 * kBlock];
   const uint32_t h = blockIdx.x, t0 = first + blockIdx.y * kBlock, n = min(kBlock, p.T - t0), tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
   const uint32_t kv = h / (p.heads / p.kv_heads), pos0 = *p.pos;
   float *rec = p.blocks + ((size_t)blockIdx.y * p.heads + h) * block_floats(p.dp);
   if (tid < kBlock) beta_s[tid] = tid < n ? p.beta[(size_t)(t0 + tid) * p.beta_ld + h] : 0.f;
-  if (tid < p.vp) {
-    float v[kBlock];
-    convolve8<T, TAPS>(p, t0, n, pos0, p.v_col + h * p.vp + tid, v);
+  const bool on = tid < p.dp, von = tid < p.vp;
+  const uint32_t cq = kv * p.dp + tid, ck = p.k_col + cq, cv = p.v_col + h * p.vp + tid, cg = h * p.dp + tid;
+  float q[kBlock], k[kBlock], g[kBlock], v[kBlock];
+#pragma unroll
+  for (uint32_t t = 0; t < kBlock; ++t) {
+    q[t] = k[t] = 0.f;
+    g[t] = on && t < n ? p.z[(size_t)(t0 + t) * p.z_ld + cg] : 0.f;
+  }
+  if constexpr (TAPS > 0) {
+    float xq[kBlock + TAPS - 1], xk[kBlock + TAPS - 1], xv[kBlock + TAPS - 1];
+    if (on) {
+      load_window<T, TAPS>(p, t0, n, pos0, cq, xq);
+      load_window<T, TAPS>(p, t0, n, pos0, ck, xk);
+    }
+    if (von) {
+      load_window<T, TAPS>(p, t0, n, pos0, cv, xv);
+      convolve8<TAPS>(p, n, cv, xv, v);
+    }
+    if (on) {
+      convolve8<TAPS>(p, n, cq, xq, q);
+      convolve8<TAPS>(p, n, ck, xk, k);
+    }
+  } else {
+    if (on) {
+      convolve8_any<T>(p, t0, n, pos0, cq, q);
+      convolve8_any<T>(p, t0, n, pos0, ck, k);
+    }
+    if (von) convolve8_any<T>(p, t0, n, pos0, cv, v);
+  }
+  if (von) {
 #pragma unroll
     for (uint32_t t = 0; t < kBlock; ++t)
       if (t < n) p.v[((size_t)(t0 + t) * p.heads + h) * p.vp + tid] = v[t];
   }
-  const bool on = tid < p.dp;
-  float q[kBlock], k[kBlock], g[kBlock];
+  const float rate = on ? p.rate[cg] : 0.f, bias = on ? p.bias[cg] : 0.f;
 #pragma unroll
-  for (uint32_t t = 0; t < kBlock; ++t) {
-    q[t] = k[t] = 0.f;
-    g[t] = 1.f;
-  }
-  if (on) {
-    convolve8<T, TAPS>(p, t0, n, pos0, kv * p.dp + tid, q);
-    convolve8<T, TAPS>(p, t0, n, pos0, p.k_col + kv * p.dp + tid, k);
-    const uint32_t c = h * p.dp + tid;
-    const float rate = p.rate[c], bias = p.bias[c];
-#pragma unroll
-    for (uint32_t t = 0; t < kBlock; ++t)
-      if (t < n) g[t] = expf(-rate * softplus_f(p.z[(size_t)(t0 + t) * p.z_ld + c] + bias));
-  }
+  for (uint32_t t = 0; t < kBlock; ++t) g[t] = t < n ? expf(-rate * softplus_f(g[t] + bias)) : 1.f;
   float ss[2 * kBlock];
 #pragma unroll
   for (uint32_t t = 0; t < kBlock; ++t) {
@@ -133,17 +158,17 @@ template <class T, int TAPS, int NT> __global__ void __launch_bounds__(NT) delta
   scatter_sum<2 * kBlock, 16>(ss, lane);  // lane: value lane / 2
   if (!(lane & 1)) sums[warp][lane >> 1] = ss[0];
   __syncthreads();
-  const float qscale = 1.0f / sqrtf((float)p.dim);
+  if (tid < 2 * kBlock) {
+    float a = 0.f;
+#pragma unroll
+    for (int w = 0; w < NW; ++w) a += sums[w][tid];
+    scale_s[tid] = 1.0f / sqrtf(a + kUnitEps) * (tid < kBlock ? 1.0f / sqrtf((float)p.dim) : 1.0f);
+  }
+  __syncthreads();
 #pragma unroll
   for (uint32_t t = 0; t < kBlock; ++t) {
-    float a = 0.f, b = 0.f;
-#pragma unroll
-    for (int w = 0; w < NW; ++w) {
-      a += sums[w][t];
-      b += sums[w][kBlock + t];
-    }
-    q[t] *= 1.0f / sqrtf(a + kUnitEps) * qscale;
-    k[t] *= 1.0f / sqrtf(b + kUnitEps);
+    q[t] *= scale_s[t];
+    k[t] *= scale_s[kBlock + t];
   }
   if (on) {
     float d = 1.f;
@@ -305,27 +330,28 @@ template <int E> __global__ void __launch_bounds__(kScanThreads) delta_scan_kern
     if (b + 1 < blocks) vnext = value(b + 1);
     if (!active) continue;
     const float *st = stage_mem + (b % kStages) * RF, *mn = st + 25 * DP + tok * kBlock;
-    auto dots = [&](const float *rows) {
-      f2 acc[kBlock][kScanCols];
+    f2 acc[2][kBlock][kScanCols];
+#pragma unroll
+    for (int r = 0; r < 2; ++r)
 #pragma unroll
       for (int t = 0; t < (int)kBlock; ++t)
 #pragma unroll
-        for (int c = 0; c < (int)kScanCols; ++c) acc[t][c] = 0;
+        for (int c = 0; c < (int)kScanCols; ++c) acc[r][t][c] = 0;
 #pragma unroll
-      for (int i = 0; i < NV; ++i)
+    for (int i = 0; i < NV; ++i)
 #pragma unroll
-        for (int t = 0; t < (int)kBlock; ++t) {
+      for (int t = 0; t < (int)kBlock; ++t)
+#pragma unroll
+        for (int r = 0; r < 2; ++r) {
           f2 x[NP];
-          load_pairs<NP>(rows + t * DP + (i * kScanLanes + l) * V, x);
+          load_pairs<NP>(st + (r * kBlock + t) * DP + (i * kScanLanes + l) * V, x);
 #pragma unroll
           for (int j = 0; j < NP; ++j)
 #pragma unroll
-            for (int c = 0; c < (int)kScanCols; ++c) acc[t][c] = fma2(S[c][i * NP + j], x[j], acc[t][c]);
+            for (int c = 0; c < (int)kScanCols; ++c) acc[r][t][c] = fma2(S[c][i * NP + j], x[j], acc[r][t][c]);
         }
-      return scatter_tokens(acc, l);
-    };
-    const float2 a = dots(st);
-    float2 o = dots(st + kBlock * DP);
+    const float2 a = scatter_tokens(acc[0], l);
+    float2 o = scatter_tokens(acc[1], l);
     const float2 w = make_float2(v.x - a.x, v.y - a.y);
     float2 u = make_float2(0.f, 0.f);
 #pragma unroll
@@ -374,9 +400,10 @@ constexpr int kFinishThreads = 256;
 template <class T> __global__ void __launch_bounds__(kFinishThreads) delta_finish_kernel(const DeltaRows p) {
   const uint32_t m = blockIdx.x, lane = threadIdx.x & 31, h = blockIdx.y * (kFinishThreads / 32) + (threadIdx.x >> 5);
   if (m + p.ntaps >= p.T) {  // one of the last ntaps tokens: later ones look back at it
-    const T *src = static_cast<const T *>(p.raw) + (size_t)m * p.raw_ld;
-    T *dst = static_cast<T *>(p.ring) + (size_t)((*p.pos + m) % p.ntaps) * p.raw_ld;
-    for (uint32_t c = blockIdx.y * kFinishThreads + threadIdx.x; c < p.raw_ld; c += gridDim.y * kFinishThreads) dst[c] = src[c];
+    const uint32_t pieces = p.raw_ld * sizeof(T) / 16;
+    const uint4 *src = static_cast<const uint4 *>(p.raw) + (size_t)m * pieces;
+    uint4 *dst = static_cast<uint4 *>(p.ring) + (size_t)((*p.pos + m) % p.ntaps) * pieces;
+    for (uint32_t c = blockIdx.y * kFinishThreads + threadIdx.x; c < pieces; c += gridDim.y * kFinishThreads) dst[c] = src[c];
   }
   if (h >= p.heads || lane * 8 >= p.vp) return;  // a lane holds eight columns
   const uint32_t lanes = 0xffffffffu >> (32 - p.vp / 8);
@@ -390,7 +417,7 @@ template <class T> __global__ void __launch_bounds__(kFinishThreads) delta_finis
   for (uint32_t i = 0; i < p.vp / 8; ++i) tot += __shfl_sync(lanes, ss, i);
   const float r = 1.0f / sqrtf(tot / (float)p.vdim + p.eps);
 #pragma unroll
-  for (int i = 0; i < 8; ++i) y[i] *= r * w[i] * sigmoid_f(z[i]);
+  for (int i = 0; i < 8; ++i) y[i] *= r * w[i] * fast_sigmoid(z[i]);
   store8(static_cast<T *>(p.out) + (size_t)m * p.out_ld + h * p.vp + lane * 8, y);
 }
 
@@ -424,19 +451,42 @@ template <class T, int E> __global__ void __launch_bounds__(kStepThreads) delta_
   const uint32_t pos = *p.pos;
 #pragma unroll
   for (int i = 0; i < E; ++i) S[i] = active && pos ? *reinterpret_cast<const float4 *>(state + i * 32) : make_float4(0.f, 0.f, 0.f, 0.f);
-  if (p.use_pdl) asm volatile("griddepcontrol.wait;" ::: "memory");
-  // convolution: query and key channels, this CTA's value channels
-  for (uint32_t i = tid; i < 2 * DP + cols; i += kStepThreads) {
-    const uint32_t c = i < DP ? kv * DP + i : i < 2 * DP ? p.k_col + kv * DP + i - DP : p.v_col + h * p.vp + c0 + i - 2 * DP;
-    const T *cur = static_cast<const T *>(p.raw) + c;
-    float a = 0.f;
-    for (uint32_t j = 0; j < p.ntaps; ++j) a = fmaf(projection<T>(p, (int)j - (int)(p.ntaps - 1), pos, c), p.taps[(size_t)c * p.ntaps + j], a);
-    a = silu_f(a);
+  // convolution: query and key channels, this CTA's value channels; the past tokens' part
+  constexpr int ROUNDS = (2 * DP + kStepCols + kStepThreads - 1) / kStepThreads;
+  uint32_t chan[ROUNDS];
+  float past[ROUNDS], last[ROUNDS];
+#pragma unroll
+  for (int r = 0; r < ROUNDS; ++r) {
+    const uint32_t i = r * kStepThreads + tid;
+    past[r] = last[r] = 0.f;
+    chan[r] = i < DP ? kv * DP + i : i < 2 * DP ? p.k_col + kv * DP + i - DP : p.v_col + h * p.vp + c0 + i - 2 * DP;
+    if (i >= 2 * DP + cols) continue;
+    const float *w = p.taps + (size_t)chan[r] * p.ntaps;
+    last[r] = w[p.ntaps - 1];
+    const uint32_t back = min(p.ntaps - 1, pos);
+    uint32_t slot = (pos - back) % p.ntaps;
+#pragma unroll 4
+    for (uint32_t j = p.ntaps - 1 - back; j < p.ntaps - 1; ++j) {
+      past[r] = fmaf(load1(static_cast<const T *>(p.ring) + (size_t)slot * p.raw_ld + chan[r]), w[j], past[r]);
+      slot = slot + 1 == p.ntaps ? 0u : slot + 1;
+    }
+  }
+  if (p.use_pdl) {
+    asm volatile("griddepcontrol.launch_dependents;");
+    asm volatile("griddepcontrol.wait;" ::: "memory");
+  }
+#pragma unroll
+  for (int r = 0; r < ROUNDS; ++r) {
+    const uint32_t i = r * kStepThreads + tid;
+    if (i >= 2 * DP + cols) continue;
+    const T x = static_cast<const T *>(p.raw)[chan[r]];
+    float a = fmaf(load1(&x), last[r], past[r]);
+    a *= fast_sigmoid(a);
     if (i < DP) q_s[i] = a;
     else if (i < 2 * DP) k_s[i - DP] = a;
     else v_s[i - 2 * DP] = a;
     // the slot of this position is read by no one in this step; heads that share a key head write the same number
-    static_cast<T *>(p.ring)[(size_t)(pos % p.ntaps) * p.raw_ld + c] = *cur;
+    static_cast<T *>(p.ring)[(size_t)(pos % p.ntaps) * p.raw_ld + chan[r]] = x;
   }
   auto finish_row = [&](uint32_t row, float z) {
 #pragma unroll
@@ -473,7 +523,6 @@ template <class T, int E> __global__ void __launch_bounds__(kStepThreads) delta_
     }
   }
   __syncthreads();
-  if (p.use_pdl) asm volatile("griddepcontrol.launch_dependents;");
   float qq = 0.f, kk = 0.f;  // every warp for itself
 #pragma unroll
   for (int i = 0; i < E; ++i) {

@@ -59,6 +59,7 @@ template <class T, int LPR, int NQ, bool SEP> __global__ void __launch_bounds__(
   __shared__ float sm_o[kRowThreads / 32][NQ][DMAX], sm_m[kRowThreads / 32][NQ], sm_l[kRowThreads / 32][NQ];
   __shared__ float sm_pm[kMaxSplits][NQ], sm_pl[kMaxSplits][NQ];
   __shared__ uint32_t last_s;
+  __shared__ float2 turn_s[kMaxPairs];
   const uint32_t per = p.heads / p.kv_heads, groups = (per + NQ - 1) / NQ;
   const uint32_t g = blockIdx.x / groups, hg = blockIdx.x % groups, h0 = g * per + hg * NQ, nh = min((uint32_t)NQ, per - hg * NQ);
   const uint32_t m = blockIdx.y, split = blockIdx.z, tid = threadIdx.x, sub = tid / LPR, l = tid % LPR, e0 = l * 8, warp = tid >> 5;
@@ -71,6 +72,30 @@ template <class T, int LPR, int NQ, bool SEP> __global__ void __launch_bounds__(
   chunk = (chunk + 31) & ~31u;
   const uint32_t c0 = min(lo + split * chunk, vis), c1 = min(c0 + chunk, vis);
   const float qs = query_scale(p, pos);
+  float rq = 1.f;
+  if (p.qk.q) {  // one raw token: every CTA norms and turns its queries, the ones that see the token itself its key
+    const bool newest = c0 < vis && c1 == vis && p.qk.kcache;
+    const T *qr = static_cast<const T *>(p.qk.q), *kr = qr + p.qk.k_col;
+    if (tid < p.qk.pairs) turn_s[tid] = turn_of(pos, p.qk.freq[tid]);
+    float sq = 0.f, sk = 0.f, v[8];
+    for (uint32_t n = tid * 8; n < p.heads * p.dp; n += kRowThreads * 8) {
+      load8(qr + n, v);
+      sq = square_sum8(v, sq);
+    }
+    for (uint32_t n = tid * 8; newest && n < p.kv_heads * p.dp; n += kRowThreads * 8) {
+      load8(kr + n, v);
+      sk = square_sum8(v, sk);
+    }
+    const float2 ss = block_sum2<kRowThreads / 32>(sq, sk);  // also: the angles are in place
+    rq = 1.0f / sqrtf(ss.x / (float)(p.heads * p.qk.dim) + p.qk.eps);
+    if (newest && tid < p.dp / 8) {
+      const uint32_t c = g * p.dp + tid * 8;
+      load8(kr + c, v);
+      norm_and_turn(v, p.qk.kw ? p.qk.kw + c : nullptr, 1.0f / sqrtf(ss.y / (float)(p.kv_heads * p.qk.dim) + p.qk.eps), tid * 8, turn_s, p.qk.pairs);
+      store8(cache_slot<T>(p.qk.kcache, p.dp, p.maxlen, pos, c), v);
+    }
+    __syncthreads();
+  }
 
   float q[NQ][8], acc[NQ][8], mx[NQ], sum[NQ];
 #pragma unroll
@@ -78,6 +103,7 @@ template <class T, int LPR, int NQ, bool SEP> __global__ void __launch_bounds__(
     Raw8<T> r;
     if (ev && i < nh) r.load(static_cast<const T *>(p.q) + (size_t)m * p.q_ld + (size_t)(h0 + i) * p.dp + e0);
     r.get(q[i]);
+    if (p.qk.q && ev && i < nh) norm_and_turn(q[i], p.qk.qw ? p.qk.qw + (size_t)(h0 + i) * p.dp + e0 : nullptr, rq, e0, turn_s, p.qk.pairs);
 #pragma unroll
     for (int e = 0; e < 8; ++e) {
       q[i][e] *= qs;
@@ -457,8 +483,8 @@ uint32_t kv_attn_counters(uint32_t T, uint32_t heads) { return T * heads; }
 cudaError_t launch_kv_attention(const KvAttn &p, bool f32, cudaStream_t s) {
   if (!p.T || !p.kv_heads || p.heads % p.kv_heads || p.dp % 16 || p.dp > 256 || p.vp % 16 || p.vp > 256 || (!p.vcache && p.vp != p.dp) || !p.splits || p.splits > kMaxSplits)
     return cudaErrorInvalidValue;
-  if (!f32 && p.T >= kTileRows) return p.vcache ? launch_tile_d<true>(p, s) : launch_tile_d<false>(p, s);
-  if (p.T > 65535) return cudaErrorInvalidValue;
+  if (!f32 && p.T >= kTileRows && !p.qk.q) return p.vcache ? launch_tile_d<true>(p, s) : launch_tile_d<false>(p, s);
+  if (p.T > 65535 || (p.qk.q && (p.T != 1 || p.qk.pairs > kMaxPairs || p.qk.k_col % 8))) return cudaErrorInvalidValue;
   if (p.vcache) return f32 ? launch_row_d<float, true>(p, s) : launch_row_d<bf16, true>(p, s);
   return f32 ? launch_row_d<float, false>(p, s) : launch_row_d<bf16, false>(p, s);
 }

@@ -9,53 +9,12 @@ namespace {
 
 constexpr int kThreads = 256, kWarps = kThreads / 32;
 
-// Sums of two numbers over the CTA, the same order every time.
-__device__ __forceinline__ float2 block_sum2(float a, float b) {
-  __shared__ float2 part[kWarps];
-  a = warp_sum(a);
-  b = warp_sum(b);
-  if ((threadIdx.x & 31) == 0) part[threadIdx.x >> 5] = make_float2(a, b);
-  __syncthreads();
-  float2 r = part[0];
-#pragma unroll
-  for (int w = 1; w < kWarps; ++w) {
-    r.x += part[w].x;
-    r.y += part[w].y;
-  }
-  return r;
-}
-
 template <class T> __global__ void __launch_bounds__(kThreads) rms_rows_kernel(const RmsRows p) {
   if (p.use_pdl) asm volatile("griddepcontrol.wait;" ::: "memory");
-  const float *x = p.x + (size_t)blockIdx.x * p.ldw;
   const size_t o = (size_t)blockIdx.x * p.ldw;
-  float ss = 0.f;
-  for (uint32_t n = threadIdx.x * 8; n < p.ldw; n += kThreads * 8) {
-    float v[8];
-    load8(x + n, v);
-#pragma unroll
-    for (int i = 0; i < 8; ++i) ss = fmaf(v[i], v[i], ss);
-  }
-  ss = block_sum2(ss, 0.f).x;
-  const float r = 1.0f / sqrtf(ss / (float)p.width + p.eps);
-  for (uint32_t n = threadIdx.x * 8; n < p.ldw; n += kThreads * 8) {
-    float v[8], w[8], y[8];
-    load8(x + n, v);
-    load8(p.w + n, w);
-#pragma unroll
-    for (int i = 0; i < 8; ++i) y[i] = v[i] * r * w[i];
-    store8(static_cast<T *>(p.h) + o + n, y);
-    if (p.w2) {
-      load8(p.w2 + n, w);
-#pragma unroll
-      for (int i = 0; i < 8; ++i) y[i] = v[i] * r * w[i];
-      store8(static_cast<T *>(p.h2) + o + n, y);
-    }
-  }
+  rms_row<T, kWarps>(p, p.x + o, static_cast<T *>(p.h) + o, static_cast<T *>(p.h2) + o);
   if (p.use_pdl) asm volatile("griddepcontrol.launch_dependents;");
 }
-
-constexpr uint32_t kMaxPairs = 128;  // head width at most 256
 
 template <class T> __global__ void __launch_bounds__(kThreads) qk_rows_kernel(const QkRows p) {
   __shared__ float2 turn[kMaxPairs];
@@ -63,45 +22,24 @@ template <class T> __global__ void __launch_bounds__(kThreads) qk_rows_kernel(co
   const uint32_t m = blockIdx.x, pos = *p.pos + m, tid = threadIdx.x;
   const uint32_t nq = p.heads * p.dp, nk = p.kcache ? p.kv_heads * p.dp : 0u;
   T *q = static_cast<T *>(p.q) + (size_t)m * p.q_ld, *k = q + p.k_col;
-  if (tid < p.pairs) {
-    float s, c;
-    sincosf((float)pos * p.freq[tid], &s, &c);
-    turn[tid] = make_float2(c, s);
-  }
-  float sq = 0.f, sk = 0.f;
+  if (tid < p.pairs) turn[tid] = turn_of(pos, p.freq[tid]);
+  float sq = 0.f, sk = 0.f, v[8];
   for (uint32_t n = tid * 8; n < nq; n += kThreads * 8) {  // padded columns are zero
-    float v[8];
     load8(q + n, v);
-#pragma unroll
-    for (int i = 0; i < 8; ++i) sq = fmaf(v[i], v[i], sq);
+    sq = square_sum8(v, sq);
   }
   for (uint32_t n = tid * 8; n < nk; n += kThreads * 8) {
-    float v[8];
     load8(k + n, v);
-#pragma unroll
-    for (int i = 0; i < 8; ++i) sk = fmaf(v[i], v[i], sk);
+    sk = square_sum8(v, sk);
   }
-  const float2 ss = block_sum2(sq, sk);  // also: every thread's angles are in place
-  const float rq = p.qw ? 1.0f / sqrtf(ss.x / (float)(p.heads * p.dim) + p.eps) : 1.f;
-  const float rk = p.kw ? 1.0f / sqrtf(ss.y / (float)(p.kv_heads * p.dim) + p.eps) : 1.f;
+  const float2 ss = block_sum2<kWarps>(sq, sk);  // also: every thread's angles are in place
+  const float rq = 1.0f / sqrtf(ss.x / (float)(p.heads * p.dim) + p.eps), rk = 1.0f / sqrtf(ss.y / (float)(p.kv_heads * p.dim) + p.eps);
   for (uint32_t n = tid * 8; n < nq + nk; n += kThreads * 8) {
     const bool key = n >= nq;
-    const uint32_t c = key ? n - nq : n, d = c % p.dp;
+    const uint32_t c = key ? n - nq : n;
     const float *w = key ? p.kw : p.qw;
-    float v[8];
     load8(key ? k + c : q + c, v);
-    const float r = key ? rk : rq;
-#pragma unroll
-    for (int i = 0; i < 8; ++i) v[i] *= w ? r * w[c + i] : 1.f;
-#pragma unroll
-    for (int i = 0; i < 8; i += 2) {
-      if ((d + i) / 2 < p.pairs) {
-        const float2 t = turn[(d + i) / 2];
-        const float a = v[i], b = v[i + 1];
-        v[i] = a * t.x - b * t.y;
-        v[i + 1] = b * t.x + a * t.y;
-      }
-    }
+    norm_and_turn(v, w ? w + c : nullptr, key ? rk : rq, c % p.dp, turn, p.pairs);
     store8(key ? cache_slot<T>(p.kcache, p.dp, p.maxlen, pos, c) : q + c, v);
   }
   if (p.use_pdl) asm volatile("griddepcontrol.launch_dependents;");

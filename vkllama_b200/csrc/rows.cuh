@@ -42,6 +42,74 @@ __device__ __forceinline__ float glu_act(uint32_t act, float limit, float g, flo
 }
 __device__ __forceinline__ float tanh_norm(float x, float alpha, float w, float b) { return tanhf(alpha * x) * w + b; }
 
+// Sums of two numbers over a CTA of WARPS warps, the same order every time.
+template <int WARPS> __device__ __forceinline__ float2 block_sum2(float a, float b) {
+  __shared__ float2 part[WARPS];
+  a = warp_sum(a);
+  b = warp_sum(b);
+  if ((threadIdx.x & 31) == 0) part[threadIdx.x >> 5] = make_float2(a, b);
+  __syncthreads();
+  float2 r = part[0];
+#pragma unroll
+  for (int w = 1; w < WARPS; ++w) {
+    r.x += part[w].x;
+    r.y += part[w].y;
+  }
+  return r;
+}
+__device__ __forceinline__ float square_sum8(const float (&v)[8], float s) {
+#pragma unroll
+  for (int i = 0; i < 8; ++i) s = fmaf(v[i], v[i], s);
+  return s;
+}
+// RMS norm of one row, for one or two weights (RmsRows), by a CTA of WARPS warps.
+template <class T, int WARPS> __device__ __forceinline__ void rms_row(const RmsRows &p, const float *x, T *h, T *h2) {
+  float ss = 0.f;
+  for (uint32_t n = threadIdx.x * 8; n < p.ldw; n += WARPS * 256) {
+    float v[8];
+    load8(x + n, v);
+    ss = square_sum8(v, ss);
+  }
+  const float r = 1.0f / sqrtf(block_sum2<WARPS>(ss, 0.f).x / (float)p.width + p.eps);
+  for (uint32_t n = threadIdx.x * 8; n < p.ldw; n += WARPS * 256) {
+    float v[8], w[8], y[8];
+    load8(x + n, v);
+    load8(p.w + n, w);
+#pragma unroll
+    for (int i = 0; i < 8; ++i) y[i] = v[i] * r * w[i];
+    store8(h + n, y);
+    if (p.w2) {
+      load8(p.w2 + n, w);
+#pragma unroll
+      for (int i = 0; i < 8; ++i) y[i] = v[i] * r * w[i];
+      store8(h2 + n, y);
+    }
+  }
+}
+// Eight consecutive dimensions of a head, from dimension d on: norm (r times the weights, if any) and rotation; turn:
+// cosine and sine per pair.
+__device__ __forceinline__ void norm_and_turn(float (&v)[8], const float *w, float r, uint32_t d, const float2 *turn, uint32_t pairs) {
+  if (w) {
+#pragma unroll
+    for (int i = 0; i < 8; ++i) v[i] *= r * w[i];
+  }
+#pragma unroll
+  for (int i = 0; i < 8; i += 2) {
+    if ((d + i) / 2 < pairs) {
+      const float2 t = turn[(d + i) / 2];
+      const float a = v[i], b = v[i + 1];
+      v[i] = a * t.x - b * t.y;
+      v[i + 1] = b * t.x + a * t.y;
+    }
+  }
+}
+constexpr uint32_t kMaxPairs = 128;  // head width at most 256
+__device__ __forceinline__ float2 turn_of(uint32_t pos, float freq) {
+  float s, c;
+  sincosf((float)pos * freq, &s, &c);
+  return make_float2(c, s);
+}
+
 __device__ __forceinline__ float softplus_f(float z) { return fmaxf(z, 0.f) + log1pf(expf(-fabsf(z))); }
 __device__ __forceinline__ float soft_cap(float v, float cap) { return cap > 0.f ? cap * tanhf(v / cap) : v; }
 

@@ -76,6 +76,35 @@ struct RowsOut {
   Residual res;
 };
 
+// ---- norms with statistics, rotation (norm_rows.cu) ----
+// RMS norm of the residual stream with up to two weights (they share the statistic): h = x / rms(x) * w, the same
+// for h2 and w2. The weights are what multiplies (a weight stored around zero has its 1 added when it is loaded).
+struct RmsRows {
+  const float *x;           // [T, ldw]
+  uint32_t T, ldw, width;
+  const float *w, *w2;      // w2 may be null
+  void *h, *h2;             // [T, ldw] compute type
+  float eps;
+  int use_pdl;
+};
+cudaError_t launch_rms_rows(const RmsRows &p, bool f32, cudaStream_t s);
+
+// RMS norm over all of a token's query rows and over all of its key rows, rotation of the first 2 * pairs dimensions
+// of each head (neighbours 2i, 2i + 1 turn by position * freq[i]); queries stay where they are, keys go to the cache.
+struct QkRows {
+  void *q;                  // [T, q_ld] compute type: queries from column 0, raw keys from column k_col
+  uint32_t q_ld, k_col;
+  const float *qw, *kw;     // norm weights, padded like the rows; null: no norm
+  float eps;
+  const float *freq;
+  uint32_t pairs;
+  void *kcache;             // null: the layer has no keys of its own
+  uint32_t T, heads, kv_heads, dim, dp, maxlen;
+  const uint32_t *pos;
+  int use_pdl;
+};
+cudaError_t launch_qk_rows(const QkRows &p, bool f32, cudaStream_t s);
+
 // ---- one token: y = W x, weights bf16 [N, K], x in the compute type, fp32 accumulation (rows_matvec.cu) ----
 struct MvRows {
   const bf16 *w;
@@ -83,6 +112,7 @@ struct MvRows {
   const void *x;            // [K]
   const void *x2;           // rows from n2 on read this vector instead; null: none
   uint32_t n2, gap0;        // rows [gap0, n2) are padding and not computed (gap0 = n2: none)
+  RmsRows norm;             // norm.x set: x (and x2, if norm.w2) are this norm's outputs, computed in the kernel
   // Routed experts. In-projection form: the chosen experts' gate/up rows (ne each, GLU order) read x too and
   // write xe [top, ke]. Out-projection form: N rows per expert over ke columns of xe, summed and weighted.
   const bf16 *we;
@@ -96,6 +126,7 @@ struct MvRows {
   int use_pdl;
   RowsOut out;
 };
+bool rows_matvec_takes_norm(uint32_t K, bool two, bool f32);  // whether the norm's outputs fit in a CTA
 cudaError_t launch_rows_matvec(const MvRows &p, bool f32, int sms, cudaStream_t s);
 
 // ---- many tokens: Y[M,N] = A[M,K] . W[N,K]^T ----
@@ -133,6 +164,7 @@ struct KvAttn {
   uint32_t T, heads, kv_heads, dp, vp, maxlen, splits;
   float *scratch;           // kv_attn_scratch_bytes
   uint32_t *counters;       // one per (row, head group), zero before and after
+  QkRows qk;                // one token: qk.q set: q is raw, norm, rotation and the key's row of the cache are done here
   int use_pdl;
 };
 size_t kv_attn_scratch_bytes(uint32_t T, uint32_t heads, uint32_t vp, uint32_t splits);
@@ -158,35 +190,6 @@ cudaError_t launch_gather_rows(const void *src, const int32_t *rows, uint32_t n,
 cudaError_t launch_combine(const float *y, uint32_t y_ld, const int32_t *slot, uint32_t top, uint32_t T, const Residual &r, bool f32, cudaStream_t s);
 // x = scale * embed[token], then the residual step without its acc.
 cudaError_t launch_embed_rows(const bf16 *emb, const uint32_t *toks, uint32_t T, float scale, const Residual &r, bool f32, cudaStream_t s);
-
-// ---- norms with statistics, rotation (norm_rows.cu) ----
-// RMS norm of the residual stream with up to two weights (they share the statistic): h = x / rms(x) * w, the same
-// for h2 and w2. The weights are what multiplies (a weight stored around zero has its 1 added when it is loaded).
-struct RmsRows {
-  const float *x;           // [T, ldw]
-  uint32_t T, ldw, width;
-  const float *w, *w2;      // w2 may be null
-  void *h, *h2;             // [T, ldw] compute type
-  float eps;
-  int use_pdl;
-};
-cudaError_t launch_rms_rows(const RmsRows &p, bool f32, cudaStream_t s);
-
-// RMS norm over all of a token's query rows and over all of its key rows, rotation of the first 2 * pairs dimensions
-// of each head (neighbours 2i, 2i + 1 turn by position * freq[i]); queries stay where they are, keys go to the cache.
-struct QkRows {
-  void *q;                  // [T, q_ld] compute type: queries from column 0, raw keys from column k_col
-  uint32_t q_ld, k_col;
-  const float *qw, *kw;     // norm weights, padded like the rows; null: no norm
-  float eps;
-  const float *freq;
-  uint32_t pairs;
-  void *kcache;             // null: the layer has no keys of its own
-  uint32_t T, heads, kv_heads, dim, dp, maxlen;
-  const uint32_t *pos;
-  int use_pdl;
-};
-cudaError_t launch_qk_rows(const QkRows &p, bool f32, cudaStream_t s);
 
 // ---- gated delta rule with a decay per key channel (delta_rule.cu) ----
 // Per head a state S [dim, vdim]: S <- g S, u = beta (v - S^T k), S <- S + k u^T, o = S^T q, then the RMS norm of o and

@@ -6,7 +6,7 @@
 // fp32 FMAs. What becomes of a row is in its segment (rows.h), so one launch runs everything that reads the
 // same input: keys, queries, head gates and the feed-forward's gate/up rows of a parallel block, and the
 // gate/up rows of the experts that the token's id names. Rows may be split between two inputs (two norms of one
-// stream). The out-projection form sums, per output row, the
+// stream), and a norm with statistics that leads to them is computed by every CTA for itself. The out-projection form sums, per output row, the
 // attention's columns, the dense feed-forward's columns (one matrix, side by side) or the chosen experts'
 // rows, and leaves the residual stream and the next norm's output behind.
 #include <algorithm>
@@ -85,6 +85,15 @@ template <class T, int KS, bool OUT> __global__ void __launch_bounds__(kThreads)
     }
     asm volatile("griddepcontrol.wait;" ::: "memory");
   }
+  const T *x1 = static_cast<const T *>(p.x), *x2 = static_cast<const T *>(p.x2);
+  if (p.norm.x) {  // every CTA for itself
+    extern __shared__ __align__(16) unsigned char xs_raw[];
+    T *xs = reinterpret_cast<T *>(xs_raw);
+    rms_row<T, kWarps>(p.norm, p.norm.x, xs, xs + p.K);
+    __syncthreads();
+    x1 = xs;
+    x2 = xs + p.K;
+  }
   const uint32_t tok = p.top ? *p.tok : 0u;
   for (uint32_t it = 0; it < rounds; ++it) {
     const uint32_t u = (it * gridDim.x + blockIdx.x) * UPC + wg;
@@ -94,10 +103,10 @@ template <class T, int KS, bool OUT> __global__ void __launch_bounds__(kThreads)
     bool main_rows = true, glu = false;
     RowSeg sg = p.out.seg[0];
     if (active) {
-      const T *x = static_cast<const T *>(p.x);
+      const T *x = x1;
       if (u < u_main) {
         n = first_row(u);
-        if (p.x2 && n >= p.n2) x = static_cast<const T *>(p.x2);
+        if (p.n2 && n >= p.n2) x = x2;
         sg = find_seg(p.out, n);
         glu = !OUT && sg.kind == ROW_GLU;
         if (glu) n = sg.n0 + glu_row((n - sg.n0) / 4);
@@ -154,16 +163,20 @@ template <class T, int KS, bool OUT> __global__ void __launch_bounds__(kThreads)
 
 template <class T, int KS, bool OUT> cudaError_t launch_t(const MvRows &p, uint32_t units, int sms, cudaStream_t s) {
   auto kern = rows_matvec_kernel<T, KS, OUT>;
-  static const int per_sm = [] {
+  const size_t smem = p.norm.x ? (p.norm.w2 ? 2 : 1) * (size_t)p.K * sizeof(T) : 0;
+  auto resident = [](size_t bytes) {
     int n = 0;
-    return cudaOccupancyMaxActiveBlocksPerMultiprocessor(&n, rows_matvec_kernel<T, KS, OUT>, kThreads, 0) == cudaSuccess && n > 0 ? n : 1;
-  }();
+    return cudaOccupancyMaxActiveBlocksPerMultiprocessor(&n, rows_matvec_kernel<T, KS, OUT>, kThreads, bytes) == cudaSuccess && n > 0 ? n : 1;
+  };
+  static const int without_norm = resident(0);
+  const int per_sm = smem ? resident(smem) : without_norm;
   // one wave, every CTA with the same number of rounds (or one less)
   const uint32_t ctas = (units + kWarps / KS - 1) / (kWarps / KS), slots = (uint32_t)(sms * per_sm);
   const uint32_t rounds = (ctas + slots - 1) / slots;
   cudaLaunchConfig_t cfg = {};
   cfg.gridDim = dim3((ctas + rounds - 1) / rounds);
   cfg.blockDim = dim3(kThreads);
+  cfg.dynamicSmemBytes = smem;
   cfg.stream = s;
   cudaLaunchAttribute attr[1];
   attr[0].id = cudaLaunchAttributeProgrammaticStreamSerialization;
@@ -188,7 +201,10 @@ template <class T, bool OUT> cudaError_t launch_ks(const MvRows &p, int sms, cud
 
 }  // namespace
 
+bool rows_matvec_takes_norm(uint32_t K, bool two, bool f32) { return (two ? 2 : 1) * (size_t)K * (f32 ? 4 : 2) <= 46 * 1024; }
+
 cudaError_t launch_rows_matvec(const MvRows &p, bool f32, int sms, cudaStream_t s) {
+  if (p.norm.x && (p.norm.ldw != p.K || (p.n2 && !p.norm.w2) || !rows_matvec_takes_norm(p.K, p.norm.w2, f32))) return cudaErrorInvalidValue;
   if (!p.N || p.N % 32 || p.K % 64 || p.gap0 % 32 || p.n2 % 32 || p.gap0 > p.n2 || p.n2 > p.N || (p.top && (p.ke % 64 || p.ne % 32))) return cudaErrorInvalidValue;
   if (f32) return p.out_proj ? launch_ks<float, true>(p, sms, s) : launch_ks<float, false>(p, sms, s);
   return p.out_proj ? launch_ks<bf16, true>(p, sms, s) : launch_ks<bf16, false>(p, sms, s);
