@@ -918,6 +918,8 @@ int run_delta(vkl_model *m, size_t r, uint32_t T, bool pdl) {
   p.z_ld = l.nl;
   p.v = (float *)d->dv->data();
   p.blocks = (float *)d->dblocks->data();
+  p.error = g.error;
+  p.sms = m->dev->prop.multiProcessorCount;
   VKL_LAUNCH(delta_launches(T), launch_delta_rows(p, f32, s));
   return VKL_OK;
 }

@@ -10,8 +10,8 @@
 // Decays only ever multiply (no quotient of products), so nothing overflows and a decay of zero is exact.
 //   blocks      a CTA per head and block: convolution, SiLU, unit norms, decays, and from them the rows P k, P q,
 //               (later decays) k, the product of the decays, M and N. Depends on no state: all blocks at once.
-//   scan        the columns of a state do not depend on each other: 16 lanes hold four columns in registers and walk
-//               over the blocks, whose rows travel through a ring of shared-memory stages. A column's arithmetic within
+//   scan        the columns of a state do not depend on each other: 16 or 32 lanes hold four columns in registers and
+//               walk over the blocks, whose rows travel through a ring of shared-memory stages. A column's arithmetic within
 //               a block is all independent dot products.
 //   finish      a warp per token and head: RMS norm of the head's outputs, gate; and the call's last projections go to
 //               the ring of past projections.
@@ -105,7 +105,7 @@ __device__ __forceinline__ uint32_t pair_a(uint32_t t, uint32_t s) { return s * 
 __device__ __forceinline__ uint32_t pair_b(uint32_t t, uint32_t s) { return kPairsA + s * 8 - s * (s - 1) / 2 + t - s; }  // s <= t
 
 // NT threads, one per key channel and one per value channel. first: token of block 0 of this launch.
-template <class T, int TAPS, int NT> __global__ void __launch_bounds__(NT, 512 / NT) delta_blocks_kernel(const DeltaRows p, uint32_t first) {
+template <class T, int TAPS, int NT> __global__ void __launch_bounds__(NT, 768 / NT) delta_blocks_kernel(const DeltaRows p, uint32_t first) {
   constexpr int NW = NT / 32;
   __shared__ float sums[NW][2 * kBlock], pairs[NW][kPairs], ab[kPairs], minv[kBlock][kBlock], beta_s[kBlock], scale_s[2 * kBlock];
   const uint32_t h = blockIdx.x, t0 = first + blockIdx.y * kBlock, n = min(kBlock, p.T - t0), tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
@@ -232,8 +232,15 @@ template <class T, int TAPS, int NT> __global__ void __launch_bounds__(NT, 512 /
   }
 }
 
-__device__ __forceinline__ void copy16(void *dst, const void *src) {
-  asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"((uint32_t)__cvta_generic_to_shared(dst)), "l"(src) : "memory");
+__device__ __forceinline__ uint32_t smem_at(const void *p) { return (uint32_t)__cvta_generic_to_shared(p); }
+constexpr uint32_t kWaitLimit = 1u << 22;
+__device__ __forceinline__ bool wait_bounded(uint64_t *bar, uint32_t parity) {
+  for (uint32_t i = 0; i < kWaitLimit; ++i) {
+    uint32_t ok;
+    asm volatile("{\n .reg .pred p;\n mbarrier.try_wait.parity.shared::cta.b64 p, [%1], %2;\n selp.u32 %0, 1, 0, p;\n}" : "=r"(ok) : "r"(smem_at(bar)), "r"(parity) : "memory");
+    if (ok) return true;
+  }
+  return false;
 }
 // Two fp32 numbers in one register pair.
 using f2 = unsigned long long;
@@ -272,29 +279,51 @@ template <int N> __device__ __forceinline__ void store_pairs(float *p, const f2 
   else *reinterpret_cast<f2 *>(p) = o[0];
 }
 
-constexpr uint32_t kScanLanes = 16, kScanCols = 4, kScanThreads = 128, kCtaCols = kScanThreads / kScanLanes * kScanCols, kStages = 3;
+constexpr uint32_t kScanCols = 4, kScanThreads = 128, kStages = 3;  // and a warp that requests the records
+__host__ __device__ constexpr uint32_t cta_cols(uint32_t lp) { return kScanThreads / lp * kScanCols; }
 
-// Sums over 16 lanes of [token][column]; lane l ends with token l / 2, columns 2 (l % 2) and the next.
-__device__ __forceinline__ float2 scatter_tokens(const f2 (&acc)[kBlock][kScanCols], uint32_t l) {
-  float a[kBlock * kScanCols];
-#pragma unroll
-  for (int t = 0; t < (int)kBlock; ++t)
-#pragma unroll
-    for (int c = 0; c < (int)kScanCols; ++c) a[t * kScanCols + c] = add_halves(acc[t][c]);
-  scatter_sum<kBlock * kScanCols, 8>(a, l);
-  return make_float2(a[0], a[1]);
-}
-
-// E: 32-element steps of the key width. Lane l holds elements (16 i + l) V .. + V - 1 of each of its columns.
-template <int E> __global__ void __launch_bounds__(kScanThreads) delta_scan_kernel(const DeltaRows p, uint32_t first, uint32_t count) {
+// E: 32-element steps of the key width. LP lanes share four columns; lane l holds elements (LP i + l) V .. + V - 1 of
+// each, and ends up with the sums of token tok = l / (LP / 8) for CP of the columns. So that the sums can be exchanged
+// without choosing registers by lane, slot t of a lane's sums is token t ^ tok and slot c column c ^ cmask.
+template <int E, int LP> __global__ void __launch_bounds__(kScanThreads + 32) delta_scan_kernel(const DeltaRows p, uint32_t first, uint32_t count) {
   constexpr uint32_t DP = E * 32, RF = block_floats(DP);
-  constexpr int V = E % 2 ? 2 : 4, NV = 2 * E / V, NP = V / 2;
+  constexpr int PER = DP / LP, V = PER % 4 ? 2 : 4, NV = PER / V, NP = V / 2, CG = LP / 8, CP = kScanCols / CG;
+  static_assert(PER % 2 == 0 && (CG == 2 || CG == 4), "pairs of elements, two or four lanes per token");
   extern __shared__ __align__(16) float stage_mem[];
-  const uint32_t h = blockIdx.x, tid = threadIdx.x, lane = tid & 31, l = lane % kScanLanes;
-  const uint32_t c0 = blockIdx.y * kCtaCols + tid / kScanLanes * kScanCols, blocks = (count + kBlock - 1) / kBlock;
-  const bool active = c0 < p.vp;  // uniform over a warp: vp is a multiple of 16
+  __shared__ __align__(8) uint64_t landed[kStages], consumed[kStages];
+  const uint32_t h = blockIdx.x, tid = threadIdx.x, l = tid % LP, tok = l / CG, cg = l % CG, cmask = cg * CP;
+  const uint32_t c0 = blockIdx.y * cta_cols(LP) + tid / LP * kScanCols, blocks = (count + kBlock - 1) / kBlock;
+  if (tid == 0) {
+    const uint32_t cols = min(cta_cols(LP), p.vp - blockIdx.y * cta_cols(LP)), warps = cols * LP / (32 * kScanCols);
+    for (uint32_t i = 0; i < kStages; ++i) {
+      asm volatile("mbarrier.init.shared::cta.b64 [%0], 1;" ::"r"(smem_at(&landed[i])) : "memory");
+      asm volatile("mbarrier.init.shared::cta.b64 [%0], %1;" ::"r"(smem_at(&consumed[i])), "r"(warps) : "memory");
+    }
+    asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
+  }
+  __syncthreads();
+  if (tid >= kScanThreads) {  // a record is one piece of memory: one lane requests them, a ring of stages ahead
+    if (tid > kScanThreads) return;
+    const float *recs = p.blocks + (size_t)h * RF;
+    uint32_t b = 0;
+    for (; b < blocks; ++b) {
+      const uint32_t s = b % kStages, bar = smem_at(&landed[s]);
+      if (b >= kStages && !wait_bounded(&consumed[s], (b / kStages - 1) & 1)) break;
+      asm volatile("mbarrier.arrive.expect_tx.shared::cta.b64 _, [%0], %1;" ::"r"(bar), "r"(RF * 4u) : "memory");
+      asm volatile("cp.async.bulk.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1], %2, [%3];" ::"r"(smem_at(stage_mem + s * RF)),
+                   "l"(recs + (size_t)b * p.heads * RF), "r"(RF * 4u), "r"(bar)
+                   : "memory");
+    }
+    if (b < blocks) {  // given up: what is still on its way lands before the CTA's memory is given back
+      *p.error = 4;
+      for (uint32_t i = b - kStages; i < b; ++i) wait_bounded(&landed[i % kStages], i / kStages & 1);
+    }
+    return;
+  }
+  if (c0 >= p.vp) return;  // a whole warp: vp is a multiple of 16
   float *state = p.state + ((size_t)h * p.vp + c0) * DP;
-  f2 S[kScanCols][E];
+  auto state_at = [&](uint32_t c, int i) { return state + (size_t)(c ^ cmask) * DP + (i * LP + l) * V; };
+  f2 S[kScanCols][NV * NP];
   const bool fresh = first == 0 && *p.pos == 0;
 #pragma unroll
   for (int c = 0; c < (int)kScanCols; ++c)
@@ -302,33 +331,26 @@ template <int E> __global__ void __launch_bounds__(kScanThreads) delta_scan_kern
     for (int i = 0; i < NV; ++i) {
 #pragma unroll
       for (int j = 0; j < NP; ++j) S[c][i * NP + j] = 0;
-      if (active && !fresh) load_pairs<NP>(state + c * DP + (i * kScanLanes + l) * V, &S[c][i * NP]);
+      if (!fresh) load_pairs<NP>(state_at(c, i), &S[c][i * NP]);
     }
-  const float *recs = p.blocks + (size_t)h * RF;
-  auto fetch = [&](uint32_t b) {
-    float *st = stage_mem + (b % kStages) * RF;
-    const float *src = recs + (size_t)b * p.heads * RF;
-    for (uint32_t i = tid * 4; i < RF; i += kScanThreads * 4) copy16(st + i, src + i);
-  };
-  const uint32_t tok = l >> 1;
-  float *vrow = p.v + ((size_t)(first + tok) * p.heads + h) * p.vp + c0 + 2 * (l & 1);
+  float *vrow = p.v + ((size_t)(first + tok) * p.heads + h) * p.vp + c0 + cmask;
   const size_t vstep = (size_t)kBlock * p.heads * p.vp;
-  auto value = [&](uint32_t b) {
-    return active && b * kBlock + tok < count ? *reinterpret_cast<const float2 *>(vrow + b * vstep) : make_float2(0.f, 0.f);
+  float vnext[CP];
+  auto next_values = [&](uint32_t b) {
+    const bool have = b * kBlock + tok < count;
+#pragma unroll
+    for (int c = 0; c < CP; ++c) vnext[c] = have ? vrow[b * vstep + c] : 0.f;
   };
-  for (uint32_t i = 0; i < kStages - 1; ++i) {
-    if (i < blocks) fetch(i);
-    asm volatile("cp.async.commit_group;" ::: "memory");
-  }
-  float2 vnext = value(0);
+  next_values(0);
   for (uint32_t b = 0; b < blocks; ++b) {
-    asm volatile("cp.async.wait_group %0;" ::"n"(kStages - 2) : "memory");
-    __syncthreads();  // this stage has landed for everyone, the one before is consumed
-    if (b + kStages - 1 < blocks) fetch(b + kStages - 1);
-    asm volatile("cp.async.commit_group;" ::: "memory");
-    const float2 v = vnext;
-    if (b + 1 < blocks) vnext = value(b + 1);
-    if (!active) continue;
+    float w[CP], o[CP], u[CP];
+#pragma unroll
+    for (int c = 0; c < CP; ++c) w[c] = vnext[c];
+    if (b + 1 < blocks) next_values(b + 1);
+    if (!__all_sync(0xffffffffu, wait_bounded(&landed[b % kStages], b / kStages & 1))) {
+      *p.error = 4;
+      return;
+    }
     const float *st = stage_mem + (b % kStages) * RF, *mn = st + 25 * DP + tok * kBlock;
     f2 acc[2][kBlock][kScanCols];
 #pragma unroll
@@ -344,56 +366,82 @@ template <int E> __global__ void __launch_bounds__(kScanThreads) delta_scan_kern
 #pragma unroll
         for (int r = 0; r < 2; ++r) {
           f2 x[NP];
-          load_pairs<NP>(st + (r * kBlock + t) * DP + (i * kScanLanes + l) * V, x);
+          load_pairs<NP>(st + (r * kBlock + (t ^ tok)) * DP + (i * LP + l) * V, x);
 #pragma unroll
           for (int j = 0; j < NP; ++j)
 #pragma unroll
             for (int c = 0; c < (int)kScanCols; ++c) acc[r][t][c] = fma2(S[c][i * NP + j], x[j], acc[r][t][c]);
         }
-    const float2 a = scatter_tokens(acc[0], l);
-    float2 o = scatter_tokens(acc[1], l);
-    const float2 w = make_float2(v.x - a.x, v.y - a.y);
-    float2 u = make_float2(0.f, 0.f);
-#pragma unroll
-    for (int s = 0; s < (int)kBlock; ++s) {
-      const float wx = __shfl_sync(0xffffffffu, w.x, 2 * s + (l & 1), kScanLanes), wy = __shfl_sync(0xffffffffu, w.y, 2 * s + (l & 1), kScanLanes);
-      const float m = mn[s], n = mn[kBlock * kBlock + s];
-      u.x = fmaf(m, wx, u.x);
-      u.y = fmaf(m, wy, u.y);
-      o.x = fmaf(n, wx, o.x);
-      o.y = fmaf(n, wy, o.y);
-    }
-    if (b * kBlock + tok < count) *reinterpret_cast<float2 *>(vrow + b * vstep) = o;
 #pragma unroll
     for (int i = 0; i < NV; ++i) {
       f2 x[NP];
-      load_pairs<NP>(st + 3 * kBlock * DP + (i * kScanLanes + l) * V, x);
+      load_pairs<NP>(st + 3 * kBlock * DP + (i * LP + l) * V, x);
 #pragma unroll
       for (int j = 0; j < NP; ++j)
 #pragma unroll
         for (int c = 0; c < (int)kScanCols; ++c) S[c][i * NP + j] = mul2(S[c][i * NP + j], x[j]);
     }
+    float sum[2][kBlock][kScanCols];
+#pragma unroll
+    for (int r = 0; r < 2; ++r) {
+#pragma unroll
+      for (int t = 0; t < (int)kBlock; ++t)
+#pragma unroll
+        for (int c = 0; c < (int)kScanCols; ++c) sum[r][t][c] = add_halves(acc[r][t][c]);
+#pragma unroll
+      for (int bit = kBlock / 2; bit; bit /= 2)
+#pragma unroll
+        for (int t = 0; t < bit; ++t)
+#pragma unroll
+          for (int c = 0; c < (int)kScanCols; ++c) sum[r][t][c] += __shfl_xor_sync(0xffffffffu, sum[r][t + bit][c], bit * CG);
+#pragma unroll
+      for (int n = kScanCols / 2, x = CG / 2; x; n /= 2, x /= 2)
+#pragma unroll
+        for (int c = 0; c < n; ++c) sum[r][0][c] += __shfl_xor_sync(0xffffffffu, sum[r][0][c + n], x);
+    }
+#pragma unroll
+    for (int c = 0; c < CP; ++c) {
+      w[c] -= sum[0][0][c];
+      o[c] = sum[1][0][c];
+      u[c] = 0.f;
+    }
 #pragma unroll
     for (int s = 0; s < (int)kBlock; ++s) {
-      f2 us[kScanCols];
+      const float m = mn[s], n = mn[kBlock * kBlock + s];
 #pragma unroll
-      for (int c = 0; c < (int)kScanCols; ++c) us[c] = both(__shfl_sync(0xffffffffu, c & 1 ? u.y : u.x, 2 * s + (c >> 1), kScanLanes));
+      for (int c = 0; c < CP; ++c) {
+        const float x = __shfl_sync(0xffffffffu, w[c], s * CG + cg, LP);
+        u[c] = fmaf(m, x, u[c]);
+        o[c] = fmaf(n, x, o[c]);
+      }
+    }
+    if (b * kBlock + tok < count) {
+#pragma unroll
+      for (int c = 0; c < CP; ++c) vrow[b * vstep + c] = o[c];
+    }
+    f2 us[kBlock][kScanCols];  // column c ^ cmask is with the lane of its group
+#pragma unroll
+    for (int s = 0; s < (int)kBlock; ++s)
+#pragma unroll
+      for (int c = 0; c < (int)kScanCols; ++c) us[s][c] = both(__shfl_sync(0xffffffffu, u[c % CP], s * CG + ((c / CP) ^ cg), LP));
+#pragma unroll
+    for (int s = 0; s < (int)kBlock; ++s)
 #pragma unroll
       for (int i = 0; i < NV; ++i) {
         f2 x[NP];
-        load_pairs<NP>(st + (2 * kBlock + s) * DP + (i * kScanLanes + l) * V, x);
+        load_pairs<NP>(st + (2 * kBlock + s) * DP + (i * LP + l) * V, x);
 #pragma unroll
         for (int j = 0; j < NP; ++j)
 #pragma unroll
-          for (int c = 0; c < (int)kScanCols; ++c) S[c][i * NP + j] = fma2(x[j], us[c], S[c][i * NP + j]);
+          for (int c = 0; c < (int)kScanCols; ++c) S[c][i * NP + j] = fma2(x[j], us[s][c], S[c][i * NP + j]);
       }
-    }
+    __syncwarp();
+    if ((tid & 31) == 0) asm volatile("mbarrier.arrive.shared::cta.b64 _, [%0];" ::"r"(smem_at(&consumed[b % kStages])) : "memory");
   }
-  if (!active) return;
 #pragma unroll
   for (int c = 0; c < (int)kScanCols; ++c)
 #pragma unroll
-    for (int i = 0; i < NV; ++i) store_pairs<NP>(state + c * DP + (i * kScanLanes + l) * V, &S[c][i * NP]);
+    for (int i = 0; i < NV; ++i) store_pairs<NP>(state_at(c, i), &S[c][i * NP]);
 }
 
 constexpr int kFinishThreads = 256;
@@ -582,10 +630,10 @@ template <class T, int TAPS> cudaError_t launch_blocks(const DeltaRows &p, uint3
   else delta_blocks_kernel<T, TAPS, 256><<<grid, 256, 0, s>>>(p, first);
   return cudaGetLastError();
 }
-template <int E> cudaError_t launch_scan(const DeltaRows &p, uint32_t first, uint32_t count, cudaStream_t s) {
+template <int E, int LP> cudaError_t launch_scan(const DeltaRows &p, uint32_t first, uint32_t count, cudaStream_t s) {
   constexpr size_t smem = (size_t)kStages * block_floats(E * 32) * sizeof(float);
-  if (cudaError_t e = cudaFuncSetAttribute(delta_scan_kernel<E>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem)) return e;
-  delta_scan_kernel<E><<<dim3(p.heads, (p.vp + kCtaCols - 1) / kCtaCols), kScanThreads, smem, s>>>(p, first, count);
+  if (cudaError_t e = cudaFuncSetAttribute(delta_scan_kernel<E, LP>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem)) return e;
+  delta_scan_kernel<E, LP><<<dim3(p.heads, (p.vp + cta_cols(LP) - 1) / cta_cols(LP)), kScanThreads + 32, smem, s>>>(p, first, count);
   return cudaGetLastError();
 }
 // f<E>() for a key width of 32 E.
@@ -631,7 +679,12 @@ cudaError_t launch_delta_rows(const DeltaRows &p, bool f32, cudaStream_t s) {
     const uint32_t count = std::min(kDeltaSlice, p.T - first);
     cudaError_t e = f32 ? (p.ntaps == 4 ? launch_blocks<float, 4>(p, first, count, s) : launch_blocks<float, 0>(p, first, count, s))
                         : (p.ntaps == 4 ? launch_blocks<bf16, 4>(p, first, count, s) : launch_blocks<bf16, 0>(p, first, count, s));
-    if (e == cudaSuccess) e = by_width(p.dp, [&](auto w) { return launch_scan<decltype(w)::value>(p, first, count, s); });
+    if (e == cudaSuccess) e = by_width(p.dp, [&](auto w) {
+      constexpr int E = decltype(w)::value;
+      if constexpr (E % 2 == 0)  // few heads: more SMs, with fewer columns each
+        if (p.heads * (p.vp / 16) <= (uint32_t)p.sms) return launch_scan<E, 32>(p, first, count, s);
+      return launch_scan<E, 16>(p, first, count, s);
+    });
     if (e != cudaSuccess) return e;
   }
   const dim3 grid(p.T, (p.heads + kFinishThreads / 32 - 1) / (kFinishThreads / 32));

@@ -64,7 +64,10 @@ template <class T, int LPR, int NQ, bool SEP> __global__ void __launch_bounds__(
   const uint32_t g = blockIdx.x / groups, hg = blockIdx.x % groups, h0 = g * per + hg * NQ, nh = min((uint32_t)NQ, per - hg * NQ);
   const uint32_t m = blockIdx.y, split = blockIdx.z, tid = threadIdx.x, sub = tid / LPR, l = tid % LPR, e0 = l * 8, warp = tid >> 5;
   const bool ev = e0 < p.dp, vv = SEP && e0 < p.vp;
-  if (p.use_pdl) asm volatile("griddepcontrol.wait;" ::: "memory");
+  if (p.use_pdl) {
+    asm volatile("griddepcontrol.launch_dependents;");  // the out-projection asks for its weights meanwhile
+    asm volatile("griddepcontrol.wait;" ::: "memory");
+  }
   const uint32_t pos = *p.pos + m, vis = pos + 1, lo = first_seen(p, pos);
   const uint32_t splits = min(p.splits, (vis - lo + kSplitRows - 1) / kSplitRows);
   if (split >= splits) return;
@@ -190,7 +193,6 @@ template <class T, int LPR, int NQ, bool SEP> __global__ void __launch_bounds__(
     }
   }
   __syncthreads();
-  if (p.use_pdl) asm volatile("griddepcontrol.launch_dependents;");
   const size_t unit = (size_t)m * gridDim.x + blockIdx.x;
   const uint32_t rec = p.vp + 4;
   float *part = p.scratch + unit * p.splits * NQ * rec;  // [split][NQ][vp + 4]: output, max, sum

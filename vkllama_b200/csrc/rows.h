@@ -217,6 +217,8 @@ struct DeltaRows {
   uint32_t z_ld, z_gate;
   float *v;                 // [T][heads * vp]: values, which the recurrence replaces by its outputs
   float *blocks;            // delta_block_floats(...): what the recurrence needs of the keys, block by block
+  uint32_t *error;          // set when a wait of the kernels runs out
+  int sms;
   // one token
   const bf16 *wl;           // second steps' weights [., low_ld]: decay rows from 0, gate rows from z_gate
   const void *low;          // [2][low_ld] compute type: the first steps' results

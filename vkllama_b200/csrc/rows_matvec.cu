@@ -64,7 +64,8 @@ template <class T> __device__ __forceinline__ void dot4(float (&acc)[4], const b
 
 __device__ __forceinline__ void prefetch_l2(const void *p) { asm volatile("prefetch.global.L2 [%0];" ::"l"(p)); }
 
-template <class T, int KS, bool OUT> __global__ void __launch_bounds__(kThreads) rows_matvec_kernel(const MvRows p) {
+// NORM: the input is p.norm's output, computed here.
+template <class T, int KS, bool OUT, bool NORM> __global__ void __launch_bounds__(kThreads) rows_matvec_kernel(const MvRows p) {
   constexpr uint32_t UPC = kWarps / KS;  // units a CTA works on at a time
   __shared__ float red[2][kWarps][4];
   const uint32_t warp = threadIdx.x >> 5, lane = threadIdx.x & 31, wg = warp / KS, ws = warp % KS;
@@ -86,7 +87,7 @@ template <class T, int KS, bool OUT> __global__ void __launch_bounds__(kThreads)
     asm volatile("griddepcontrol.wait;" ::: "memory");
   }
   const T *x1 = static_cast<const T *>(p.x), *x2 = static_cast<const T *>(p.x2);
-  if (p.norm.x) {  // every CTA for itself
+  if constexpr (NORM) {  // every CTA for itself
     extern __shared__ __align__(16) unsigned char xs_raw[];
     T *xs = reinterpret_cast<T *>(xs_raw);
     rms_row<T, kWarps>(p.norm, p.norm.x, xs, xs + p.K);
@@ -161,12 +162,12 @@ template <class T, int KS, bool OUT> __global__ void __launch_bounds__(kThreads)
   if (p.use_pdl) asm volatile("griddepcontrol.launch_dependents;");
 }
 
-template <class T, int KS, bool OUT> cudaError_t launch_t(const MvRows &p, uint32_t units, int sms, cudaStream_t s) {
-  auto kern = rows_matvec_kernel<T, KS, OUT>;
-  const size_t smem = p.norm.x ? (p.norm.w2 ? 2 : 1) * (size_t)p.K * sizeof(T) : 0;
+template <class T, int KS, bool OUT, bool NORM> cudaError_t launch_t(const MvRows &p, uint32_t units, int sms, cudaStream_t s) {
+  auto kern = rows_matvec_kernel<T, KS, OUT, NORM>;
+  const size_t smem = NORM ? (p.norm.w2 ? 2 : 1) * (size_t)p.K * sizeof(T) : 0;
   auto resident = [](size_t bytes) {
     int n = 0;
-    return cudaOccupancyMaxActiveBlocksPerMultiprocessor(&n, rows_matvec_kernel<T, KS, OUT>, kThreads, bytes) == cudaSuccess && n > 0 ? n : 1;
+    return cudaOccupancyMaxActiveBlocksPerMultiprocessor(&n, rows_matvec_kernel<T, KS, OUT, NORM>, kThreads, bytes) == cudaSuccess && n > 0 ? n : 1;
   };
   static const int without_norm = resident(0);
   const int per_sm = smem ? resident(smem) : without_norm;
@@ -186,16 +187,16 @@ template <class T, int KS, bool OUT> cudaError_t launch_t(const MvRows &p, uint3
   return cudaLaunchKernelEx(&cfg, kern, p);
 }
 
-template <class T, bool OUT> cudaError_t launch_ks(const MvRows &p, int sms, cudaStream_t s) {
+template <class T, bool OUT, bool NORM> cudaError_t launch_ks(const MvRows &p, int sms, cudaStream_t s) {
   const uint32_t units = (p.N - (p.n2 - p.gap0)) / 4 + (OUT ? 0u : p.top * (p.ne / 4));
   // enough warps to keep the memory system busy, as long as each has a step of K of its own
   uint32_t ks = 1;
   while (ks < 8 && units * ks < (uint32_t)sms * 24 && p.K >= 512 * ks) ks *= 2;
   switch (ks) {
-    case 1: return launch_t<T, 1, OUT>(p, units, sms, s);
-    case 2: return launch_t<T, 2, OUT>(p, units, sms, s);
-    case 4: return launch_t<T, 4, OUT>(p, units, sms, s);
-    default: return launch_t<T, 8, OUT>(p, units, sms, s);
+    case 1: return launch_t<T, 1, OUT, NORM>(p, units, sms, s);
+    case 2: return launch_t<T, 2, OUT, NORM>(p, units, sms, s);
+    case 4: return launch_t<T, 4, OUT, NORM>(p, units, sms, s);
+    default: return launch_t<T, 8, OUT, NORM>(p, units, sms, s);
   }
 }
 
@@ -206,8 +207,9 @@ bool rows_matvec_takes_norm(uint32_t K, bool two, bool f32) { return (two ? 2 : 
 cudaError_t launch_rows_matvec(const MvRows &p, bool f32, int sms, cudaStream_t s) {
   if (p.norm.x && (p.norm.ldw != p.K || (p.n2 && !p.norm.w2) || !rows_matvec_takes_norm(p.K, p.norm.w2, f32))) return cudaErrorInvalidValue;
   if (!p.N || p.N % 32 || p.K % 64 || p.gap0 % 32 || p.n2 % 32 || p.gap0 > p.n2 || p.n2 > p.N || (p.top && (p.ke % 64 || p.ne % 32))) return cudaErrorInvalidValue;
-  if (f32) return p.out_proj ? launch_ks<float, true>(p, sms, s) : launch_ks<float, false>(p, sms, s);
-  return p.out_proj ? launch_ks<bf16, true>(p, sms, s) : launch_ks<bf16, false>(p, sms, s);
+  if (p.norm.x) return p.out_proj ? cudaErrorInvalidValue : f32 ? launch_ks<float, false, true>(p, sms, s) : launch_ks<bf16, false, true>(p, sms, s);
+  if (f32) return p.out_proj ? launch_ks<float, true, false>(p, sms, s) : launch_ks<float, false, false>(p, sms, s);
+  return p.out_proj ? launch_ks<bf16, true, false>(p, sms, s) : launch_ks<bf16, false, false>(p, sms, s);
 }
 
 }  // namespace vkl
