@@ -285,7 +285,7 @@ __host__ __device__ constexpr uint32_t cta_cols(uint32_t lp) { return kScanThrea
 // E: 32-element steps of the key width. LP lanes share four columns; lane l holds elements (LP i + l) V .. + V - 1 of
 // each, and ends up with the sums of token tok = l / (LP / 8) for CP of the columns. So that the sums can be exchanged
 // without choosing registers by lane, slot t of a lane's sums is token t ^ tok and slot c column c ^ cmask.
-template <int E, int LP> __global__ void __launch_bounds__(kScanThreads + 32) delta_scan_kernel(const DeltaRows p, uint32_t first, uint32_t count) {
+template <int E, int LP> __global__ void __launch_bounds__(kScanThreads + 32, 1) delta_scan_kernel(const DeltaRows p, uint32_t first, uint32_t count) {
   constexpr uint32_t DP = E * 32, RF = block_floats(DP);
   constexpr int PER = DP / LP, V = PER % 4 ? 2 : 4, NV = PER / V, NP = V / 2, CG = LP / 8, CP = kScanCols / CG;
   static_assert(PER % 2 == 0 && (CG == 2 || CG == 4), "pairs of elements, two or four lanes per token");
