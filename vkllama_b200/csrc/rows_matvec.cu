@@ -85,6 +85,7 @@ template <class T, int KS, bool OUT, bool NORM> __global__ void __launch_bounds_
         for (int r = 0; r < 4; ++r) prefetch_l2(w + (size_t)r * p.K + k);
     }
     asm volatile("griddepcontrol.wait;" ::: "memory");
+    asm volatile("griddepcontrol.launch_dependents;");  // the next kernel asks for its weights as this one's CTAs make room
   }
   const T *x1 = static_cast<const T *>(p.x), *x2 = static_cast<const T *>(p.x2);
   if constexpr (NORM) {  // every CTA for itself
@@ -159,7 +160,6 @@ template <class T, int KS, bool OUT, bool NORM> __global__ void __launch_bounds_
       rows_one<T>(p.out, sg, n + lane, lane == 0 ? acc[0] : lane == 1 ? acc[1] : lane == 2 ? acc[2] : acc[3]);
     }
   }
-  if (p.use_pdl) asm volatile("griddepcontrol.launch_dependents;");
 }
 
 template <class T, int KS, bool OUT, bool NORM> cudaError_t launch_t(const MvRows &p, uint32_t units, int sms, cudaStream_t s) {
