@@ -262,7 +262,9 @@ int vkl_model_synth_weights(vkl_model *m, uint64_t seed, float wstd, float nstd)
  * in many-token passes and takes the last token through the decode kernel: it must
  * end inside the context length, and the last block's query is rotated at the
  * token's own position (the single-device form rotates it at the call's first, as
- * the reference does after clipping Q). */
+ * the reference does after clipping Q). A decoder design with recurrent layers takes a sequence
+ * only on from where it stands: offset is 0 (a new sequence) or the number of tokens that the
+ * passes before have left in its states, else FAILED_PRECONDITION. */
 int vkl_model_forward(vkl_model *m, const uint32_t *toks, size_t n, size_t offset,
                       float *logits_out);
 /* The same pass with the logits of chosen tokens of the call: rows[i] indexes toks, logits_out is
@@ -333,10 +335,10 @@ int vkl_model_block_forward(vkl_model *m, uint32_t layer, const void *x_fp16, si
  * first CTA; 0 on the multi-kernel path, which is timed with an event after every launch).
  * Appends to the KV cache at `offset`. */
 int vkl_model_decode_profile(vkl_model *m, uint32_t token, size_t offset, float out_us[20]);
-/* The same for one pass over n >= 2 prompt tokens from position 0: out_us[0..7] by the classes above. A
+/* The same for one pass over n >= 2 prompt tokens from position 0: out_us[0..9] by the classes above. A
  * decoder design's classes: 1 everything that reads the norm, 2 attention, 3 out-projection of a prompt pass,
  * 4 the experts' gate/up rows (with routing gather), 5 out-projection of a decode step, the experts' down rows
- * and their sum. */
+ * and their sum, 8 a recurrent layer's steps between its projections, 9 norms with a kernel of their own. */
 int vkl_model_prefill_profile(vkl_model *m, const uint32_t *toks, size_t n, float out_us[10]);
 /* The same step with a global-timer stamp (ns) by every CTA of the persistent kernel at six
  * points of every op: out[(op * grid + cta) * 8 + k], k = 0 op entered, 1 input vector
