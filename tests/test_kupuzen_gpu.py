@@ -157,6 +157,18 @@ def test_long_decoding(dev, dtype):
     m.close()
 
 
+@DTYPES
+def test_prompts_of_more_than_a_thousand_tokens_and_many_heads(dev, dtype):
+    """Longer than the delta rule's slices, and state columns enough to fill the GPU's SMs."""
+    case = U.config([(U.delta(40, 20, 64, 64, 4, (6, 11)), 48), (U.delta(10, 5, 100, 256, 4, (13, 5)), None)], width=64, vocab=70)
+    W, toks = U.weights(case, 63), U.tokens(case[0], 1090, 64)
+    want = D.run(case[0], W, toks)
+    m = load(dev, case, W, 1090, dtype)
+    for sizes in ([1090], [7, 1030, 2, 50, 1], [1024, 64, 1]):
+        assert U.rel_err(run_portions(m, toks, sizes), want) < U.REL[dtype], sizes
+    m.close()
+
+
 def test_a_decode_window_that_is_split_over_several_ctas(dev):
     case = U.config([(U.attn(8, 2, 32, 32, 700, 32), 64)], width=64, vocab=60)
     W, toks = U.weights(case, 65), U.tokens(case[0], 1000, 66)
