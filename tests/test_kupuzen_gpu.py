@@ -169,6 +169,17 @@ def test_prompts_of_more_than_a_thousand_tokens_and_many_heads(dev, dtype):
     m.close()
 
 
+def test_a_stream_too_wide_for_the_norm_inside_the_decode_projection(dev):
+    case = U.config([(U.attn(2, 1, 32, 32, 9, 8), 24), (U.delta(2, 1, 32, 16, 4, (5, 5)), 16)], width=6016, vocab=40)
+    W, toks = U.weights(case, 67), U.tokens(case[0], 30, 68)
+    want = D.run(case[0], W, toks)
+    m = load(dev, case, W, 30, "float32")
+    for sizes in ([30], [20, 1]):
+        assert U.rel_err(run_portions(m, toks, sizes), want) < U.REL["float32"], sizes
+    assert m.generate(toks[:20], 2)[0][0] == np.argmax(want[19])
+    m.close()
+
+
 def test_a_decode_window_that_is_split_over_several_ctas(dev):
     case = U.config([(U.attn(8, 2, 32, 32, 700, 32), 64)], width=64, vocab=60)
     W, toks = U.weights(case, 65), U.tokens(case[0], 1000, 66)
